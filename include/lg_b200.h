@@ -70,6 +70,14 @@ void mtp_free_device(struct mtp *t);
 /* model_forward_spec with a run-time width n in [1, 8] (n = 1 is plain decode). */
 int  lg_forward_spec_n(struct model *m, struct kvcache *kv, int n, const int *toks, int pos, int *out);
 
+/* model_prefill that also hands back logits: want[0..n_want) are places in tokens[0..n), in strictly ascending order, and
+ * logits receives one row of n_vocab floats for each.  0, or -1 on bad arguments. */
+int  lg_prefill_logits(struct model *m, struct kvcache *kv, const int *tokens, int n, int pos0, const int *want, int n_want,
+                       float *logits);
+/* 1: models opened from now on run every product and keep their cache in 32-bit (models described by a layer plan only);
+ * 0 (default): the precision the library serves them in.  Set before kvcache_init. */
+void lg_set_compute_f32(int on);
+
 /* Device-resident rounds: [drafts -> verify of width n -> greedy accept -> advance] repeated
  * n_rounds times with NO host synchronisation in between.  mode 0: no drafts (n must be 1),
  * 1: drafts from head t, 2: drafts from the table given to lg_set_replay (head t, if given,

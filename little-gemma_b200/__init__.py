@@ -27,7 +27,7 @@ ABI_SYMBOLS = [
     "model_kv_host", "kvcache_init", "kvcache_free", "kvcache_save_prefix", "kvcache_restore_prefix",
     "model_forward", "model_forward_next", "model_prefill", "model_prefill_embd", "model_prefill_mixed",
     "model_prefill_reserve", "model_forward_spec", "mtp_draft_device", "mtp_draft_chain_device", "mtp_free_device",
-    "lg_forward_spec_n", "lg_set_replay", "lg_rounds_begin", "lg_rounds_enqueue", "lg_rounds_collect",
+    "lg_forward_spec_n", "lg_prefill_logits", "lg_set_compute_f32", "lg_set_replay", "lg_rounds_begin", "lg_rounds_enqueue", "lg_rounds_collect",
     "lg_set_round_width", "lg_set_replay_origin", "lg_host_syncs", "lg_set_draft_margin", "lg_drafts_skipped", "lg_weight_bytes", "lg_round_launches", "lg_last_hidden", "lg_kv_row", "lg_stream", "lg_engine_release",
     "lg_bench_matmul_pass", "lg_bench_prefill_pass", "lg_set_attn_deep", "lg_flash_decode_noalloc",
     "lg_debug_bounded_wait", "lg_debug_stamps", "lg_debug_clear_stamps", "lg_matmul_resid_host",
@@ -48,6 +48,10 @@ def load() -> C.CDLL:
     L = C.CDLL(LIB_PATH)
     L.lgs_open.restype = C.c_void_p
     L.lgs_open.argtypes = [C.c_char_p, C.c_char_p, C.c_int, C.c_int]
+    L.lgs_open_as.restype = C.c_void_p
+    L.lgs_open_as.argtypes = [C.c_char_p, C.c_char_p, C.c_int, C.c_int]
+    L.lgs_prefill_logits.argtypes = [C.c_void_p, _i32p, C.c_int, C.c_int, _i32p, C.c_int, _f32p]; L.lgs_prefill_logits.restype = C.c_int
+    L.lgs_prefix.argtypes = [C.c_void_p, C.c_int, C.c_int]
     L.lgs_close.argtypes = [C.c_void_p]
     for n in ("lgs_n_vocab", "lgs_n_embd", "lgs_n_layer", "lgs_has_head"):
         getattr(L, n).argtypes = [C.c_void_p]; getattr(L, n).restype = C.c_int
@@ -199,11 +203,16 @@ def flash_decode_noalloc(d_q: int, d_k: int, d_v: int, M: int, H: int, n_head_kv
 
 
 class Session:
-    """One loaded target model (+ optional draft head) with its KV cache on the GPU."""
+    """One loaded target model (+ optional draft head) with its KV cache on the GPU.
 
-    def __init__(self, target: str, head: str | None = None, max_seq: int = 4096, mtp_n: int = 4):
+    `target` is a GGUF file or a checkpoint folder (config.json + model.safetensors).  dtype "float32" runs every product and
+    keeps the cache in 32-bit (models described by a layer plan only); None is the precision the library serves the model in."""
+
+    def __init__(self, target: str, head: str | None = None, max_seq: int = 4096, mtp_n: int = 4, dtype: str | None = None):
+        if dtype not in (None, "bfloat16", "float32"):
+            raise ValueError(f"dtype {dtype!r}")
         self.L = load()
-        self.h = self.L.lgs_open(target.encode(), (head or "").encode(), max_seq, 1)
+        self.h = self.L.lgs_open_as(target.encode(), (head or "").encode(), max_seq, int(dtype == "float32"))
         if not self.h:
             raise RuntimeError(f"cannot open {target}")
         self.n_vocab = self.L.lgs_n_vocab(self.h)
@@ -242,6 +251,22 @@ class Session:
     def prefill(self, toks, pos0: int = 0):
         toks = np.ascontiguousarray(toks, dtype=np.int32)
         self.L.lgs_prefill(self.h, toks, len(toks), pos0)
+
+    def prefill_logits(self, toks, pos0: int, want) -> np.ndarray:
+        """Prompt pass over toks at positions pos0.. that returns the logits at the places `want` (indices into toks, any order)."""
+        toks = np.ascontiguousarray(toks, dtype=np.int32)
+        places, back = np.unique(np.asarray(want, dtype=np.int32), return_inverse=True)
+        out = np.empty((len(places), self.n_vocab), dtype=np.float32)
+        if self.L.lgs_prefill_logits(self.h, toks, len(toks), pos0, np.ascontiguousarray(places), len(places), out.reshape(-1)):
+            raise ValueError("tokens, places or positions out of range")
+        return out[back.reshape(-1)]
+
+    def save_prefix(self, n: int):
+        """Keep a copy of the first n cache rows of every layer; restore_prefix brings them back."""
+        self.L.lgs_prefix(self.h, n, 0)
+
+    def restore_prefix(self, n: int):
+        self.L.lgs_prefix(self.h, n, 1)
 
     def prefill_mixed(self, rows, ids, pos0: int = 0):
         """model_prefill_mixed: ids[i] >= 0 is a token id, ids[i] < 0 names embedding row -ids[i]-1 of `rows` [n_rows, n_embd]."""

@@ -19,18 +19,29 @@ CUDA = os.path.join(HERE, "csrc", "cuda")
 LIB = os.path.join(HERE, "liblg_b200.so")
 NVCC = os.environ.get("NVCC", "/usr/local/cuda/bin/nvcc")
 
-HOST_SRC = ["lg_gguf.c", "lg_quant.c", "lg_setup.c", "lg_session.c"]
-CUDA_SRC = ["lg_engine.cu"]
-DEPS = [os.path.join(HOST, f) for f in HOST_SRC + ["lg_host.h"]] + \
-       [os.path.join(CUDA, f) for f in CUDA_SRC + ["lg_kernels.cuh", "lg_capi.cuh", "lg_prefill.cuh", "lg_attn_deep.cuh", "lg_attn_cluster.cuh"]] + \
-       [os.path.join(INC, "lg_abi.h"), os.path.join(INC, "lg_b200.h"), os.path.abspath(__file__)]
+HOST_SRC = ["lg_gguf.c", "lg_ckpt.c", "lg_quant.c", "lg_plan.c", "lg_setup.c", "lg_session.c"]
+CUDA_SRC = {"lg_engine.cu": ["lg_engine.h", "lg_device.cuh", "lg_kernels.cuh", "lg_capi.cuh", "lg_prefill.cuh", "lg_attn_deep.cuh", "lg_attn_cluster.cuh"],
+            "lg_plan.cu": ["lg_engine.h", "lg_device.cuh", "lg_dense.cuh", "lg_latent.cuh"]}
+HEADERS = [os.path.join(INC, f) for f in ("lg_abi.h", "lg_b200.h", "lg_plan.h")] + [os.path.join(HOST, f) for f in ("lg_host.h", "lg_formats.h")]
+SELF = os.path.abspath(__file__)
+
+
+def sources(f: str) -> list[str]:
+    """Everything an object file depends on."""
+    if f in CUDA_SRC:
+        return [os.path.join(CUDA, g) for g in [f] + CUDA_SRC[f]] + HEADERS + [SELF]
+    return [os.path.join(HOST, f)] + HEADERS + [SELF]
+
+
+def newer(deps: list[str], target: str) -> bool:
+    if not os.path.exists(target):
+        return True
+    t = os.path.getmtime(target)
+    return any(os.path.getmtime(d) > t for d in deps)
 
 
 def stale() -> bool:
-    if not os.path.exists(LIB):
-        return True
-    t = os.path.getmtime(LIB)
-    return any(os.path.getmtime(d) > t for d in DEPS)
+    return any(newer(sources(f), LIB) for f in [*HOST_SRC, *CUDA_SRC])
 
 
 def build(mtp_n: int = 4, force: bool = False, ptxas_v: bool = False, stamps: bool = False) -> str:
@@ -38,22 +49,34 @@ def build(mtp_n: int = 4, force: bool = False, ptxas_v: bool = False, stamps: bo
         return LIB
     objdir = os.path.join(HERE, "build")
     os.makedirs(objdir, exist_ok=True)
-    objs = []
     defs = [f"-DLG_MTP_N={mtp_n}"] + (["-DLG_STAMPS"] if stamps else [])     # stamps: profiling build with phase time stamps
-    for f in HOST_SRC:
+    # objects are reused only between builds with the same options
+    tag = os.path.join(objdir, "options")
+    want = " ".join(defs)
+    same = os.path.exists(tag) and open(tag).read() == want
+    jobs, objs = [], []
+    for f in [*CUDA_SRC, *HOST_SRC]:                                          # the CUDA units first: they take longest
         o = os.path.join(objdir, f + ".o")
-        subprocess.check_call(["gcc", "-O2", "-fPIC", "-std=gnu11", "-Wall", "-Wextra", *defs, f"-I{INC}", f"-I{HOST}",
-                               "-c", os.path.join(HOST, f), "-o", o])
         objs.append(o)
-    for f in CUDA_SRC:
-        o = os.path.join(objdir, f + ".o")
-        cmd = [NVCC, "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
-               "-Xcompiler", "-fPIC", *defs, f"-I{INC}", f"-I{HOST}", f"-I{CUDA}", "-c", os.path.join(CUDA, f), "-o", o]
-        if ptxas_v:
-            cmd[1:1] = ["-Xptxas", "-v"]
-        subprocess.check_call(cmd)
-        objs.append(o)
-    subprocess.check_call([NVCC, "-shared", "-o", LIB, *objs, "-lcudart"])
+        if same and not force and not newer(sources(f), o):
+            continue
+        if f in CUDA_SRC:
+            cmd = [NVCC, "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
+                   "-Xcompiler", "-fPIC", *defs, f"-I{INC}", f"-I{HOST}", f"-I{CUDA}", "-c", os.path.join(CUDA, f), "-o", o]
+            if ptxas_v:
+                cmd[1:1] = ["-Xptxas", "-v"]
+        else:
+            cmd = ["gcc", "-O2", "-fPIC", "-std=gnu11", "-Wall", "-Wextra", *defs, f"-I{INC}", f"-I{HOST}",
+                   "-c", os.path.join(HOST, f), "-o", o]
+        jobs.append((cmd, subprocess.Popen(cmd)))
+    failed = [cmd for cmd, p in jobs if p.wait() != 0]
+    if failed:
+        raise subprocess.CalledProcessError(1, failed[0])
+    with open(tag, "w") as t:
+        t.write(want)
+    tmp = f"{LIB}.{os.getpid()}"                                              # a reader never sees half a library
+    subprocess.check_call([NVCC, "-shared", "-o", tmp, *objs, "-lcudart"])
+    os.replace(tmp, LIB)
     return LIB
 
 

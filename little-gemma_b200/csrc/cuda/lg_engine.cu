@@ -8,25 +8,16 @@
 // One engine per process (the reference keeps its device state in file-scope statics too):
 // weights are uploaded and repacked on first use, every forward is a CUDA graph of fused
 // kernels whose parameters never change -- position and token ids live in device memory.
-#include <cstdio>
-#include <cstdlib>
-#include <cstring>
-#include <cmath>
-#include <vector>
-#include <map>
-#include <string>
+#include "lg_engine.h"
 #include "lg_kernels.cuh"
 #include "lg_prefill.cuh"
 #include "lg_attn_deep.cuh"
 #include "lg_attn_cluster.cuh"
-#include "lg_host.h"
-#include "lg_b200.h"
-
-#define LG_CHECK(x) do { cudaError_t e_ = (x); if (e_ != cudaSuccess) { \
-    fprintf(stderr, "lg_b200: CUDA error %s at %s:%d\n", cudaGetErrorString(e_), __FILE__, __LINE__); exit(1); } } while (0)
 
 extern "C" const int model_kv_host = 0;      // cache rows live on the device: mtp.c must call the device hooks
 extern "C" int lg_set_replay(struct model *m, const int *replay, int n);
+
+using namespace lg;
 
 namespace {
 
@@ -34,147 +25,7 @@ constexpr int RING_SPARE = 1024;             // ring rows beyond the window (cov
 
 constexpr int LOG_CAP = 1 << 20;
 
-struct WMat {
-    uint4 *wq = nullptr; uint2 *ws = nullptr; uint2 *wd = nullptr; uint4 *wm = nullptr;      // tiles, scales (see lg_kernels.cuh)
-    int fmt = 0, m = 0, k = 0, nkp = 0, n_row_tiles = 0, ldo = 0;
-    size_t file_bytes = 0;
-};
-
-struct Panel { LgPanel p{}; };
-
-struct LayerW {
-    WMat qkv, o, gateup, down, inp_gate, proj;
-    // q / k / v tensors of different formats cannot share one stacked matrix: they are kept apart, each multiplied on its
-    // own into its rows of the projection buffer (qkv then only carries the row stride)
-    std::vector<WMat> qkv_parts; std::vector<int> qkv_row0;
-    float *attn_norm = nullptr, *q_norm = nullptr, *k_norm = nullptr, *post_attn = nullptr, *ffn_norm = nullptr,
-          *post_ffw = nullptr, *post_norm = nullptr;
-    float out_scale = 1.0f;
-    int has_v = 1, owns_kv = 1, src = 0, local = 0, hd = 0, nkv = 0, nff = 0;
-};
-
-struct DraftBlockW {
-    WMat q, o, gateup, down;
-    float *attn_norm, *q_norm, *post_attn, *ffn_norm, *post_ffw;
-    float out_scale; int hd, local, src;
-};
-struct DraftW {
-    WMat pre, post, head;
-    float *out_norm = nullptr;
-    std::vector<DraftBlockW> blk;
-    int ni = 0, nb = 0, nff = 0, n_head = 0, n_vocab = 0, has_post = 0;
-    float eps = 0, base_full = 0, base_swa = 0, softcap = 0;
-    // activations (one token)
-    float *cat = nullptr, *x = nullptr, *hbuf = nullptr, *qbuf = nullptr, *qrot = nullptr, *obuf = nullptr, *gu = nullptr, *part = nullptr;
-    float *amax_val = nullptr; int *amax_idx = nullptr, *best = nullptr;
-    float *amax_val2 = nullptr, *margin = nullptr;      // runner-up logits per CTA; best - second best of the latest draft
-    float2 *part_ml = nullptr;
-    LgPanel p_cat{}, p_ni{}, p_attn{}, p_ff{};
-    float2 *rope_local = nullptr, *rope_global = nullptr; int hd_local = 0, hd_global = 0;
-    int n_slots_local = 0, n_slots_global = 0;
-    std::map<std::string, cudaGraphExec_t> graphs;
-};
-
-// Buffers of the wide prompt pass (blocks of up to LG_PF_MAXN tokens), allocated at its first use.
-struct PrefillBuf {
-    bool ready = false;
-    __half *a_ne = nullptr, *a_attn = nullptr, *a_ff = nullptr;     // f16 matmul inputs [LG_PF_MAXN][k]
-    float *x = nullptr, *qkv = nullptr, *o = nullptr;               // residual rows, projection rows, o/down rows
-    int *toks = nullptr, *pos = nullptr;                            // token ids; pos[g] = position of the g-th group of 8
-    float2 *rope_local = nullptr, *rope_global = nullptr;
-    __half *q_hi = nullptr, *q_lo = nullptr;                        // normed + rotated queries [LG_PF_MAXN][H][hd], f16 hi + lo
-    float *tokrow = nullptr, *pproj = nullptr, *ipl = nullptr, *pg = nullptr;   // per-layer-embedding rows [LG_PF_MAXN][ple * n_layer], gate rows
-    __half *a_ple = nullptr;
-    float *rows = nullptr; int *ridx = nullptr;                     // media rows of the block and, per token, its row or -1
-    int ld_attn = 0, ld_ff = 0;
-};
-
-struct Engine {
-    const struct model *m = nullptr;
-    const struct gguf_context *ctx = nullptr;
-    cudaStream_t stream = nullptr;
-    int sm_count = 148;
-    // weights
-    std::vector<LayerW> L;
-    WMat head, pmp;                           // token_embd (tied head), per_layer_model_proj
-    uint8_t *ple_table = nullptr; int ple_table_type = 0;   // per_layer_token_embd, file layout
-    float *out_norm = nullptr, *ple_proj_norm = nullptr, *rope_div = nullptr;
-    float2 *rope_local = nullptr, *rope_global = nullptr; int hd_local = 0, hd_global = 0;
-    int has_ple = 0;
-    size_t weight_bytes = 0;
-    // activations
-    float *x = nullptr, *qkv = nullptr, *qrot = nullptr, *oout = nullptr, *gu = nullptr, *dout = nullptr, *hidden = nullptr,
-          *h_prev = nullptr, *part = nullptr, *tokrow = nullptr, *pproj = nullptr, *ipl = nullptr, *pg = nullptr, *logits = nullptr;
-    float *amax_val = nullptr; int *amax_idx = nullptr;
-    float2 *part_ml = nullptr;
-    LgPanel p_ne{}, p_attn{}, p_ff{}, p_ple{};
-    int max_ks = 4, head_ctas = 0;
-    int part_slots = 0;
-    // session
-    LgRoundState *st = nullptr;               // device
-    LgRoundState *st_host = nullptr;          // pinned mirror for uploads / downloads
-    int *log = nullptr, *replay = nullptr, *d_n_replay = nullptr; int n_replay = 0, replay_cap = 0;   // replay table (capacity grows; its length lives on the device)
-    int *err = nullptr, *tickets = nullptr;
-    std::map<std::string, cudaGraphExec_t> graphs;
-    const struct kvcache *kv_bound = nullptr;
-    DraftW *draft = nullptr; const struct mtp *draft_owner = nullptr;
-    float *pick_rows = nullptr;               // host logits rows for model_pick
-    long long launches = 0;                   // kernels enqueued by the most recent graph build
-    int pdl = 1;                              // programmatic dependent launch (LG_PDL=0 turns it off)
-    long long round_launches = 0;
-    PrefillBuf pf;
-    float4 *sums = nullptr;                   // SUMS epilogue: per work item and token the partial sums the next kernel builds the norms from
-    int pos_hi = 0;                           // host-side upper bound of the device position (device-resident rounds)
-    // One host synchronisation per round behind the blocking calls: mtp_draft_device runs the WHOLE round and keeps its
-    // outcome here; the chained-draft and verify calls that follow are answered from it when they ask what was computed.
-    struct { bool valid = false; int n = 0, pos = 0, adv = 0, toks[LG_MAXM] = {0}, out[LG_MAXM] = {0}; bool chained = false; } lazy;
-    int replay_off = 0; bool lazy_replay = false;   // replay table index of a draft = its position + replay_off (lg_set_replay_origin)
-    long long host_syncs = 0;                 // blocking device-to-host waits made by the reference-shaped calls
-    float *d_margin_thr = nullptr;            // confidence margin below which a draft calls off the drafts after it (0: never)
-    cudaEvent_t mid_event = nullptr;          // LG_MTP_PROFILE: recorded between the layers and the head of a forward
-    int mm_launches = 0;                      // kernels in the captured matmul-only pass             // kernels in one captured round (lg_rounds_enqueue)
-};
-
 Engine *g_eng = nullptr;
-
-// Kernel launch on the engine's stream, marked for programmatic dependent launch so the kernel may
-// start while its predecessor drains (every forward kernel begins with pdl_wait()).
-template <typename... KArgs, typename... Args>
-void launch_k(Engine *e, void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, Args... args) {
-    cudaLaunchConfig_t cfg = {};
-    cfg.gridDim = grid; cfg.blockDim = block; cfg.dynamicSmemBytes = smem; cfg.stream = e->stream;
-    cudaLaunchAttribute at[1];
-    at[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-    at[0].val.programmaticStreamSerializationAllowed = 1;
-    cfg.attrs = at; cfg.numAttrs = e->pdl ? 1 : 0;
-    LG_CHECK(cudaLaunchKernelEx(&cfg, kernel, KArgs(args)...));
-    e->launches++;
-}
-// The same with the CTAs of one blockIdx.x forming a thread-block cluster (1, grid.y, 1).
-template <typename... KArgs, typename... Args>
-void launch_k_cluster_y(Engine *e, void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, Args... args) {
-    cudaLaunchConfig_t cfg = {};
-    cfg.gridDim = grid; cfg.blockDim = block; cfg.dynamicSmemBytes = smem; cfg.stream = e->stream;
-    cudaLaunchAttribute at[2];
-    at[0].id = cudaLaunchAttributeClusterDimension;
-    at[0].val.clusterDim.x = 1; at[0].val.clusterDim.y = grid.y; at[0].val.clusterDim.z = 1;
-    at[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-    at[1].val.programmaticStreamSerializationAllowed = 1;
-    cfg.attrs = at; cfg.numAttrs = e->pdl ? 2 : 1;
-    LG_CHECK(cudaLaunchKernelEx(&cfg, kernel, KArgs(args)...));
-    e->launches++;
-}
-
-
-// Zero-filled device allocation.  The fill runs on the legacy stream, which does not order against the
-// engine's non-blocking stream, so wait for it before anyone can use the buffer.
-template <typename T> T *dalloc(size_t n) {
-    T *p = nullptr;
-    LG_CHECK(cudaMalloc(&p, n * sizeof(T) > 0 ? n * sizeof(T) : 16));
-    LG_CHECK(cudaMemset(p, 0, n * sizeof(T)));
-    LG_CHECK(cudaDeviceSynchronize());
-    return p;
-}
 
 LgPanel panel_alloc(int k) {
     LgPanel P;
@@ -185,25 +36,6 @@ LgPanel panel_alloc(int k) {
 }
 void panel_free(LgPanel &P) { cudaFree(P.q); cudaFree(P.s); P.q = nullptr; P.s = nullptr; }
 
-// Host -> device copy that is complete on return.  A pageable-source cudaMemcpy may return while
-// its last DMA is still in flight on the legacy stream, which the engine's non-blocking stream does
-// not order against, so wait for the device.
-void h2d_sync(void *dst, const void *src, size_t bytes) {
-    LG_CHECK(cudaMemcpy(dst, src, bytes, cudaMemcpyHostToDevice));
-    LG_CHECK(cudaDeviceSynchronize());
-}
-
-float *upload_f32(const float *src, size_t n) {
-    float *d = dalloc<float>(n);
-    h2d_sync(d, src, n * 4);
-    return d;
-}
-
-const struct gguf_tensor *find_t(const struct gguf_context *g, int L, const char *leaf) {
-    char name[96];
-    if (L >= 0) snprintf(name, sizeof name, "blk.%d.%s", L, leaf); else snprintf(name, sizeof name, "%s", leaf);
-    return gguf_find_tensor(g, name);
-}
 float *upload_norm(const struct gguf_context *g, int L, const char *leaf) {
     const struct gguf_tensor *t = find_t(g, L, leaf);
     if (!t) return nullptr;
@@ -331,7 +163,6 @@ void free_wmat(WMat &W) { cudaFree(W.wq); cudaFree(W.ws); cudaFree(W.wd); cudaFr
 // ------------------------------------------------------------------------------------------
 // launch helpers
 // ------------------------------------------------------------------------------------------
-int env_int(const char *name, int fb) { const char *v = getenv(name); return v && v[0] ? atoi(v) : fb; }
 
 struct GemvPlan { int r, ks, gx, ns, cl; size_t smem; };
 // dynamic shared memory of the small-M matmul: panel slice | ring | warp partials | item sums | peers' sums (cluster) | mbarriers
@@ -640,47 +471,12 @@ size_t attn_smem(int nq, int hd) {
 // ---- the wide (prompt) matmul -----------------------------------------------------------------
 // Tiled-copy descriptor of an f16 activation block [rows][k] (row-major), box = 64 columns x nt rows,
 // 128-byte swizzle: the layout tcgen05.mma reads as a K-major operand.
-typedef CUresult (*EncodeTiledFn)(CUtensorMap *, CUtensorMapDataType, cuuint32_t, void *, const cuuint64_t *, const cuuint64_t *,
-                                  const cuuint32_t *, const cuuint32_t *, CUtensorMapInterleave, CUtensorMapSwizzle,
-                                  CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
 CUtensorMap act_tensor_map(const __half *ptr, int k, int rows, int nt) {
-    static EncodeTiledFn fn = nullptr;
-    if (!fn) {
-        void *p = nullptr;
-        cudaDriverEntryPointQueryResult qr;
-        LG_CHECK(cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &p, cudaEnableDefault, &qr));
-        if (!p || qr != cudaDriverEntryPointSuccess) { fprintf(stderr, "lg_b200: the driver has no cuTensorMapEncodeTiled\n"); exit(1); }
-        fn = (EncodeTiledFn)p;
-    }
-    CUtensorMap map;
-    cuuint64_t dims[2] = {(cuuint64_t)k, (cuuint64_t)rows};
-    cuuint64_t strides[1] = {(cuuint64_t)k * 2};
-    cuuint32_t box[2] = {(cuuint32_t)LG_PF_BK, (cuuint32_t)nt};
-    cuuint32_t estr[2] = {1, 1};
-    CUresult r = fn(&map, CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 2, (void *)ptr, dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
-                    CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
-    if (r != CUDA_SUCCESS) { fprintf(stderr, "lg_b200: cuTensorMapEncodeTiled failed (%d) for k=%d rows=%d\n", (int)r, k, rows); exit(1); }
-    return map;
+    return tiled_map(ptr, CU_TENSOR_MAP_DATA_TYPE_FLOAT16, k, rows, (long long)k * 2, LG_PF_BK, nt);
 }
 
 CUtensorMap kv_tensor_map(const __half *ptr, int kv_dim, int seq, int S) {
-    static EncodeTiledFn fn = nullptr;
-    if (!fn) {
-        void *p = nullptr;
-        cudaDriverEntryPointQueryResult qr;
-        LG_CHECK(cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &p, cudaEnableDefault, &qr));
-        if (!p || qr != cudaDriverEntryPointSuccess) { fprintf(stderr, "lg_b200: the driver has no cuTensorMapEncodeTiled\n"); exit(1); }
-        fn = (EncodeTiledFn)p;
-    }
-    CUtensorMap map;
-    cuuint64_t dims[2] = {(cuuint64_t)kv_dim, (cuuint64_t)seq};
-    cuuint64_t strides[1] = {(cuuint64_t)kv_dim * 2};
-    cuuint32_t box[2] = {64u, (cuuint32_t)S};
-    cuuint32_t estr[2] = {1, 1};
-    CUresult r = fn(&map, CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 2, (void *)ptr, dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
-                    CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
-    if (r != CUDA_SUCCESS) { fprintf(stderr, "lg_b200: cuTensorMapEncodeTiled failed (%d) for a cache of %d rows x %d\n", (int)r, seq, kv_dim); exit(1); }
-    return map;
+    return tiled_map(ptr, CU_TENSOR_MAP_DATA_TYPE_FLOAT16, kv_dim, seq, (long long)kv_dim * 2, 64, S);
 }
 
 template <int NT, int FMT> void launch_pf_nt(Engine *e, const CUtensorMap &tm, const LgPfGemmArgs &a, int epi, dim3 grid) {
@@ -876,6 +672,14 @@ int tiles_for(int window, int max_seq, int M, int hd) {
 // engine construction
 // ------------------------------------------------------------------------------------------
 void engine_free(Engine *e);
+bool g_compute_f32 = false;                   // lg_set_compute_f32: the next model opened runs in 32-bit
+
+void session_state(Engine *e) {
+    e->st = dalloc<LgRoundState>(1);
+    LG_CHECK(cudaMallocHost(&e->st_host, sizeof(LgRoundState)));
+    memset(e->st_host, 0, sizeof(LgRoundState));
+    e->log = dalloc<int>(LOG_CAP);
+}
 
 Engine *engine_for(const struct model *m) {
     if (g_eng && g_eng->m == m && g_eng->ctx == m->ctx) return g_eng;
@@ -898,6 +702,22 @@ Engine *engine_for(const struct model *m) {
     { float thr = (float)atof(getenv("LG_DRAFT_MARGIN") ? getenv("LG_DRAFT_MARGIN") : "0"); if (thr != 0.0f) h2d_sync(e->d_margin_thr, &thr, 4); }
 
     const int ne = c->n_embd, H = c->n_head, ple = c->n_embd_per_layer;
+    e->fam = lg_family_for ? lg_family_for(g) : nullptr;
+    if (e->fam) {
+        // another family: its own weights and activations; the residual rows, hidden rows, argmax candidates and the round
+        // state are the engine's
+        e->f32 = g_compute_f32;
+        e->x = dalloc<float>((size_t)LG_MAXM * ne);
+        e->hidden = dalloc<float>((size_t)LG_MAXM * ne);
+        e->h_prev = dalloc<float>(ne);
+        e->amax_val = dalloc<float>((size_t)e->head_ctas * LG_MAXM);
+        e->amax_idx = dalloc<int>((size_t)e->head_ctas * LG_MAXM);
+        session_state(e);
+        e->fam->load(e);
+        g_eng = e;
+        return e;
+    }
+    if (g_compute_f32) { fprintf(stderr, "lg_b200: the block-quantised models do not run in 32-bit\n"); exit(1); }
     const struct gguf_tensor *emb = find_t(g, -1, "token_embd.weight");
     if (!emb) { fprintf(stderr, "lg_b200: token_embd.weight is missing\n"); exit(1); }
     e->head = build_wmat(e, {emb});
@@ -991,10 +811,7 @@ Engine *engine_for(const struct model *m) {
     }
     e->amax_val = dalloc<float>((size_t)e->head_ctas * LG_MAXM);
     e->amax_idx = dalloc<int>((size_t)e->head_ctas * LG_MAXM);
-    e->st = dalloc<LgRoundState>(1);
-    LG_CHECK(cudaMallocHost(&e->st_host, sizeof(LgRoundState)));
-    memset(e->st_host, 0, sizeof(LgRoundState));
-    e->log = dalloc<int>(LOG_CAP);
+    session_state(e);
     g_eng = e;
     return e;
 }
@@ -1024,6 +841,7 @@ void engine_free(Engine *e) {
     cudaStreamSynchronize(e->stream);
     free_graphs(e->graphs);
     draft_free(e->draft);
+    if (e->fam) e->fam->release(e);
     for (auto &w : e->L) {
         free_wmat(w.qkv); free_wmat(w.o); free_wmat(w.gateup); free_wmat(w.down); free_wmat(w.inp_gate); free_wmat(w.proj);
         for (auto &pw : w.qkv_parts) free_wmat(pw);
@@ -1045,10 +863,11 @@ void engine_free(Engine *e) {
 
 // Scratch for the flash-decode partials depends on the cache geometry; (re)bind when the cache changes.
 void bind_kv(Engine *e, const struct kvcache *kv) {
-    if (e->kv_bound == kv && e->part) return;
+    if (e->kv_bound == kv && (e->part || e->fam)) return;
     LG_CHECK(cudaStreamSynchronize(e->stream));
     free_graphs(e->graphs);
     if (e->draft) free_graphs(e->draft->graphs);
+    if (e->fam) { e->fam->bind(e, kv); e->kv_bound = kv; return; }
     const struct config *c = &e->m->cfg;
     int slots = 0, maxhd = 0;
     for (int l = 0; l < c->n_layer; l++) {
@@ -1067,13 +886,14 @@ void bind_kv(Engine *e, const struct kvcache *kv) {
 // ------------------------------------------------------------------------------------------
 // the forward of M token rows (enqueue only; captured into graphs by the callers)
 // ------------------------------------------------------------------------------------------
-enum { F_HEAD = 1, F_LOGITS = 2, F_ACCEPT = 4, F_ADVANCE = 8, F_NOEMBED = 16 };   // NOEMBED: x rows are already in place
-
-// `only` selects kernel classes (the benchmark times them in isolation); the default runs everything.
-// C_FUSED: a class-restricted pass keeps the epilogue variants of the full step (the o / down / PLE projections that leave
-// complete rows and the partial sums of the norms that follow them) instead of the plain ones.
-enum { C_QKV = 1, C_O = 2, C_GATEUP = 4, C_DOWN = 8, C_HEAD = 16, C_PLE = 32, C_NORM = 64, C_ATTN = 256, C_MISC = 512,
-       C_ALL = 1023, C_FUSED = 1024 };
+// The end of a forward with a head: greedy successors from the argmax candidates, acceptance, position advance.
+void enqueue_pick(Engine *e, int M, int flags, int gx, int only) {
+    const int ne = e->m->cfg.n_embd;
+    if (!(flags & F_HEAD)) return;
+    if (only & C_MISC) launch_k(e, lg_argmax_final, dim3(M), dim3(256), 0, (const float *)e->amax_val, (const int *)e->amax_idx, gx, e->st->out, (const float *)nullptr, (float *)nullptr);
+    if ((flags & F_ACCEPT) && (only & C_MISC))
+        launch_k(e, lg_accept_kernel, dim3(1), dim3(256), 0, e->st, M, e->hidden, ne, ne, e->h_prev, e->log, LOG_CAP, (flags & F_ADVANCE) ? 1 : 0);
+}
 
 void enqueue_forward(Engine *e, const struct kvcache *kv, int M, int flags, int only = C_ALL | C_FUSED) {
     const struct model *m = e->m;
@@ -1081,6 +901,11 @@ void enqueue_forward(Engine *e, const struct kvcache *kv, int M, int flags, int 
     const int ne = c->n_embd, H = c->n_head, ple = c->n_embd_per_layer, nl = c->n_layer;
     const int *d_toks = e->st->toks, *d_pos = &e->st->pos;
 
+    if (e->fam) {
+        const int gx = e->fam->forward(e, kv, M, flags, only);
+        enqueue_pick(e, M, flags, gx, only);
+        return;
+    }
     if ((only & C_MISC) && !(flags & F_NOEMBED))
         launch_k(e, lg_embed_rows, dim3(M), dim3(1024), 0, e->head.wq, e->head.ws, e->head.wd, e->head.wm, e->head.fmt, e->head.nkp, e->head.m, d_toks,
                  sqrtf((float)ne), e->x, ne);
@@ -1187,10 +1012,7 @@ void enqueue_forward(Engine *e, const struct kvcache *kv, int M, int flags, int 
         int gx = 0;
         GemvExtra xh; xh.softcap = c->logit_softcap; xh.logits = lg; xh.amax_val = e->amax_val; xh.amax_idx = e->amax_idx; xh.gx_out = &gx;
         if (only & C_HEAD) launch_gemv(e, e->head, e->p_ne, M, nullptr, LG_EPI_HEAD, 1, xh); else gx = 1;
-        if (only & C_MISC) launch_k(e, lg_argmax_final, dim3(M), dim3(256), 0, (const float *)e->amax_val, (const int *)e->amax_idx, gx, e->st->out, (const float *)nullptr, (float *)nullptr);
-        if (flags & F_ACCEPT) {
-            if (only & C_MISC) launch_k(e, lg_accept_kernel, dim3(1), dim3(256), 0, e->st, M, e->hidden, ne, ne, e->h_prev, e->log, LOG_CAP, (flags & F_ADVANCE) ? 1 : 0);
-        }
+        enqueue_pick(e, M, flags, gx, only);
     }
 }
 
@@ -1405,12 +1227,14 @@ void upload_round(Engine *e, const int *toks, int n, int pos) {
     LG_CHECK(cudaMemcpyAsync(e->st, h, sizeof(int) * (1 + n), cudaMemcpyHostToDevice, e->stream));
 }
 
-void check_err(Engine *e) {
+}  // namespace
+void lg::check_err(Engine *e) {
     int err = 0;
     LG_CHECK(cudaMemcpyAsync(&err, e->err, sizeof(int), cudaMemcpyDeviceToHost, e->stream));
     LG_CHECK(cudaStreamSynchronize(e->stream));
     if (err) { fprintf(stderr, "lg_b200: device status %d (a bounded wait inside a kernel gave up)\n", err); exit(1); }
 }
+namespace {
 
 // ------------------------------------------------------------------------------------------
 // draft head
@@ -1545,7 +1369,7 @@ void enqueue_draft(Engine *e, DraftW *d, const struct kvcache *kv, int slot, boo
 }
 
 DraftW *draft_for(Engine *e, struct mtp *t, const struct kvcache *kv) {
-    if (t->cuda == (void *)-1) return nullptr;
+    if (t->cuda == (void *)-1 || e->fam) return nullptr;       // heads read a block-quantised target's K / V rows
     if (e->draft && e->draft_owner == t) return e->draft;
     if (e->draft) { draft_free(e->draft); e->draft = nullptr; }
     e->draft = draft_build(e, t, kv);
@@ -1677,6 +1501,11 @@ int kvcache_init(struct kvcache *kv, const struct model *m, int max_seq) {
     kv->k = (void **)calloc(c->n_layer, sizeof(void *));
     kv->v = (void **)calloc(c->n_layer, sizeof(void *));
     if (!kv->kv_dim || !kv->seq || !kv->f16 || !kv->k || !kv->v) return -1;
+    if (const LgFamily *fam = lg_family_for ? lg_family_for(m->ctx) : nullptr) {
+        if (fam->kv_init(kv, m, g_compute_f32) != 0) return -1;
+        LG_CHECK(cudaDeviceSynchronize());
+        return 0;
+    }
     for (int L = 0; L < c->n_layer; L++) {
         kv->kv_dim[L] = m->n_head_kv[L] * m->head_dim[L];
         if (L >= c->n_kv_start) continue;
@@ -1709,6 +1538,9 @@ void kvcache_free(struct kvcache *kv) {
     kv->kv_dim = kv->seq = kv->f16 = nullptr;
 }
 
+// bytes per cache element: f16 (1) and bf16 (2) rows, f32 (0) rows
+static size_t kv_elem(const struct kvcache *kv, int L) { return kv->f16[L] ? 2 : 4; }
+
 void kvcache_save_prefix(struct kvcache *kv, int n) {
     kv->px_k = (void **)calloc(kv->n_layer, sizeof(void *));
     kv->px_v = (void **)calloc(kv->n_layer, sizeof(void *));
@@ -1717,9 +1549,11 @@ void kvcache_save_prefix(struct kvcache *kv, int n) {
     for (int L = 0; L < kv->n_layer; L++) {
         if (!kv->k[L]) continue;
         int rows = n < kv->seq[L] ? n : kv->seq[L];
-        size_t bytes = (size_t)rows * kv->kv_dim[L] * 2;
-        LG_CHECK(cudaMalloc(&kv->px_k[L], bytes)); LG_CHECK(cudaMalloc(&kv->px_v[L], bytes));
+        size_t bytes = (size_t)rows * kv->kv_dim[L] * kv_elem(kv, L);
+        LG_CHECK(cudaMalloc(&kv->px_k[L], bytes));
         LG_CHECK(cudaMemcpy(kv->px_k[L], kv->k[L], bytes, cudaMemcpyDeviceToDevice));
+        if (!kv->v[L]) continue;                     // one row per position holds keys and values (latent rows)
+        LG_CHECK(cudaMalloc(&kv->px_v[L], bytes));
         LG_CHECK(cudaMemcpy(kv->px_v[L], kv->v[L], bytes, cudaMemcpyDeviceToDevice));
     }
     LG_CHECK(cudaDeviceSynchronize());
@@ -1731,9 +1565,9 @@ void kvcache_restore_prefix(struct kvcache *kv, int n) {
     for (int L = 0; L < kv->n_layer; L++) {
         if (!kv->px_k[L]) continue;
         int rows = n < kv->seq[L] ? n : kv->seq[L];
-        size_t bytes = (size_t)rows * kv->kv_dim[L] * 2;
+        size_t bytes = (size_t)rows * kv->kv_dim[L] * kv_elem(kv, L);
         LG_CHECK(cudaMemcpyAsync(kv->k[L], kv->px_k[L], bytes, cudaMemcpyDeviceToDevice, s));
-        LG_CHECK(cudaMemcpyAsync(kv->v[L], kv->px_v[L], bytes, cudaMemcpyDeviceToDevice, s));
+        if (kv->px_v[L]) LG_CHECK(cudaMemcpyAsync(kv->v[L], kv->px_v[L], bytes, cudaMemcpyDeviceToDevice, s));
     }
 }
 
@@ -1757,7 +1591,9 @@ int model_forward_next(struct model *m, struct kvcache *kv, int token, int pos) 
 
 // The prompt pass.  ids[i] >= 0: token id; ids[i] < 0 (only with rows): media position, embedding row -ids[i]-1 of
 // `rows` enters as it is and the per-layer table row of token 0 is used (src/cpu/model-cpu.c:459-465,489-497).
-static void prefill_impl(struct model *m, struct kvcache *kv, const float *rows, const int *ids, int n, int pos0) {
+// want / n_want: places whose logits are asked for, in ascending order; they go to logits [n_want][n_vocab].
+static void prefill_impl(struct model *m, struct kvcache *kv, const float *rows, const int *ids, int n, int pos0,
+                         const int *want = nullptr, int n_want = 0, float *logits = nullptr) {
     Engine *e = engine_for(m);
     const int ne = m->cfg.n_embd;
     if (n <= 0) return;
@@ -1770,7 +1606,15 @@ static void prefill_impl(struct model *m, struct kvcache *kv, const float *rows,
         if (ids[i] < 0) { if (!rows) { fprintf(stderr, "lg_b200: a media position without embedding rows\n"); exit(1); } media = true; }
     }
     int i = 0;
-    if (prefill_wide_ok(e) && n >= 4 * LG_MAXM) {
+    const size_t n_vocab = (size_t)m->cfg.n_vocab;
+    if (e->fam && !media && n > LG_MAXM) {
+        bind_kv(e, kv);
+        i = e->fam->prefill(e, kv, toks.data(), n, pos0, want, n_want, logits);
+    }
+    // the wide pass leaves no logits: with places asked for, it ends before the first of them
+    const int n_all = n, n_wide = n_want > 0 ? std::min(n, want[0]) : n;
+    if (!e->fam && prefill_wide_ok(e) && n_wide >= 4 * LG_MAXM) {
+        n = n_wide;
         // Blocks of up to LG_PF_MAXN tokens on the wide pass.  A ragged tail of more than one attention group is padded to
         // a whole number of groups by repeating the last token (src/cuda/prefill-kernel.cuh:631-660 pads its tail the same
         // way): the cache rows the pad positions write lie past the prompt, where the next step overwrites them before any
@@ -1811,7 +1655,10 @@ static void prefill_impl(struct model *m, struct kvcache *kv, const float *rows,
             i += real;
         }
         check_err(e);                                               // the one wait: every copy above has read its host buffer by now
+        n = n_all;
     }
+    int w = 0;
+    while (w < n_want && want[w] < i) w++;
     for (; i < n; i += LG_MAXM) {
         int b = n - i < LG_MAXM ? n - i : LG_MAXM;
         upload_round(e, toks.data() + i, b, pos0 + i);
@@ -1819,16 +1666,22 @@ static void prefill_impl(struct model *m, struct kvcache *kv, const float *rows,
         for (int j = 0; j < b; j++) blk_media |= ids[i + j] < 0;
         if (blk_media) {
             // token embeddings first, then the media rows over them; the forward then starts from x as it stands
-            launch_k(e, lg_embed_rows, dim3(b), dim3(256), 0, e->head.wq, e->head.ws, e->head.wd, e->head.wm, e->head.fmt, e->head.nkp, e->head.m,
-                     (const int *)e->st->toks, sqrtf((float)ne), e->x, ne);
+            if (e->fam) e->fam->embed(e, b);
+            else launch_k(e, lg_embed_rows, dim3(b), dim3(256), 0, e->head.wq, e->head.ws, e->head.wd, e->head.wm, e->head.fmt, e->head.nkp, e->head.m,
+                          (const int *)e->st->toks, sqrtf((float)ne), e->x, ne);
             for (int j = 0; j < b; j++)
                 if (ids[i + j] < 0)
                     LG_CHECK(cudaMemcpyAsync(e->x + (size_t)j * ne, rows + (size_t)(-ids[i + j] - 1) * ne, sizeof(float) * ne,
                                              cudaMemcpyHostToDevice, e->stream));
         }
-        run_forward(e, kv, b, blk_media ? F_NOEMBED : 0);
+        const bool head = w < n_want && want[w] < i + b;
+        run_forward(e, kv, b, (blk_media ? F_NOEMBED : 0) | (head ? F_HEAD | F_LOGITS : 0));
+        for (; w < n_want && want[w] < i + b; w++)
+            LG_CHECK(cudaMemcpyAsync(logits + (size_t)w * n_vocab, e->logits + (size_t)(want[w] - i) * e->head.ldo, n_vocab * 4,
+                                     cudaMemcpyDeviceToHost, e->stream));
         LG_CHECK(cudaStreamSynchronize(e->stream));      // st_host is reused by the next upload
     }
+    if (n_want > 0) check_err(e);
 }
 
 void model_prefill(struct model *m, struct kvcache *kv, const int *tokens, int n, int pos0) {
@@ -1843,6 +1696,17 @@ void model_prefill_mixed(struct model *m, struct kvcache *kv, const float *rows,
     prefill_impl(m, kv, rows, ids, n, pos0);
 }
 void model_prefill_reserve(void) {}
+
+int lg_prefill_logits(struct model *m, struct kvcache *kv, const int *tokens, int n, int pos0, const int *want, int n_want, float *logits) {
+    if (n < 1 || n_want < 0 || !pos_in_cache(kv, pos0, n, "lg_prefill_logits")) return -1;
+    for (int i = 0; i < n_want; i++)
+        if (want[i] < 0 || want[i] >= n || (i && want[i] <= want[i - 1])) return -1;
+    for (int i = 0; i < n; i++)
+        if (tokens[i] < 0 || tokens[i] >= m->cfg.n_vocab) return -1;
+    prefill_impl(m, kv, nullptr, tokens, n, pos0, want, n_want, logits);
+    return 0;
+}
+void lg_set_compute_f32(int on) { g_compute_f32 = on != 0; }
 
 int model_forward_spec(struct model *m, struct kvcache *kv, const int *toks, int pos, int *out) {
     return spec_n(m, kv, LG_MTP_N, toks, pos, out);
@@ -1940,8 +1804,19 @@ int lg_kv_row(struct model *m, struct kvcache *kv, int layer, int pos, float *k,
     Engine *e = engine_for(m);
     if (layer < 0 || layer >= kv->n_layer || !kv->k[layer]) return 0;
     int d = kv->kv_dim[layer];
-    std::vector<__half> hk(d), hv(d);
     LG_CHECK(cudaStreamSynchronize(e->stream));
+    if (e->fam) {                                // latent rows: bf16 or f32, keys and values share them
+        const size_t es = kv_elem(kv, layer);
+        std::vector<uint8_t> row((size_t)d * es);
+        LG_CHECK(cudaMemcpy(row.data(), (const uint8_t *)kv->k[layer] + (size_t)(pos % kv->seq[layer]) * d * es, row.size(), cudaMemcpyDeviceToHost));
+        for (int i = 0; i < d; i++) {
+            if (es == 4) memcpy(&k[i], row.data() + (size_t)i * 4, 4);
+            else { uint16_t b; memcpy(&b, row.data() + (size_t)i * 2, 2); const uint32_t u = (uint32_t)b << 16; memcpy(&k[i], &u, 4); }
+            v[i] = k[i];
+        }
+        return d;
+    }
+    std::vector<__half> hk(d), hv(d);
     size_t off = (size_t)(pos % kv->seq[layer]) * d;
     LG_CHECK(cudaMemcpy(hk.data(), (__half *)kv->k[layer] + off, d * 2, cudaMemcpyDeviceToHost));
     LG_CHECK(cudaMemcpy(hv.data(), (__half *)kv->v[layer] + off, d * 2, cudaMemcpyDeviceToHost));
@@ -2074,10 +1949,14 @@ int lg_bench_matmul_pass(struct model *m, int n, int classes) {
 // and with the attention class the KV rows at the buffered positions are overwritten.
 int lg_bench_prefill_pass(struct model *m, int n, int classes) {
     Engine *e = engine_for(m);
-    if (n < 1 || n > LG_PF_MAXN || !e->kv_bound || !prefill_wide_ok(e)) return -1;
-    prefill_alloc(e);
     if (classes <= 0) classes = C_QKV | C_O | C_GATEUP | C_DOWN;
     long long before = e->launches;
+    if (e->fam) {
+        if (n < 1 || !e->kv_bound || e->fam->bench_block(e, e->kv_bound, n, 0, classes) != 0) return -1;
+        return (int)(e->launches - before);
+    }
+    if (n < 1 || n > LG_PF_MAXN || !e->kv_bound || !prefill_wide_ok(e)) return -1;
+    prefill_alloc(e);
     enqueue_prefill_block(e, e->kv_bound, n, classes);
     return (int)(e->launches - before);
 }

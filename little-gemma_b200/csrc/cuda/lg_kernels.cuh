@@ -27,50 +27,7 @@
 #include <cuda_fp16.h>
 #include <stdint.h>
 #include "lg_formats.h"
-
-#define LG_MAXM 8              // widest verify block
-#define LG_QMAX 32639.0f       // 127*256 + 127: keeps both bytes of the split in [-128,127]
-#define LG_SPIN_LIMIT (1 << 20)
-
-// error bits a kernel may raise in the engine's status word
-#define LG_ERR_MBAR_TIMEOUT 1
-
-struct LgPanel {               // quantised activations of <= 8 tokens, k = 32*nsb columns
-    int8_t *q;                 // [2][nsb][256]
-    float2 *s;                 // [2][nsb][4]   (scale, scale * sum of the group's integers)
-    int nsb;
-};
-
-// ---------------------------------------------------------------------------------------------
-// small helpers
-// ---------------------------------------------------------------------------------------------
-__device__ __forceinline__ float warp_sum(float v) {
-    #pragma unroll
-    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-    return v;
-}
-__device__ __forceinline__ float warp_max(float v) {
-    #pragma unroll
-    for (int o = 16; o > 0; o >>= 1) v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, o));
-    return v;
-}
-// Sum over the block in a fixed order (independent of anything but blockDim). `red` >= 32 floats.
-__device__ __forceinline__ float block_sum(float v, float *red) {
-    v = warp_sum(v);
-    __syncthreads();
-    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
-    __syncthreads();
-    int nw = (blockDim.x + 31) >> 5;
-    float t = (threadIdx.x < nw) ? red[threadIdx.x] : 0.0f;
-    if (threadIdx.x < 32) t = warp_sum(t);
-    if (threadIdx.x == 0) red[0] = t;
-    __syncthreads();
-    return red[0];
-}
-
-__device__ __forceinline__ float gelu_tanh(float x) {
-    return 0.5f * x * (1.0f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
-}
+#include "lg_device.cuh"
 
 // byte offset of element kk (0..31) inside one 32-byte panel column (B-fragment order)
 __device__ __forceinline__ int panel_elem(int kk) { return ((kk & 15) >> 2) * 8 + (kk >> 4) * 4 + (kk & 3); }
@@ -93,49 +50,6 @@ __device__ __forceinline__ void quant_group_store(float y, int lane, int tok, in
     if (lane == 0) P.s[((size_t)(tok >> 2) * P.nsb + sb) * 4 + (tok & 3)] = make_float2(d, d * (float)isum);
 }
 
-// Programmatic dependent launch: every kernel of a forward may be started before its predecessor
-// has finished.  pdl_launch() lets the successor begin its own prologue; pdl_wait() blocks until the
-// predecessor grid has completed and its writes are visible.  Nothing produced by an earlier kernel
-// may be read, and nothing may be written, before pdl_wait().  (No-ops for a plain launch.)
-__device__ __forceinline__ void pdl_launch() { asm volatile("griddepcontrol.launch_dependents;" ::: "memory"); }
-__device__ __forceinline__ void pdl_wait() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
-
-__device__ __forceinline__ uint32_t smem_u32(const void *p) { return (uint32_t)__cvta_generic_to_shared(p); }
-
-// ---- phase time stamps (profiling builds only: -DLG_STAMPS) ------------------------------------
-// Thread 0 of a CTA records the global nanosecond timer at named points of a kernel into
-// lg_stamps[launch tag][CTA][slot]; the host reads the array back after a forward and lays the launches of a
-// layer on one time axis (lg_debug_stamps).  Compiled out of the product build.
-#define LG_STAMP_LAUNCHES 96
-#define LG_STAMP_CTAS 320
-#define LG_STAMP_SLOTS 12
-#ifdef LG_STAMPS
-__device__ long long lg_stamps[LG_STAMP_LAUNCHES][LG_STAMP_CTAS][LG_STAMP_SLOTS];
-__device__ __forceinline__ void lg_stamp(int tag, int slot) {
-    if (threadIdx.x == 0 && tag >= 0 && tag < LG_STAMP_LAUNCHES) {
-        const int cta = blockIdx.x + gridDim.x * (blockIdx.y + gridDim.y * blockIdx.z);
-        if (cta < LG_STAMP_CTAS) {
-            long long t;
-            asm volatile("mov.u64 %0, %%globaltimer;" : "=l"(t));
-            lg_stamps[tag][cta][slot] = t;
-        }
-    }
-}
-#define LG_STAMP(tag, slot) lg_stamp(tag, slot)
-// the last slot of CTA 0 names the kernel (1 matmul store, 2 head, 3 GeGLU, 4 matmul with sums, 5 attention/ticket, 6 attention/cluster, 7 norm / residual update)
-#define LG_STAMP_KIND(tag, kind) do { if (threadIdx.x == 0 && blockIdx.x == 0 && blockIdx.y == 0 && (tag) >= 0 && (tag) < LG_STAMP_LAUNCHES) lg_stamps[tag][0][LG_STAMP_SLOTS - 1] = (kind); } while (0)
-#else
-#define LG_STAMP(tag, slot) do { } while (0)
-#define LG_STAMP_KIND(tag, kind) do { } while (0)
-#endif
-
-// streaming 16-byte weight load: read-only path, do not keep in L1
-__device__ __forceinline__ uint4 ldg_stream16(const uint4 *p) {
-    uint4 v;
-    asm("ld.global.nc.L1::no_allocate.v4.u32 {%0,%1,%2,%3}, [%4];"
-                 : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "l"(p));
-    return v;
-}
 __device__ __forceinline__ uint2 ldg_stream8(const uint2 *p) {
     uint2 v;
     asm("ld.global.nc.L1::no_allocate.v2.u32 {%0,%1}, [%2];" : "=r"(v.x), "=r"(v.y) : "l"(p));
@@ -150,57 +64,6 @@ __device__ __forceinline__ void mma_s8(int (&c)[4], uint32_t a0, uint32_t a1, ui
 }
 
 // ---- bulk (TMA, non-tensor) global -> shared copy completed on an mbarrier --------------------
-__device__ __forceinline__ void mbar_init(uint64_t *bar, int count) {
-    asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" :: "r"(smem_u32(bar)), "r"(count));
-    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
-}
-__device__ __forceinline__ void mbar_expect_tx(uint64_t *bar, uint32_t bytes) {
-    asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" :: "r"(smem_u32(bar)), "r"(bytes) : "memory");
-}
-// dst, src 16-byte aligned, bytes a multiple of 16
-__device__ __forceinline__ void bulk_g2s(void *dst, const void *src, uint32_t bytes, uint64_t *bar) {
-    asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
-                 :: "r"(smem_u32(dst)), "l"(src), "r"(bytes), "r"(smem_u32(bar)) : "memory");
-}
-// Bounded wait: returns false (and the caller raises LG_ERR_MBAR_TIMEOUT) instead of spinning forever.
-__device__ __forceinline__ bool mbar_wait(uint64_t *bar, uint32_t parity) {
-    for (int it = 0; it < LG_SPIN_LIMIT; ++it) {
-        uint32_t ok;
-        asm volatile("{\n\t.reg .pred p;\n\tmbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\n\tselp.u32 %0, 1, 0, p;\n\t}"
-                     : "=r"(ok) : "r"(smem_u32(bar)), "r"(parity) : "memory");
-        if (ok) return true;
-    }
-    return false;
-}
-
-__device__ __forceinline__ uint32_t cluster_rank() { uint32_t r; asm volatile("mov.u32 %0, %%cluster_ctarank;" : "=r"(r)); return r; }
-__device__ __forceinline__ void cluster_sync_all() {
-    asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
-}
-__device__ __forceinline__ void dsmem_store(float *local_addr, uint32_t rank, float v) {
-    uint32_t la = smem_u32(local_addr), ra;
-    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(ra) : "r"(la), "r"(rank));
-    asm volatile("st.shared::cluster.f32 [%0], %1;" :: "r"(ra), "f"(v) : "memory");
-}
-// One f32 into a peer CTA's shared memory, counted (4 bytes) on that peer's mbarrier: the receiver waits for the byte
-// count instead of a cluster-wide barrier, so threads that never join a barrier (a producer warp) are no obstacle.
-__device__ __forceinline__ void dsmem_st_async_f32(float *local_addr, uint64_t *local_bar, uint32_t rank, float v) {
-    uint32_t ra, rb;
-    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(ra) : "r"(smem_u32(local_addr)), "r"(rank));
-    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(rb) : "r"(smem_u32(local_bar)), "r"(rank));
-    asm volatile("st.async.weak.shared::cluster.mbarrier::complete_tx::bytes.f32 [%0], %1, [%2];" :: "r"(ra), "f"(v), "r"(rb) : "memory");
-}
-// Bounded wait with cluster-scope acquire: the data counted on the barrier came from peer CTAs.
-__device__ __forceinline__ bool mbar_wait_cluster(uint64_t *bar, uint32_t parity) {
-    for (int it = 0; it < LG_SPIN_LIMIT; ++it) {
-        uint32_t ok;
-        asm volatile("{\n\t.reg .pred p;\n\tmbarrier.try_wait.parity.acquire.cluster.shared::cta.b64 p, [%1], %2;\n\tselp.u32 %0, 1, 0, p;\n\t}"
-                     : "=r"(ok) : "r"(smem_u32(bar)), "r"(parity) : "memory");
-        if (ok) return true;
-    }
-    return false;
-}
-
 // Bounded-wait probe: waits on an mbarrier nobody completes, for at most `polls` polls, then reports like the kernels do.
 __global__ void lg_wait_probe_kernel(int *err, int polls) {
     __shared__ __align__(8) uint64_t bar;
@@ -488,9 +351,6 @@ enum { LG_EPI_STORE = 0, LG_EPI_HEAD = 1, LG_EPI_GEGLU = 2, LG_EPI_SUMS = 3, LG_
 #define LG_GEMV_STAGE_TILES 32         // 16x64 q4 weight tiles per stage (R row tiles x 32/R positions); i8 tiles: 16
 template <int FMT> __host__ __device__ constexpr int gemv_stage_tiles() { return FMT >= LG_FMT_I8 ? 16 : LG_GEMV_STAGE_TILES; }
 
-__device__ __forceinline__ void mbar_arrive(uint64_t *bar) {
-    asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" :: "r"(smem_u32(bar)) : "memory");
-}
 __device__ __forceinline__ void consumer_sync() {       // the consumer warps only; the producer warp never joins
     asm volatile("bar.sync 1, %0;" :: "n"(LG_GEMV_CW * 32) : "memory");
 }
@@ -1296,24 +1156,6 @@ struct LgAttnArgs {
 // keys per tile: 128, or 64 for head sizes whose K/V tiles would not fit in shared memory otherwise
 __host__ __device__ constexpr int lg_attn_tile(int hd) { return hd > 256 ? 64 : 128; }
 
-__device__ __forceinline__ void ldsm_x4(uint32_t (&r)[4], const void *p) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
-}
-__device__ __forceinline__ void ldsm_x4_t(uint32_t (&r)[4], const void *p) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
-}
-__device__ __forceinline__ void mma_f16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.f16.f16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ void cp_async16(void *dst, const void *src) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" :: "r"(smem_u32(dst)), "l"(src) : "memory");
-}
-__device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wait_all;" ::: "memory"); }
-
 // cos / sin of the NeoX rotation angles of the block's M positions, computed once per forward and
 // shared by every CTA of every layer of that kind: tab[tok][i] = (cos, sin)(pos_tok * base^(-2i/hd) / div[i]).
 __global__ void lg_rope_table_kernel(const int *pos, int M, int hd, float base, const float *div, float2 *tab) {
@@ -1715,17 +1557,6 @@ __global__ void lg_ple_build_kernel(const float *__restrict__ proj, const float 
 // ---------------------------------------------------------------------------------------------
 // greedy acceptance, position advance and hand-off to the next round -- all on the device
 // ---------------------------------------------------------------------------------------------
-struct LgRoundState {          // lives in device memory; one per session
-    int pos;                   // position of toks[0] of the round being built
-    int toks[LG_MAXM];         // toks[0] = chosen token, toks[1..] = drafts
-    int out[LG_MAXM];          // greedy successors of toks[j]
-    int adv;                   // tokens advanced by the last verify (1..M)
-    int n_emitted;             // tokens appended to the log so far
-    int n_draft, n_accept;
-    int dpos;                  // position the draft head is drafting for
-    int stop;                  // this round's remaining drafts are called off (a draft's confidence margin fell below the threshold)
-    int n_skipped;             // drafts called off so far
-};
 // After a verify of M rows: adv = 1 + run of out[j-1] == toks[j]; append toks[1..adv-1] and
 // out[adv-1] to the token log; next round starts at pos+adv with toks[0] = out[adv-1];
 // h_prev <- normed hidden of row adv-1.  (The cache needs no rollback: rows past pos+adv are

@@ -1,0 +1,693 @@
+// lg_plan.cu -- the family of models described by a layer plan (lg_plan.h): dense bf16 weights, per-layer mixers (latent
+// attention so far), f32 residual rows.  Decode and verify steps run the small-M matmuls and the split attention over the
+// latent cache; prompts run blocks of up to PLAN_BLOCK tokens through the tcgen05 matmul and the block attention.  In 32-bit
+// mode every product, activation and cache row is f32.
+#include <algorithm>
+#include "lg_engine.h"
+#include "lg_plan.h"
+#include "lg_latent.cuh"
+
+namespace lg {
+
+constexpr int PLAN_BLOCK = 2048;              // tokens of one wide block
+constexpr int PLAN_HEAD_ROWS = 128;           // logits rows made at once behind a wide block
+constexpr size_t PLAN_SMEM_MAX = 227 * 1024;          // dynamic shared memory of a CTA: all of it, and what kernels with static arrays ask for
+constexpr size_t PLAN_SMEM_SMALL = 200 * 1024;
+
+inline int up(int v, int m) { return (v + m - 1) / m * m; }
+
+// A dense matrix on the device: [rows_alloc][ldk], zero beyond its rows and columns.
+struct DMat {
+    void *w = nullptr;
+    int rows = 0, k = 0, ldk = 0, rows_alloc = 0;             // rows: a multiple of 32
+    CUtensorMap map[2];                                       // bf16: boxes of 128 and of 256 rows
+};
+
+struct PlanLayer {
+    struct lg_plan_layer p;
+    int dimp, rotp, kvp, vdp, ffp, ldc;                       // sizes padded to whole 16-element groups; ldc: cache row
+    int kv_off, rot_off, g_off;                               // columns of the input projection's row: [query latent | latent | key part | gate]
+    int owns, spec;                                           // spec: which rotation table
+    int rt;                                                   // row tiles of 16 per CTA of the decode attention (0: the row kernel)
+    DMat in, uq, ukT, ukv, uv, o, gu, down;
+    float *norm1, *norm1b, *norm2 = nullptr, *norm2b = nullptr, *q_norm, *kv_norm = nullptr, *sink;
+};
+
+// Activations of up to `cap` token rows.
+struct PlanBuf {
+    int cap = 0;
+    float *x = nullptr, *pj = nullptr, *o = nullptr, *gu = nullptr;
+    void *h = nullptr, *cq = nullptr, *q = nullptr, *qa = nullptr, *ol = nullptr, *at = nullptr, *act = nullptr;
+    std::vector<float2 *> tab;
+    int *toks = nullptr, *pos = nullptr;                      // of the block (narrow: the engine's round state)
+};
+
+struct PlanModel {
+    struct lg_plan *plan = nullptr;
+    std::vector<PlanLayer> L;
+    DMat embed;
+    float *out_norm = nullptr;
+    struct Rot { float base; int dims; double *freq; };
+    std::vector<Rot> rot;
+    PlanBuf nb, wb;
+    bool wide_ok = false;
+    // bound to a cache
+    int max_seq = 0, seq_alloc = 0, C = 1;
+    float *part = nullptr; float2 *part_ml = nullptr;
+    bf16 *ex = nullptr;
+    int *want = nullptr; void *hg = nullptr; float *wlog = nullptr;
+    float *logits = nullptr;                                  // 32-bit: rows of a head without F_LOGITS
+    std::map<std::pair<const void *, long long>, CUtensorMap> maps;
+};
+
+// ------------------------------------------------------------------------------------------
+// loading
+// ------------------------------------------------------------------------------------------
+const struct gguf_tensor *need(Engine *e, int L, const char *leaf, int rows, int cols) {
+    char name[96];
+    snprintf(name, sizeof name, "%s.weight", leaf);
+    const struct gguf_tensor *t = find_t(e->ctx, L, name);
+    if (!t) { fprintf(stderr, "lg_b200: layer %d: tensor %s is missing from the model\n", L, leaf); exit(1); }
+    if ((int)t->dims[0] != (cols ? cols : rows) || (int)t->dims[1] != (cols ? rows : 1)) {
+        fprintf(stderr, "lg_b200: %s is %d x %d, expected %d x %d\n", t->name, (int)t->dims[1], (int)t->dims[0], cols ? rows : 1, cols ? cols : rows);
+        exit(1);
+    }
+    if (t->type != GGML_TYPE_BF16 && t->type != GGML_TYPE_F32 && t->type != GGML_TYPE_F16) {
+        fprintf(stderr, "lg_b200: %s: layer-plan models have dense weights (bf16, f16, f32), not ggml type %u\n", t->name, t->type);
+        exit(1);
+    }
+    return t;
+}
+std::vector<float> row_f32(const struct gguf_tensor *t, int row) {
+    const size_t n = (size_t)t->dims[0];
+    std::vector<float> f(n);
+    dequantize_into(t->type, (const uint8_t *)t->data + (size_t)row * n * (t->type == GGML_TYPE_F32 ? 4 : 2), f.data(), (int64_t)n);
+    return f;
+}
+float *vec(Engine *e, int L, const char *leaf, int n) { return upload_f32(row_f32(need(e, L, leaf, n, 0), 0).data(), (size_t)n); }
+
+uint16_t bf16_bits(float f) {
+    uint32_t u;
+    memcpy(&u, &f, 4);
+    return (uint16_t)((u + 0x7fff + ((u >> 16) & 1)) >> 16);
+}
+
+// A matrix under construction on the host, in the element type of the engine's mode.
+struct MatBuild {
+    bool f32; int rows, k, ldk;
+    std::vector<uint8_t> buf;
+    MatBuild(Engine *e, int rows_, int k_) : f32(e->f32), rows(up(rows_, 32)), k(k_), ldk(up(k_, 64)) { buf.assign((size_t)rows * ldk * (f32 ? 4 : 2), 0); }
+    void put(size_t i, float v) {
+        if (f32) memcpy(&buf[i * 4], &v, 4);
+        else { const uint16_t b = bf16_bits(v); memcpy(&buf[i * 2], &b, 2); }
+    }
+    // row `src` of t; its columns come in segments of seg that start every seg_to columns here (0: one piece)
+    void row(int dst, const struct gguf_tensor *t, int src, int seg = 0, int seg_to = 0) {
+        const int n = (int)t->dims[0];
+        if (!f32 && t->type == GGML_TYPE_BF16 && seg == seg_to) {
+            memcpy(&buf[(size_t)dst * ldk * 2], (const uint8_t *)t->data + (size_t)src * n * 2, (size_t)n * 2);
+            return;
+        }
+        const std::vector<float> f = row_f32(t, src);
+        for (int i = 0; i < n; i++) put((size_t)dst * ldk + (seg ? i / seg * seg_to + i % seg : i), f[i]);
+    }
+    DMat upload(Engine *e) {
+        DMat m;
+        m.rows = rows; m.k = k; m.ldk = ldk; m.rows_alloc = up(rows, 256);
+        const size_t es = f32 ? 4 : 2;
+        m.w = dalloc<uint8_t>((size_t)m.rows_alloc * ldk * es);
+        h2d_sync(m.w, buf.data(), buf.size());
+        e->weight_bytes += (size_t)rows * k * es;
+        if (!f32)
+            for (int i = 0; i < 2; i++) m.map[i] = tiled_map(m.w, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, ldk, m.rows_alloc, (long long)ldk * 2, DN_GEMM_BK, 128 << i);
+        return m;
+    }
+};
+
+// `groups` groups of `rows` rows of t, each padded to `to` rows; rows of group g start at g * t_stride
+void put_groups(MatBuild &b, int dst0, const struct gguf_tensor *t, int groups, int rows, int to) {
+    for (int g = 0; g < groups; g++)
+        for (int r = 0; r < rows; r++) b.row(dst0 + g * to + r, t, g * rows + r);
+}
+
+template <typename K> void smem_attr(K kernel, size_t bytes = PLAN_SMEM_MAX) { LG_CHECK(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes)); }
+template <int EPI, bool RMSX> void gemv_attrs() {
+    smem_attr(lg_dn_gemv_kernel<EPI, 1, RMSX>, PLAN_SMEM_SMALL); smem_attr(lg_dn_gemv_kernel<EPI, 2, RMSX>, PLAN_SMEM_SMALL);
+    smem_attr(lg_dn_gemv_kernel<EPI, 4, RMSX>, PLAN_SMEM_SMALL); smem_attr(lg_dn_gemv_kernel<EPI, 8, RMSX>, PLAN_SMEM_SMALL);
+}
+void plan_attributes() {
+    static bool done[64] = {false};
+    int dev = 0;
+    LG_CHECK(cudaGetDevice(&dev));
+    if (dev < 0 || dev >= 64 || done[dev]) return;
+    done[dev] = true;
+    gemv_attrs<DN_STORE, true>();
+    smem_attr(lg_dn_gemm_kernel<128, DN_G_F32>, dn_gemm_smem<128>()); smem_attr(lg_dn_gemm_kernel<256, DN_G_F32>, dn_gemm_smem<256>());
+    smem_attr(lg_dn_gemm_kernel<128, DN_G_BF16>, dn_gemm_smem<128>()); smem_attr(lg_dn_gemm_kernel<256, DN_G_BF16>, dn_gemm_smem<256>());
+    smem_attr(lg_dn_gemm_kernel<128, DN_G_GLU>, dn_gemm_smem<128>()); smem_attr(lg_dn_gemm_kernel<256, DN_G_GLU>, dn_gemm_smem<256>());
+    smem_attr(lg_latent_dec_attn_kernel<1, 2>); smem_attr(lg_latent_dec_attn_kernel<1, 4>); smem_attr(lg_latent_dec_attn_kernel<1, 8>);
+    smem_attr(lg_latent_dec_attn_kernel<2, 2>); smem_attr(lg_latent_dec_attn_kernel<2, 4>); smem_attr(lg_latent_dec_attn_kernel<2, 8>);
+    smem_attr(lg_latent_pf_attn_kernel<8>); smem_attr(lg_latent_pf_attn_kernel<16>); smem_attr(lg_latent_pf_attn_kernel<32>);
+    smem_attr(lg_latent_merge_kernel, PLAN_SMEM_SMALL); smem_attr(lg_latent_attn_rows_kernel<float>, PLAN_SMEM_SMALL); smem_attr(lg_latent_attn_rows_kernel<bf16>, PLAN_SMEM_SMALL);
+}
+
+void buf_alloc(Engine *e, PlanBuf &b, int cap, bool narrow) {
+    PlanModel *pm = e->plan;
+    const size_t es = e->f32 ? 4 : 2;
+    size_t pj = 0, o = up(pm->plan->width, 32), gu = 0, cq = 0, q = 0, qa = 0, ol = 0, at = 0, act = 0;
+    for (auto &l : pm->L) {
+        const size_t H = l.p.heads;
+        pj = std::max(pj, (size_t)l.in.rows); cq = std::max(cq, (size_t)l.uq.ldk);
+        q = std::max(q, (size_t)up((int)H * (l.dimp + l.rotp), 32));
+        qa = std::max(qa, H * l.ldc); ol = std::max(ol, H * l.kvp); at = std::max(at, (size_t)l.o.ldk);
+        if (l.p.ff) { act = std::max(act, (size_t)l.down.ldk); gu = std::max(gu, (size_t)l.gu.rows); }
+    }
+    auto elems = [&](size_t per) { return (void *)dalloc<uint8_t>(((size_t)cap * per + 256) * es); };
+    b.cap = cap;
+    b.x = narrow ? e->x : dalloc<float>((size_t)cap * pm->plan->width);
+    b.pj = dalloc<float>(cap * pj); b.o = dalloc<float>(cap * o);
+    if (e->f32) b.gu = dalloc<float>(cap * gu + 16);
+    b.h = elems(up(pm->plan->width, 64)); b.cq = elems(cq); b.q = elems(q); b.at = elems(at); b.act = elems(act + 64);
+    if (narrow || e->f32) { b.qa = elems(qa); b.ol = elems(ol); }
+    for (auto &r : pm->rot) b.tab.push_back(dalloc<float2>((size_t)cap * (r.dims / 2) + 1));
+    if (!narrow) { b.toks = nullptr; b.pos = dalloc<int>(1); }
+}
+void buf_free(PlanBuf &b, bool narrow) {
+    if (!narrow) cudaFree(b.x);
+    cudaFree(b.pj); cudaFree(b.o); cudaFree(b.gu); cudaFree(b.h); cudaFree(b.cq); cudaFree(b.q); cudaFree(b.qa); cudaFree(b.ol); cudaFree(b.at); cudaFree(b.act);
+    for (auto t : b.tab) cudaFree(t);
+    cudaFree(b.toks); cudaFree(b.pos);
+    b = PlanBuf();
+}
+
+void layer_sizes(PlanLayer &l) {
+    const struct lg_plan_layer &p = l.p;
+    l.dimp = up(p.dim, 16); l.rotp = up(p.rot_dim, 16); l.kvp = up(p.kv_rank, 16); l.vdp = up(p.vdim, 16); l.ffp = up(p.ff, 16);
+    l.ldc = l.kvp + l.rotp;
+}
+
+void plan_load(Engine *e) {
+    PlanModel *pm = e->plan = new PlanModel();
+    plan_attributes();
+    pm->plan = lg_plan_read(e->ctx);
+    if (!pm->plan) exit(1);
+    const struct lg_plan *P = pm->plan;
+    const int W = P->width;
+    if (W > 16 * 1024) { fprintf(stderr, "lg_b200: rows of %d elements exceed the norm kernel's 16384\n", W); exit(1); }
+    pm->L.resize(P->n_layer);
+    pm->wide_ok = true;
+    for (int i = 0; i < P->n_layer; i++) {
+        PlanLayer &l = pm->L[i];
+        l.p = P->layer[i];
+        layer_sizes(l);
+        const struct lg_plan_layer &p = l.p;
+        const int H = p.heads;
+        l.owns = p.kv_src == i;
+        l.kv_off = up(p.q_rank, 16);
+        l.rot_off = l.kv_off + (l.owns ? l.kvp : 0);
+        l.g_off = l.rot_off + (l.owns ? l.rotp : 0);
+        {   // everything that reads the layer's input: query latent, cached latent and key part, output gate
+            MatBuild b(e, l.g_off + H * l.vdp, W);
+            put_groups(b, 0, need(e, i, "attn_q_a", p.q_rank, W), 1, p.q_rank, 0);
+            if (l.owns) {
+                const struct gguf_tensor *t = need(e, i, "attn_kv_a", p.kv_rank + p.rot_dim, W);
+                for (int r = 0; r < p.kv_rank + p.rot_dim; r++) b.row(r < p.kv_rank ? l.kv_off + r : l.rot_off + r - p.kv_rank, t, r);
+            }
+            put_groups(b, l.g_off, need(e, i, "attn_gate", H * p.vdim, W), H, p.vdim, l.vdp);
+            l.in = b.upload(e);
+        }
+        {   // queries: per head [unrotated | rotated]
+            const struct gguf_tensor *t = need(e, i, "attn_q_b", H * (p.dim + p.rot_dim), p.q_rank);
+            MatBuild b(e, H * (l.dimp + l.rotp), p.q_rank);
+            for (int h = 0; h < H; h++)
+                for (int r = 0; r < p.dim + p.rot_dim; r++)
+                    b.row(h * (l.dimp + l.rotp) + (r < p.dim ? r : l.dimp + r - p.dim), t, h * (p.dim + p.rot_dim) + r);
+            l.uq = b.upload(e);
+        }
+        const struct gguf_tensor *uk = need(e, i, "attn_k_b", H * p.dim, p.kv_rank), *uv = need(e, i, "attn_v_b", H * p.vdim, p.kv_rank);
+        {   // the key expansion transposed per head: rows = latent columns, contraction over the head's dimensions
+            MatBuild b(e, H * l.kvp, p.dim);
+            for (int h = 0; h < H; h++)
+                for (int d = 0; d < p.dim; d++) {
+                    const std::vector<float> f = row_f32(uk, h * p.dim + d);
+                    for (int r = 0; r < p.kv_rank; r++) b.put((size_t)(h * l.kvp + r) * b.ldk + d, f[r]);
+                }
+            l.ukT = b.upload(e);
+        }
+        {
+            MatBuild b(e, H * l.vdp, p.kv_rank);
+            put_groups(b, 0, uv, H, p.vdim, l.vdp);
+            l.uv = b.upload(e);
+        }
+        if (!e->f32) {   // both expansions, for the prompt pass
+            MatBuild b(e, H * (l.dimp + l.vdp), p.kv_rank);
+            put_groups(b, 0, uk, H, p.dim, l.dimp);
+            put_groups(b, H * l.dimp, uv, H, p.vdim, l.vdp);
+            const size_t before = e->weight_bytes;
+            l.ukv = b.upload(e);
+            e->weight_bytes = before;                        // a second copy of weights already counted
+        }
+        {
+            const struct gguf_tensor *t = need(e, i, "attn_output", W, H * p.vdim);
+            MatBuild b(e, W, H * l.vdp);
+            for (int r = 0; r < W; r++) b.row(r, t, r, p.vdim, l.vdp);
+            l.o = b.upload(e);
+        }
+        if (p.ff) {
+            const struct gguf_tensor *g = need(e, i, "ffn_gate", p.ff, W), *u = need(e, i, "ffn_up", p.ff, W), *d = need(e, i, "ffn_down", W, p.ff);
+            MatBuild b(e, 2 * l.ffp, W);
+            for (int r = 0; r < p.ff; r++) { b.row(r / 8 * 16 + r % 8, g, r); b.row(r / 8 * 16 + 8 + r % 8, u, r); }   // 8 gate rows, their 8 up rows
+            l.gu = b.upload(e);
+            MatBuild c(e, W, l.ffp);
+            for (int r = 0; r < W; r++) c.row(r, d, r);
+            l.down = c.upload(e);
+            l.norm2 = vec(e, i, "ffn_norm", W); l.norm2b = vec(e, i, "post_ffw_norm", W);
+        }
+        l.norm1 = vec(e, i, "attn_norm", W); l.norm1b = vec(e, i, "post_attention_norm", W);
+        l.q_norm = vec(e, i, "attn_q_a_norm", p.q_rank);
+        if (l.owns) l.kv_norm = vec(e, i, "attn_kv_a_norm", p.kv_rank);
+        l.sink = vec(e, i, "attn_sinks", H);
+        l.spec = -1;
+        for (size_t s = 0; s < pm->rot.size(); s++) if (pm->rot[s].base == p.rot_base && pm->rot[s].dims == p.rot_dims) l.spec = (int)s;
+        if (l.spec < 0) {
+            std::vector<double> f(p.rot_dims / 2 + 1);
+            for (int j = 0; j < p.rot_dims / 2; j++) f[j] = pow((double)p.rot_base, -2.0 * j / p.rot_dims);
+            double *d = dalloc<double>(f.size());
+            h2d_sync(d, f.data(), f.size() * 8);
+            l.spec = (int)pm->rot.size();
+            pm->rot.push_back({p.rot_base, p.rot_dims, d});
+        }
+        l.rt = l.kvp > 512 ? 0 : lg_latent_dec_smem(2, l.ldc) <= PLAN_SMEM_MAX ? 2 : lg_latent_dec_smem(1, l.ldc) <= PLAN_SMEM_MAX ? 1 : 0;
+        if (e->f32) l.rt = 0;
+        if (l.vdp > 256 || lg_latent_pf_smem(l.dimp + l.rotp, l.vdp) > PLAN_SMEM_MAX) pm->wide_ok = false;
+        if ((size_t)(l.ldc + l.kvp + 128) * 4 > PLAN_SMEM_SMALL || (size_t)LG_LM_GROUPS * l.kvp * 4 > PLAN_SMEM_SMALL ||
+            (size_t)LG_MAXM * (l.uq.ldk + 8) * 2 > PLAN_SMEM_SMALL) { fprintf(stderr, "lg_b200: layer %d: latent sizes beyond what the kernels hold\n", i); exit(1); }
+    }
+    if (e->f32) pm->wide_ok = true;
+    static const int wide = env_int("LG_PREFILL_WIDE", 1);
+    if (!wide) pm->wide_ok = false;
+    {
+        const struct gguf_tensor *t = need(e, -1, "token_embd", P->vocab, W);
+        MatBuild b(e, P->vocab, W);
+        for (int r = 0; r < P->vocab; r++) b.row(r, t, r);
+        pm->embed = b.upload(e);
+    }
+    e->head.ldo = pm->embed.rows;
+    pm->out_norm = vec(e, -1, "output_norm", W);
+    buf_alloc(e, pm->nb, LG_MAXM, true);
+    if (e->f32) pm->logits = dalloc<float>((size_t)LG_MAXM * e->head.ldo);
+}
+
+void dmat_free(DMat &m) { cudaFree(m.w); m = DMat(); }
+void plan_unbind(PlanModel *pm) {
+    cudaFree(pm->part); cudaFree(pm->part_ml); cudaFree(pm->ex); cudaFree(pm->want); cudaFree(pm->hg); cudaFree(pm->wlog);
+    pm->part = nullptr; pm->part_ml = nullptr; pm->ex = nullptr; pm->want = nullptr; pm->hg = nullptr; pm->wlog = nullptr;
+    if (pm->wb.cap) buf_free(pm->wb, false);
+    pm->maps.clear();
+}
+void plan_release(Engine *e) {
+    PlanModel *pm = e->plan;
+    if (!pm) return;
+    plan_unbind(pm);
+    for (auto &l : pm->L) {
+        for (DMat *m : {&l.in, &l.uq, &l.ukT, &l.ukv, &l.uv, &l.o, &l.gu, &l.down}) dmat_free(*m);
+        for (float *v : {l.norm1, l.norm1b, l.norm2, l.norm2b, l.q_norm, l.kv_norm, l.sink}) cudaFree(v);
+    }
+    for (auto &r : pm->rot) cudaFree(r.freq);
+    dmat_free(pm->embed);
+    cudaFree(pm->out_norm); cudaFree(pm->logits);
+    buf_free(pm->nb, true);
+    lg_plan_free(pm->plan);
+    delete pm;
+    e->plan = nullptr;
+}
+
+// ------------------------------------------------------------------------------------------
+// cache
+// ------------------------------------------------------------------------------------------
+int cache_rows(int max_seq) { return up(max_seq, 128); }      // whole boxes of the tiled copies
+
+int plan_kv_init(struct kvcache *kv, const struct model *m, bool f32) {
+    struct lg_plan *P = lg_plan_read(m->ctx);
+    if (!P) return -1;
+    for (int i = 0; i < P->n_layer; i++) {
+        PlanLayer l;
+        l.p = P->layer[i];
+        layer_sizes(l);
+        kv->kv_dim[i] = l.ldc;
+        kv->f16[i] = f32 ? 0 : 2;
+        if (l.p.kv_src != i) continue;                        // borrows the rows of an earlier layer
+        kv->seq[i] = kv->max_seq;
+        const size_t bytes = (size_t)cache_rows(kv->max_seq) * l.ldc * (f32 ? 4 : 2);
+        LG_CHECK(cudaMalloc(&kv->k[i], bytes));
+        LG_CHECK(cudaMemset(kv->k[i], 0, bytes));
+    }
+    lg_plan_free(P);
+    return 0;
+}
+
+void plan_bind(Engine *e, const struct kvcache *kv) {
+    PlanModel *pm = e->plan;
+    plan_unbind(pm);
+    pm->max_seq = kv->max_seq; pm->seq_alloc = cache_rows(kv->max_seq);
+    if (e->f32) return;
+    // Splits of the decode attention: as many CTAs as there are SMs for the row groups of one token, a property of the cache
+    // length and the head counts alone (never of the block's width or the position).
+    int groups = 1;
+    size_t rows = 0;
+    for (auto &l : pm->L) {
+        if (l.rt) groups = std::max(groups, (l.p.heads + 16 * l.rt - 1) / (16 * l.rt));
+        rows = std::max(rows, (size_t)l.p.heads * LG_MAXM * l.kvp);
+    }
+    pm->C = std::max(1, std::min({e->sm_count / groups, (kv->max_seq + LG_LD_S - 1) / LG_LD_S, LG_LM_MAXC}));
+    size_t heads = 0;
+    for (auto &l : pm->L) heads = std::max(heads, (size_t)l.p.heads);
+    pm->part = dalloc<float>(rows * pm->C);
+    pm->part_ml = dalloc<float2>(heads * LG_MAXM * pm->C);
+}
+
+// ------------------------------------------------------------------------------------------
+// matmul launches
+// ------------------------------------------------------------------------------------------
+// Slices of k per 16-row tile: enough warps to keep every SM's loads in flight, at least two chunks of 32 columns each.  A
+// property of the matrix alone: it fixes the order in which a row's products are added.
+int gemv_ks(const Engine *e, const DMat &W) {
+    const int tiles = W.rows / 16, nchunk = W.ldk / 32;
+    int ks = 1;
+    while (ks < 8 && tiles * ks < e->sm_count * 16 && nchunk / (ks * 2) >= 2) ks *= 2;
+    return ks;
+}
+template <int EPI, bool RMSX>
+int launch_dn_gemv(Engine *e, const DMat &W, LgDnGemvArgs a, int cap_ctas = 1 << 20) {
+    a.w = (const bf16 *)W.w; a.ldk = W.ldk; a.n_tiles = W.rows / 16;
+    const int ks = gemv_ks(e, W), tpc = 8 / ks;
+    a.n_main = std::min((a.n_tiles + tpc - 1) / tpc, cap_ctas);
+    const dim3 grid(a.n_main + (a.job ? a.M : 0));
+    const size_t sm = RMSX ? (size_t)a.M * (W.ldk + 8) * 2 : 0;
+    switch (ks) {
+    case 1: launch_k(e, lg_dn_gemv_kernel<EPI, 1, RMSX>, grid, dim3(DN_GEMV_THREADS), sm, a); break;
+    case 2: launch_k(e, lg_dn_gemv_kernel<EPI, 2, RMSX>, grid, dim3(DN_GEMV_THREADS), sm, a); break;
+    case 4: launch_k(e, lg_dn_gemv_kernel<EPI, 4, RMSX>, grid, dim3(DN_GEMV_THREADS), sm, a); break;
+    default: launch_k(e, lg_dn_gemv_kernel<EPI, 8, RMSX>, grid, dim3(DN_GEMV_THREADS), sm, a); break;
+    }
+    return a.n_main;
+}
+// x: [x_rows][ldx] bf16, of which n rows count
+template <int EPI>
+void launch_dn_gemm(Engine *e, const DMat &W, const void *x, int ldx, int x_rows, int n, void *out, int ldo) {
+    PlanModel *pm = e->plan;
+    const auto key = std::make_pair(x, (long long)ldx << 32 | W.k);
+    auto it = pm->maps.find(key);
+    if (it == pm->maps.end())
+        it = pm->maps.emplace(key, tiled_map(x, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, std::min(W.k, ldx), x_rows, (long long)ldx * 2, DN_GEMM_BK, DN_GEMM_BM)).first;
+    LgDnGemmArgs a{};
+    a.nkb = W.ldk / DN_GEMM_BK; a.n_tok = n; a.cols = W.rows; a.out = out; a.ldo = ldo; a.err = e->err;
+    const int ty = (n + DN_GEMM_BM - 1) / DN_GEMM_BM;
+    if ((W.rows + 255) / 256 * ty >= e->sm_count)
+        launch_k(e, lg_dn_gemm_kernel<256, EPI>, dim3((W.rows + 255) / 256, ty), dim3(DN_GEMM_THREADS), dn_gemm_smem<256>(), it->second, W.map[1], a);
+    else
+        launch_k(e, lg_dn_gemm_kernel<128, EPI>, dim3((W.rows + 127) / 128, ty), dim3(DN_GEMM_THREADS), dn_gemm_smem<128>(), it->second, W.map[0], a);
+}
+void launch_f32(Engine *e, const DMat &W, const void *x, int ldx, int n, void *out, int ldo, int groups = 1, int group_rows = 0, int x_group = 0, int out_group = 0) {
+    LgDnF32Args a{};
+    a.w = (const float *)W.w; a.ldk = W.ldk; a.rows = groups > 1 ? group_rows : W.rows; a.k = W.k;
+    if (groups == 1 && group_rows) a.rows = group_rows;
+    a.x = (const float *)x; a.ldx = ldx; a.n = n; a.out = (float *)out; a.ldo = ldo;
+    a.w_group = (size_t)group_rows * W.ldk; a.x_group = x_group; a.out_group = out_group;
+    launch_k(e, lg_dn_gemm_f32_kernel, dim3((a.rows + 63) / 64, (n + 63) / 64, groups), dim3(256), 0, a);
+}
+
+void launch_row_norm(Engine *e, int n, LgRowNormArgs a) {
+    // few rows: as many threads as the row has elements, for latency; many rows: fewer threads per row, for throughput
+    const int threads = std::min(1024, std::max(128, up(n > 16 ? a.n / 8 : a.n, 32)));
+    const int ept = (a.n + threads - 1) / threads;
+    auto go = [&](auto kernel) { launch_k(e, kernel, dim3(n), dim3(threads), 0, a); };
+    if (e->f32) {
+        if (ept <= 4) go(lg_row_norm_kernel<float, 4>); else if (ept <= 8) go(lg_row_norm_kernel<float, 8>); else go(lg_row_norm_kernel<float, 16>);
+    } else {
+        if (ept <= 4) go(lg_row_norm_kernel<bf16, 4>); else if (ept <= 8) go(lg_row_norm_kernel<bf16, 8>); else go(lg_row_norm_kernel<bf16, 16>);
+    }
+}
+
+// ------------------------------------------------------------------------------------------
+// a pass over the layers
+// ------------------------------------------------------------------------------------------
+struct Pass {
+    PlanBuf *b;
+    int n; bool wide;
+    const int *toks, *pos;                        // device
+    int pos0;                                     // wide: the host's copy of *pos
+};
+
+void plan_embed_rows(Engine *e, const int *toks, int n, float *x) {
+    const DMat &E = e->plan->embed;
+    const int W = e->plan->plan->width;
+    if (e->f32) launch_k(e, lg_dn_embed_rows<float>, dim3(n), dim3(256), 0, (const float *)E.w, E.ldk, e->plan->plan->vocab, toks, x, W);
+    else launch_k(e, lg_dn_embed_rows<bf16>, dim3(n), dim3(256), 0, (const bf16 *)E.w, E.ldk, e->plan->plan->vocab, toks, x, W);
+}
+
+void latent_attention(Engine *e, const struct kvcache *kv, PlanLayer &l, const Pass &p, int only) {
+    PlanModel *pm = e->plan;
+    PlanBuf &b = *p.b;
+    const int H = l.p.heads, n = p.n, qh = l.dimp + l.rotp, ldq = up(H * qh, 32), ld_at = l.o.ldk;
+    const float eps = pm->plan->norm_eps;
+    void *cache = kv->k[l.p.kv_src];
+    const float *gate = b.pj + l.g_off;
+    LgCacheRow cr{};
+    cr.src = b.pj; cr.ld = l.in.rows; cr.kv_off = l.kv_off; cr.rot_off = l.rot_off; cr.norm_w = l.kv_norm; cr.eps = eps;
+    cr.kv_rank = l.p.kv_rank; cr.rot_dim = l.p.rot_dim; cr.rot_dims = l.p.rot_dims; cr.tab = b.tab[l.spec];
+    cr.cache = cache; cr.ldc = l.ldc; cr.rot_at = l.kvp; cr.pos = p.pos;
+    LgRotQ rq{};
+    rq.q = b.q; rq.ldq = ldq; rq.head_stride = qh; rq.rot_at_q = l.dimp; rq.out = b.qa; rq.ldc = l.ldc; rq.rot_at = l.kvp;
+    rq.H = H; rq.rot_dim = l.p.rot_dim; rq.rot_dims = l.p.rot_dims; rq.tab = b.tab[l.spec];
+    LgLatentPrepArgs pa{};
+    pa.src = b.pj; pa.ld = l.in.rows; pa.q_off = 0; pa.q_rank = l.p.q_rank; pa.q_norm = l.q_norm; pa.eps = eps;
+    pa.cq = b.cq; pa.ldcq = l.uq.ldk; pa.owns = l.owns; pa.cr = cr;
+    LgLatentRowsArgs ra{};
+    ra.q = b.qa; ra.cache = cache; ra.ldc = l.ldc; ra.kvp = l.kvp; ra.H = H; ra.sink = l.sink; ra.scale = l.p.scale; ra.pos = p.pos; ra.out = b.ol;
+    const size_t rows_sm = (size_t)(l.ldc + l.kvp + 128) * 4;
+
+    if (e->f32) {
+        launch_k(e, lg_latent_prep_kernel<float>, dim3(n), dim3(128), 0, pa);
+        launch_f32(e, l.uq, b.cq, l.uq.ldk, n, b.q, ldq);
+        launch_f32(e, l.ukT, b.q, ldq, n, b.qa, H * l.ldc, H, l.kvp, qh, l.ldc);
+        launch_k(e, lg_latent_rot_q_kernel<float>, dim3(1, n), dim3(128), 0, rq);
+        launch_k(e, lg_latent_attn_rows_kernel<float>, dim3(H, n), dim3(128), rows_sm, ra);
+        launch_f32(e, l.uv, b.ol, H * l.kvp, n, b.at, ld_at, H, l.vdp, l.kvp, l.vdp);
+        launch_k(e, lg_dn_gate_rows, dim3((H * l.vdp + 255) / 256, n), dim3(256), 0, (float *)b.at, ld_at, gate, l.in.rows, H * l.vdp);
+        return;
+    }
+    if (p.wide) {
+        const int keys = p.pos0 + n, ldx = up(H * (l.dimp + l.vdp), 32);
+        if (only & C_MISC) launch_k(e, lg_latent_prep_kernel<bf16>, dim3(n), dim3(128), 0, pa);
+        if (only & C_QKV) launch_dn_gemm<DN_G_BF16>(e, l.uq, b.cq, l.uq.ldk, b.cap, n, b.q, ldq);
+        if (only & C_PLE) launch_dn_gemm<DN_G_BF16>(e, l.ukv, cache, l.ldc, pm->seq_alloc, keys, pm->ex, ldx);
+        if (!(only & C_ATTN)) return;
+        LgLatentPfArgs a{};
+        a.q = (const bf16 *)b.q; a.ldq = ldq; a.ex = pm->ex; a.ldx = ldx; a.cache = (const bf16 *)cache; a.ldc = l.ldc; a.rot_at = l.kvp;
+        a.H = H; a.dimp = l.dimp; a.rotp = l.rotp; a.rot_dims = l.p.rot_dims; a.vdp = l.vdp; a.n = n;
+        a.tab = b.tab[l.spec]; a.sink = l.sink; a.scale = l.p.scale; a.gate = gate; a.ldg = l.in.rows; a.pos = p.pos;
+        a.out = (bf16 *)b.at; a.ldo = ld_at;
+        const dim3 grid((n + LG_LP_Q - 1) / LG_LP_Q, H), block(LG_LP_THREADS);
+        const size_t sm = lg_latent_pf_smem(qh, l.vdp);
+        if (l.vdp <= 64) launch_k(e, lg_latent_pf_attn_kernel<8>, grid, block, sm, a);
+        else if (l.vdp <= 128) launch_k(e, lg_latent_pf_attn_kernel<16>, grid, block, sm, a);
+        else launch_k(e, lg_latent_pf_attn_kernel<32>, grid, block, sm, a);
+        return;
+    }
+    if (only & C_QKV) {
+        LgDnGemvArgs q{};                          // normed query latent -> queries; beside it, the cache rows
+        q.xf = b.pj; q.ldxf = l.in.rows; q.kx = l.p.q_rank; q.rms_w = l.q_norm; q.eps = eps; q.M = n; q.outh = (bf16 *)b.q; q.ldoh = ldq;
+        if (l.owns) { q.job = DN_JOB_CACHE_ROW; q.cr = cr; }
+        launch_dn_gemv<DN_STORE, true>(e, l.uq, q);
+        LgDnGemvArgs k{};                          // per head onto the latent; beside it, the rotated parts
+        k.x = (const bf16 *)b.q; k.ldx = ldq; k.tiles_per_group = l.kvp / 16; k.x_group = qh; k.out_group = l.ldc; k.M = n;
+        k.outh = (bf16 *)b.qa; k.ldoh = H * l.ldc; k.job = DN_JOB_ROT_Q; k.rq = rq;
+        launch_dn_gemv<DN_STORE, false>(e, l.ukT, k);
+    }
+    if (only & C_ATTN) {
+        if (!l.rt) launch_k(e, lg_latent_attn_rows_kernel<bf16>, dim3(H, n), dim3(128), rows_sm, ra);
+        else {
+            LgLatentDecArgs a{};
+            a.q = (const bf16 *)b.qa; a.cache = (const bf16 *)cache; a.ldc = l.ldc; a.kvp = l.kvp; a.rows = n * H; a.H = H;
+            a.scale = l.p.scale; a.pos = p.pos; a.part = pm->part; a.part_ml = pm->part_ml;
+            const int rt = n * H > 16 ? l.rt : 1;
+            const dim3 grid(pm->C, (n * H + 16 * rt - 1) / (16 * rt)), block(LG_LD_THREADS);
+            const size_t sm = lg_latent_dec_smem(rt, l.ldc);
+            if (rt == 2) {
+                if (l.kvp <= 128) launch_k(e, lg_latent_dec_attn_kernel<2, 2>, grid, block, sm, a);
+                else if (l.kvp <= 256) launch_k(e, lg_latent_dec_attn_kernel<2, 4>, grid, block, sm, a);
+                else launch_k(e, lg_latent_dec_attn_kernel<2, 8>, grid, block, sm, a);
+            } else {
+                if (l.kvp <= 128) launch_k(e, lg_latent_dec_attn_kernel<1, 2>, grid, block, sm, a);
+                else if (l.kvp <= 256) launch_k(e, lg_latent_dec_attn_kernel<1, 4>, grid, block, sm, a);
+                else launch_k(e, lg_latent_dec_attn_kernel<1, 8>, grid, block, sm, a);
+            }
+            LgLatentMergeArgs m{};
+            m.part = pm->part; m.part_ml = pm->part_ml; m.rows = n * H; m.H = H; m.kvp = l.kvp; m.C = pm->C; m.sink = l.sink; m.pos = p.pos; m.out = (bf16 *)b.ol;
+            launch_k(e, lg_latent_merge_kernel, dim3(n * H), dim3(LG_LM_THREADS), (size_t)LG_LM_GROUPS * l.kvp * 4, m);
+        }
+    }
+    if (only & C_O) {
+        LgDnGemvArgs v{};                          // latent outputs -> gated head values
+        v.x = (const bf16 *)b.ol; v.ldx = H * l.kvp; v.tiles_per_group = l.vdp / 16; v.x_group = l.kvp; v.out_group = l.vdp; v.M = n;
+        v.outh = (bf16 *)b.at; v.ldoh = ld_at; v.gate = gate; v.ld_gate = l.in.rows;
+        launch_dn_gemv<DN_SIGMOID_GATE, false>(e, l.uv, v);
+    }
+}
+
+// out (f32 rows) = W x
+void project(Engine *e, const DMat &W, const void *x, int ldx, const Pass &p, float *out) {
+    if (e->f32) launch_f32(e, W, x, ldx, p.n, out, W.rows);
+    else if (p.wide) launch_dn_gemm<DN_G_F32>(e, W, x, ldx, p.b->cap, p.n, out, W.rows);
+    else {
+        LgDnGemvArgs a{};
+        a.x = (const bf16 *)x; a.ldx = ldx; a.M = p.n; a.out = out; a.ldo = W.rows;
+        launch_dn_gemv<DN_STORE, false>(e, W, a);
+    }
+}
+// rows of W x through the gated unit of a feed-forward
+void gated(Engine *e, PlanLayer &l, const void *x, int ldx, const Pass &p) {
+    PlanBuf &b = *p.b;
+    if (e->f32) {
+        launch_f32(e, l.gu, x, ldx, p.n, b.gu, l.gu.rows);
+        launch_k(e, lg_dn_glu_rows, dim3((l.ffp + 255) / 256, p.n), dim3(256), 0, (const float *)b.gu, l.gu.rows, l.ffp, (float *)b.act, l.down.ldk);
+    } else if (p.wide) launch_dn_gemm<DN_G_GLU>(e, l.gu, x, ldx, b.cap, p.n, b.act, l.down.ldk);
+    else {
+        LgDnGemvArgs a{};
+        a.x = (const bf16 *)x; a.ldx = ldx; a.M = p.n; a.outh = (bf16 *)b.act; a.ldoh = l.down.ldk;
+        launch_dn_gemv<DN_GLU, false>(e, l.gu, a);
+    }
+}
+
+// x in place -> every layer -> (with final_norm) the normed rows in b->h and, narrow, in e->hidden
+void plan_layers(Engine *e, const struct kvcache *kv, const Pass &p, bool final_norm, int only) {
+    PlanModel *pm = e->plan;
+    PlanBuf &b = *p.b;
+    const struct lg_plan *P = pm->plan;
+    const int W = P->width, ldh = up(W, 64);
+    if (only & C_MISC)
+        for (size_t s0 = 0; s0 < pm->rot.size(); s0 += 8) {
+            LgRotTables a{};
+            const int ns = (int)std::min(pm->rot.size() - s0, (size_t)8);
+            int half = 1;
+            for (int i = 0; i < ns; i++) { a.s[i] = {pm->rot[s0 + i].freq, pm->rot[s0 + i].dims / 2, b.tab[s0 + i]}; half = std::max(half, a.s[i].half); }
+            a.pos = p.pos; a.n_tok = p.n;
+            launch_k(e, lg_dn_rot_tables, dim3((unsigned)std::min(592, (p.n * half + 127) / 128), ns), dim3(128), 0, a);
+        }
+    LgRowNormArgs r{};
+    r.x = b.x; r.ldx = W; r.n = W; r.eps = P->norm_eps; r.center = P->norm_kind == LG_NORM_LAYER; r.mult = P->residual_mult;
+    r.y = b.h; r.ldy = ldh;
+    r.norm_w = pm->L[0].norm1;
+    if (only & C_NORM) launch_row_norm(e, p.n, r);
+    r.add = b.o;
+    for (int i = 0; i < P->n_layer; i++) {
+        PlanLayer &l = pm->L[i];
+        const bool last = i + 1 == P->n_layer;
+        float *next = last ? (final_norm ? pm->out_norm : nullptr) : pm->L[i + 1].norm1;
+        auto resid = [&](const float *add_w, const float *norm_w, bool end) {
+            r.add_w = add_w; r.norm_w = norm_w; r.ld_add = l.o.rows;
+            r.yf = end && last && final_norm && !p.wide ? e->hidden : nullptr; r.ldyf = W;
+            if (only & C_NORM) launch_row_norm(e, p.n, r);
+        };
+        if (only & C_QKV) project(e, l.in, b.h, ldh, p, b.pj);
+        latent_attention(e, kv, l, p, only);
+        if (only & C_O) project(e, l.o, b.at, l.o.ldk, p, b.o);
+        resid(l.norm1b, l.p.ff ? l.norm2 : next, !l.p.ff);
+        if (!l.p.ff) continue;
+        if (only & C_GATEUP) gated(e, l, b.h, ldh, p);
+        if (only & C_DOWN) project(e, l.down, b.act, l.down.ldk, p, b.o);
+        resid(l.norm2b, next, true);
+    }
+}
+
+void plan_embed(Engine *e, int M) { plan_embed_rows(e, e->st->toks, M, e->x); }
+
+int plan_forward(Engine *e, const struct kvcache *kv, int M, int flags, int only) {
+    PlanModel *pm = e->plan;
+    if ((only & C_MISC) && !(flags & F_NOEMBED)) plan_embed(e, M);
+    Pass p{&pm->nb, M, false, e->st->toks, &e->st->pos, 0};
+    plan_layers(e, kv, p, flags & F_HEAD, only);
+    if (e->mid_event) LG_CHECK(cudaEventRecord(e->mid_event, e->stream));
+    if (!(flags & F_HEAD) || !(only & C_HEAD)) return 1;
+    float *lg = flags & F_LOGITS ? e->logits : nullptr;
+    const int ldh = up(pm->plan->width, 64);
+    if (e->f32) {
+        if (!lg) lg = pm->logits;
+        launch_f32(e, pm->embed, pm->nb.h, ldh, M, lg, e->head.ldo);
+        launch_k(e, lg_dn_argmax_rows, dim3(32, M), dim3(256), 0, (const float *)lg, e->head.ldo, pm->plan->vocab, e->amax_val, e->amax_idx);
+        return 32;
+    }
+    LgDnGemvArgs a{};
+    a.x = (const bf16 *)pm->nb.h; a.ldx = ldh; a.M = M; a.rows = pm->plan->vocab; a.out = lg; a.ldo = e->head.ldo;
+    a.amax_val = e->amax_val; a.amax_idx = e->amax_idx;
+    return launch_dn_gemv<DN_HEAD, false>(e, pm->embed, a, e->head_ctas);
+}
+
+// buffers of the wide pass, at its first use
+bool wide_ready(Engine *e) {
+    PlanModel *pm = e->plan;
+    if (!pm->wide_ok) return false;
+    if (pm->wb.cap) return true;
+    const int cap = std::max(128, std::min(PLAN_BLOCK, pm->seq_alloc));
+    buf_alloc(e, pm->wb, cap, false);
+    pm->wb.toks = dalloc<int>(pm->seq_alloc);
+    pm->want = dalloc<int>(pm->seq_alloc);
+    const int ldh = up(pm->plan->width, 64);
+    pm->hg = dalloc<uint8_t>((size_t)PLAN_HEAD_ROWS * ldh * (e->f32 ? 4 : 2));
+    pm->wlog = dalloc<float>((size_t)PLAN_HEAD_ROWS * pm->embed.rows);
+    size_t ex = 0;
+    for (auto &l : pm->L) ex = std::max(ex, (size_t)up(l.p.heads * (l.dimp + l.vdp), 32));
+    if (!e->f32) pm->ex = dalloc<bf16>((size_t)pm->seq_alloc * ex);
+    return true;
+}
+
+int plan_prefill(Engine *e, const struct kvcache *kv, const int *toks, int n, int pos0, const int *want, int n_want, float *logits) {
+    PlanModel *pm = e->plan;
+    if (!wide_ready(e)) return 0;
+    PlanBuf &b = pm->wb;
+    const int V = pm->plan->vocab, ldh = up(pm->plan->width, 64), row_bytes = ldh * (e->f32 ? 4 : 2);
+    std::vector<int> rel(n_want), starts;
+    int i = 0, w = 0;
+    for (int k = 0; k < n_want; k++) rel[k] = want[k] % b.cap;
+    LG_CHECK(cudaMemcpyAsync(b.toks, toks, (size_t)n * 4, cudaMemcpyHostToDevice, e->stream));
+    if (n_want) LG_CHECK(cudaMemcpyAsync(pm->want, rel.data(), (size_t)n_want * 4, cudaMemcpyHostToDevice, e->stream));
+    starts.reserve(n / b.cap + 1);
+    while (n - i > LG_MAXM) {                                // a last stretch of <= 8 tokens goes through the verify path
+        const int m = std::min(b.cap, n - i);
+        starts.push_back(pos0 + i);
+        LG_CHECK(cudaMemcpyAsync(b.pos, &starts.back(), 4, cudaMemcpyHostToDevice, e->stream));
+        Pass p{&b, m, true, b.toks + i, b.pos, pos0 + i};
+        int hi = w;
+        while (hi < n_want && want[hi] < i + m) hi++;
+        plan_embed_rows(e, p.toks, m, b.x);
+        plan_layers(e, kv, p, hi > w, C_ALL);
+        for (; w < hi; w += PLAN_HEAD_ROWS) {
+            const int c = std::min(PLAN_HEAD_ROWS, hi - w);
+            launch_k(e, lg_dn_gather_rows, dim3(c), dim3(128), 0, (const void *)b.h, (const int *)(pm->want + w), pm->hg, row_bytes);
+            if (e->f32) launch_f32(e, pm->embed, pm->hg, ldh, c, pm->wlog, pm->embed.rows);
+            else launch_dn_gemm<DN_G_F32>(e, pm->embed, pm->hg, ldh, PLAN_HEAD_ROWS, c, pm->wlog, pm->embed.rows);
+            LG_CHECK(cudaMemcpy2DAsync(logits + (size_t)w * V, (size_t)V * 4, pm->wlog, (size_t)pm->embed.rows * 4, (size_t)V * 4, c, cudaMemcpyDeviceToHost, e->stream));
+        }
+        w = hi;
+        i += m;
+    }
+    check_err(e);
+    return i;
+}
+
+int plan_bench_block(Engine *e, const struct kvcache *kv, int n, int pos0, int only) {
+    PlanModel *pm = e->plan;
+    if (!wide_ready(e) || n > pm->wb.cap || pos0 + n > kv->max_seq) return -1;
+    LG_CHECK(cudaMemsetAsync(pm->wb.pos, 0, 4, e->stream));
+    Pass p{&pm->wb, n, true, pm->wb.toks, pm->wb.pos, 0};
+    if (only & C_MISC) plan_embed_rows(e, p.toks, n, pm->wb.x);
+    plan_layers(e, kv, p, false, only);
+    return 0;
+}
+
+const LgFamily plan_family = {"layer plan", plan_load, plan_release, plan_kv_init, plan_bind, plan_forward, plan_embed, plan_prefill, plan_bench_block};
+
+}  // namespace lg
+
+extern "C" const lg::LgFamily *lg_family_for(const struct gguf_context *ctx) { return lg_plan_present(ctx) ? &lg::plan_family : nullptr; }

@@ -10,6 +10,7 @@
 #include <string.h>
 #include "lg_host.h"
 #include "lg_b200.h"
+#include "lg_plan.h"
 
 /* The sampling hook lives in the caller (the reference defines it in its CLI, src/run.c:83).
  * A weak NULL default keeps the library loadable on its own; a caller's definition wins. */
@@ -25,18 +26,29 @@ struct lg_session {
 
 long long lgs_host_syncs(void *p) { return lg_host_syncs(&((struct lg_session *)p)->m); }
 
-void *lgs_open(const char *target, const char *head, int max_seq, int kv_f16_all_ignored) {
-    (void)kv_f16_all_ignored;                       /* the device cache is always f16 */
+/* Open a model -- a GGUF file or a checkpoint folder -- with an optional draft head.  f32: every product and the cache in
+ * 32-bit; only models described by a layer plan run that way. */
+void *lgs_open_as(const char *target, const char *head, int max_seq, int f32) {
     struct lg_session *s = calloc(1, sizeof *s);
     if (!s) return NULL;
-    s->g = load_gguf(target);
+    s->g = load_model(target);
     if (!s->g) { free(s); return NULL; }
+    if (f32 && !lg_plan_present(s->g)) {
+        fprintf(stderr, "session: %s does not run in 32-bit\n", target);
+        free_gguf(s->g); free(s);
+        return NULL;
+    }
+    lg_set_compute_f32(f32);
     if (model_init(&s->m, s->g) != 0) { free_gguf(s->g); free(s); return NULL; }
     if (kvcache_init(&s->kv, &s->m, max_seq) != 0) { model_free(&s->m); free_gguf(s->g); free(s); return NULL; }
     if (head && head[0]) s->head = mtp_open(head, &s->m);
     s->mtp_n = LG_MTP_N;
     lg_set_round_width(LG_MTP_N);
     return s;
+}
+void *lgs_open(const char *target, const char *head, int max_seq, int kv_f16_all_ignored) {
+    (void)kv_f16_all_ignored;                       /* the cache's element type is the model's */
+    return lgs_open_as(target, head, max_seq, 0);
 }
 void lgs_close(void *p) {
     struct lg_session *s = p;
@@ -69,6 +81,13 @@ void lgs_forward(void *p, int tok, int pos, float *logits) {
 void lgs_last_hidden(void *p, float *out) { lg_last_hidden(&((struct lg_session *)p)->m, out); }
 int  lgs_next(void *p, int tok, int pos) { struct lg_session *s = p; return model_forward_next(&s->m, &s->kv, tok, pos); }
 void lgs_prefill(void *p, const int *toks, int n, int pos0) { struct lg_session *s = p; model_prefill(&s->m, &s->kv, toks, n, pos0); }
+int  lgs_prefill_logits(void *p, const int *toks, int n, int pos0, const int *want, int n_want, float *logits) {
+    struct lg_session *s = p; return lg_prefill_logits(&s->m, &s->kv, toks, n, pos0, want, n_want, logits);
+}
+void lgs_prefix(void *p, int n, int restore) {
+    struct lg_session *s = p;
+    if (restore) kvcache_restore_prefix(&s->kv, n); else kvcache_save_prefix(&s->kv, n);
+}
 void lgs_prefill_mixed(void *p, const float *rows, const int *ids, int n, int pos0) {
     struct lg_session *s = p; model_prefill_mixed(&s->m, &s->kv, rows, ids, n, pos0);
 }

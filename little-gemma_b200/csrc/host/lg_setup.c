@@ -1,6 +1,7 @@
 /* lg_setup.c -- host-side set-up: hyper-parameters and per-layer geometry of the target model,
  * and opening / validating a draft head.  Independent implementation of the behaviour of the
  * little-gemma host (src/model.c:67-189 target; src/mtp.c:124-262 head):
+ *   - a model described by a layer plan (lg_plan.h) takes its geometry from the plan; for the others:
  *   - metadata keys are prefixed with general.architecture;
  *   - head_count, head_count_kv, feed_forward_length may be scalars or per-layer i32 arrays;
  *   - n_vocab is the length of tokenizer.ggml.tokens;
@@ -14,6 +15,7 @@
 #include <stdlib.h>
 #include <string.h>
 #include "lg_host.h"
+#include "lg_plan.h"
 
 extern const int model_kv_host;
 int  mtp_draft_device(struct mtp *, const struct model *, const struct kvcache *, int, int);
@@ -71,6 +73,7 @@ int config_load(struct config *c, const struct gguf_context *g) {
     c->n_kv_start = shared > 0 ? c->n_layer - shared : c->n_layer;
     const struct gguf_meta *vocab = gguf_find_meta(g, "tokenizer.ggml.tokens");
     if (vocab && vocab->type == GGUF_TYPE_ARRAY) c->n_vocab = (int)vocab->value.arr.n;
+    else c->n_vocab = arch_int(g, arch, "vocab_size", 0, 0);
     if (c->n_layer <= 0 || c->n_layer > 4096) {
         fprintf(stderr, "config: %s.block_count = %d is not a usable layer count\n", arch, c->n_layer);
         return -1;
@@ -82,6 +85,19 @@ static const struct gguf_tensor *layer_tensor(const struct gguf_context *g, int 
     char name[96];
     snprintf(name, sizeof name, "blk.%d.%s", L, leaf);
     return gguf_find_tensor(g, name);
+}
+
+/* geometry of a model described by a layer plan: one latent row per position and layer, read by every head */
+static int plan_geometry(struct model *m, const struct gguf_context *g) {
+    struct lg_plan *p = lg_plan_read(g);
+    if (!p) return -1;
+    for (int L = 0; L < p->n_layer; L++) {
+        m->ffn_len[L] = p->layer[L].ff;
+        m->head_dim[L] = p->layer[L].dim + p->layer[L].rot_dim;
+        m->n_head_kv[L] = 1;
+    }
+    lg_plan_free(p);
+    return 0;
 }
 
 int model_init(struct model *m, const struct gguf_context *g) {
@@ -96,6 +112,8 @@ int model_init(struct model *m, const struct gguf_context *g) {
     m->n_head_kv = calloc(nl, sizeof(int));
     m->last_hidden = calloc((size_t)(c->n_embd > 0 ? c->n_embd : 1), sizeof(float));
     if (!m->is_local || !m->ffn_len || !m->head_dim || !m->n_head_kv || !m->last_hidden) return -1;
+
+    if (lg_plan_present(g)) return plan_geometry(m, g);
 
     const struct gguf_meta *pat = arch_meta(g, c->arch, "attention.sliding_window_pattern");
     int have_pat = pat && pat->type == GGUF_TYPE_ARRAY && pat->value.arr.type == GGUF_TYPE_BOOL;
