@@ -4,6 +4,7 @@
     python bench.py [--gpus N] [--steps K] [--warmup W] [--impl ours|reference]
                     [--config b12|b12k|e4b|tiny|c5] [--depth D] [--p P] [--mtp-n M]
     python bench.py --sweep e4b|b12|b12k [--sweep-out FILE.md]
+    python bench.py --design mubopel [--design-out FILE.md]
 
 One "step" is one MTP round at batch 1: M-1 draft-head forwards, one M-token verify forward of
 the target (every weight streamed once), greedy acceptance and position advance -- all on the
@@ -26,6 +27,10 @@ recorded plain-greedy stream with probability p, because a random-init head acce
 --config c5 is the serving workload of the plan: a 2048-token prompt and 1024 generated tokens at
 p = 0.7 per session (K is then the number of rounds that took).  --sweep runs the plan's tables for
 one model (KV depth x verify width x acceptance) and writes them as markdown.
+
+--design mubopel times prefill and decode of the latent-attention design at sizes of real models' layers (random weights)
+beside the block-quantised family at equal width, heads, feed-forward, depth and vocabulary, kernel class by kernel class
+against its roofline; it replaces the benchmark line.
 
 N > 1 (torchrun): one independent replica per GPU, own prompt seed, no collective on the data
 path; a gloo barrier brackets the timed region and the max time over ranks is used.
@@ -291,6 +296,172 @@ def sweep(a, lg, synth, torch):
         f.write("\n".join(lines) + "\n")
 
 
+# ---------------------------------------------------------------------------------------------
+# the latent-attention design beside the block-quantised family
+# ---------------------------------------------------------------------------------------------
+C_QKV, C_O, C_GATEUP, C_DOWN, C_HEAD, C_EXPAND, C_NORM, C_ATTN, C_MISC, C_FUSED = 1, 2, 4, 8, 16, 32, 64, 256, 512, 1024
+
+
+def design_shapes(synth, name):
+    """(layer-plan shape, block-quantised shape) of equal width, head count, feed-forward, layers and vocabulary"""
+    W, H, q, ff, n, V = {"2b": (2048, 16, 768, 8192, 8, 32768), "8b": (4096, 32, 1536, 14336, 6, 32768),
+                         "16b": (5120, 64, 1536, 16384, 4, 32768)}[name]
+    lay = [synth.LatentLayer(heads=H, dim=128, rot_dim=64, vdim=128, q_rank=q, kv_rank=512, ff=ff) for _ in range(n)]
+    return (synth.LatentShape(width=W, vocab=V, layers=lay),
+            synth.TargetShape(n_layer=n, n_embd=W, n_head=H, n_head_kv=max(4, H // 4), head_dim=128, n_ff=ff, n_vocab=V, window=1 << 20,
+                              local_per_global=0, ple=0))
+
+
+class DesignTimer:
+    """Device time of enqueued work, cold: L2 is overwritten before every timed iteration."""
+
+    def __init__(self, torch, sess):
+        self.t, self.stream = torch, torch.cuda.ExternalStream(sess.stream())
+        self.flush = torch.empty(512 << 20, dtype=torch.uint8, device="cuda")
+
+    def __call__(self, fn, reps=8, warm=3):
+        for _ in range(warm):
+            fn()
+        self.t.cuda.synchronize()
+        total = 0.0
+        for _ in range(reps):
+            with self.t.cuda.stream(self.stream):
+                self.flush.zero_()
+                a, b = self.t.cuda.Event(enable_timing=True), self.t.cuda.Event(enable_timing=True)
+                a.record(self.stream)
+                fn()
+                b.record(self.stream)
+            b.synchronize()
+            total += a.elapsed_time(b)
+        return total / reps
+
+
+def design_model(a, lg, synth, torch, path, latent, shape, n_pf, depths, peaks):
+    """One model: whole-step and per-class device times, with the algorithmic bytes or operations of each class."""
+    L = len(shape.layers) if latent else shape.n_layer
+    W, V = (shape.width, shape.vocab) if latent else (shape.n_embd, shape.n_vocab)
+    hbm, tc = float(peaks.get("hbm_gbs", 6650.0)) * 1e9, float(peaks.get("bf16_tflops_sustained", 1400.0)) * 1e12
+    bpw = 2.0 if latent else 0.5625
+    if latent:
+        l = shape.layers[0]
+        H, hd, ff = l.heads, l.dim + l.rot_dim, l.ff
+        proj = W * (l.q_rank + l.kv_rank + l.rot_dim + H * l.vdim) + l.q_rank * H * hd
+        kv_w, out_w = l.kv_rank * H * l.dim, l.kv_rank * H * l.vdim
+        par = {"qkv": proj + kv_w, "o": out_w + H * l.vdim * W, "gateup": 2 * W * ff, "down": W * ff}
+        pf_par = {"qkv": proj, "o": H * l.vdim * W, "gateup": 2 * W * ff, "down": W * ff}
+        kv_row, pair = 2 * (l.kv_rank + l.rot_dim), 2 * H * (hd + l.vdim)
+    else:
+        H, Hkv, hd, ff = shape.n_head, shape.n_head_kv, shape.head_dim, shape.n_ff
+        par = {"qkv": W * (H + 2 * Hkv) * hd, "o": H * hd * W, "gateup": 2 * W * ff, "down": W * ff}
+        pf_par, kv_row, pair = par, 4 * Hkv * hd, 4 * H * hd
+    cls = {"qkv": C_QKV, "o": C_O, "gateup": C_GATEUP, "down": C_DOWN}
+    res = {"decode": {}, "prefill": {}}
+    with lg.Session(path, None, max(depths) + 512) as s:
+        tm = DesignTimer(torch, s)
+        prompt = synth.prompt_ids(max(depths), V, seed=11)
+        for d in depths:
+            s.prefill(prompt[:d - 1], 0)
+            first = s.next(int(prompt[d - 1]), d - 1)
+            def steps(n):
+                s.rounds_begin(first, d, 1)
+                s.rounds_enqueue(1, 0, n)
+            steps(16)
+            torch.cuda.synchronize()
+            clk = ClockSampler()
+            clk.start()
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            s.rounds_begin(first, d, 1)
+            e0.record(tm.stream)
+            s.rounds_enqueue(1, 0, 128)
+            e1.record(tm.stream)
+            e1.synchronize()
+            ms = e0.elapsed_time(e1) / 128
+            byts = bpw * (L * sum(par.values()) + W * V) + L * d * kv_row
+            r = {"step": {"us": ms * 1e3, "tok_s": 1e3 / ms, "frac": byts / (ms * 1e-3) / hbm}, "clocks": clk.stop()}
+            s.rounds_begin(first, d, 1)
+            torch.cuda.synchronize()
+            for name, c in cls.items():
+                us = tm(lambda c=c: s.matmul_pass(1, c | C_FUSED)) * 1e3 / L
+                r[name] = {"us": us, "frac": bpw * par[name] / (us * 1e-6) / hbm}
+            us = tm(lambda: s.matmul_pass(1, C_HEAD)) * 1e3
+            r["head"] = {"us": us, "frac": bpw * W * V / (us * 1e-6) / hbm}
+            us = tm(lambda: s.matmul_pass(1, C_ATTN)) * 1e3 / L
+            r["attention"] = {"us": us, "frac": d * kv_row / (us * 1e-6) / hbm}
+            us = tm(lambda: s.matmul_pass(1, C_NORM)) * 1e3 / L
+            r["norms"] = {"us": us}
+            res["decode"][d] = r
+        for n in n_pf:
+            s.prefill(prompt[:n], 0)
+            torch.cuda.synchronize()
+            t0 = time.perf_counter()
+            for _ in range(3):
+                s.prefill(prompt[:n], 0)
+            torch.cuda.synchronize()
+            ms = (time.perf_counter() - t0) / 3 * 1e3
+            pairs = n * (n + 1) / 2
+            fl = 2.0 * L * n * (sum(pf_par.values()) + ((kv_w + out_w) if latent else 0)) + L * pairs * pair
+            r = {"prompt": {"ms": ms, "tok_s": n / ms * 1e3, "frac": fl / (ms * 1e-3) / tc}}
+            blk = min(n, 2048 if latent else 256)              # the family's own block
+            keys0 = 0 if latent else (n - 1) // 256 * 256      # where the block the class passes repeat sits
+            if latent:
+                cl = dict(cls, expand=C_EXPAND)
+                pp = dict(pf_par, expand=kv_w + out_w)
+            else:
+                cl, pp = cls, pf_par
+            for name, c in cl.items():
+                us = tm(lambda c=c: s.prefill_pass(blk, c)) * 1e3 / L
+                r[name] = {"us": us, "frac": 2.0 * blk * pp[name] / (us * 1e-6) / tc}
+            us = tm(lambda: s.prefill_pass(blk, C_ATTN)) * 1e3 / L
+            pairs = blk * (keys0 + (blk + 1) / 2)
+            r["attention"] = {"us": us, "frac": pairs * pair / (us * 1e-6) / tc}
+            us = tm(lambda: s.prefill_pass(blk, C_NORM)) * 1e3 / L
+            r["norms"] = {"us": us, "block": blk}
+            res["prefill"][n] = r
+    return res
+
+
+def design(a, lg, synth, torch):
+    peaks = load_peaks()
+    lines = ["# The latent-attention design beside the block-quantised family", "",
+             "`python bench.py --design mubopel`: random weights, batch 1.  `latent` = Mubopel (bf16), `q4` = the block-quantised family (q4_0) of",
+             "equal width, heads, feed-forward, layers and vocabulary.  `frac` = algorithmic bytes (decode) or operations (prefill) over device",
+             f"time, of the measured copy bandwidth ({peaks.get('hbm_gbs')} GB/s) or sustained bf16 throughput ({peaks.get('bf16_tflops_sustained')} TFLOP/s).",
+             "Kernel classes: device time per layer, all layers' launches of the class back to back, L2 overwritten before each pass; prefill",
+             "classes on one block (2048 tokens from position 0, or the q4 family's last block of 256).", ""]
+    out = {}
+    for name in a.design_sizes.split(","):
+        ls, ts = design_shapes(synth, name)
+        lp = os.path.join(CACHE, f"mubopel_{name}")
+        if not os.path.exists(os.path.join(lp, "config.json")):
+            synth.write_checkpoint(lp, ls, 0, fast=True)
+        tp = synth.cached(CACHE, f"plain_{name}.gguf", synth.write_target, ts, 0, "cuda")
+        torch.cuda.empty_cache()
+        depths, n_pf = [1024, 8192], [2048]
+        both = {"latent": design_model(a, lg, synth, torch, lp, True, ls, n_pf, depths, peaks)}
+        if not a.design_alone:
+            both["q4"] = design_model(a, lg, synth, torch, tp, False, ts, n_pf, depths, peaks)
+        out[name] = both
+        lines += [f"## {name}: width {ls.width}, {ls.layers[0].heads} heads, ff {ls.layers[0].ff}, {len(ls.layers)} layers", "",
+                  "| | latent | frac | q4 | frac |", "|---|---|---|---|---|"]
+        for kind in ("decode", "prefill"):
+            for d, rl in both["latent"][kind].items():
+                rq = both.get("q4", {kind: {d: {}}})[kind][d]
+                for k, v in rl.items():
+                    if k == "clocks":
+                        continue
+                    q = rq.get(k, {})
+                    show = lambda x: "" if not x else (f"{x['tok_s']:.0f} tok/s ({x.get('ms', x.get('us', 0) / 1e3):.2f} ms)" if "tok_s" in x else f"{x['us']:.1f} us")
+                    fr = lambda x: f"{x['frac']:.3f}" if "frac" in x else ""
+                    lines.append(f"| {kind} {d}: {k} | {show(v)} | {fr(v)} | {show(q)} | {fr(q)} |")
+        lines += [""] + [f"clocks ({k}): {v['decode'][1024]['clocks']}" for k, v in both.items()] + [""]
+    text = "\n".join(lines)
+    if a.design_out:
+        with open(a.design_out, "w") as f:
+            f.write(text + "\n")
+    print(text, flush=True)
+    print(json.dumps({"design": "mubopel", "results": out}), flush=True)
+
+
 def load_peaks():
     try:
         return json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json")))
@@ -356,6 +527,10 @@ def main():
     ap.add_argument("--profile-prefill", type=int, default=None, metavar="CLASSES",
                     help="short path for profilers: load, model_prefill of 512 tokens, 3 wide prompt blocks of 256 tokens "
                          "restricted to kernel classes (4 = gate/up matmul, 1023 = everything), exit")
+    ap.add_argument("--design", default=None, choices=["mubopel"], help="time a design beside the block-quantised family instead of the benchmark line")
+    ap.add_argument("--design-sizes", default="2b,8b,16b")
+    ap.add_argument("--design-alone", action="store_true", help="with --design: leave the block-quantised family out")
+    ap.add_argument("--design-out", default=None, help="with --design: also write the table to this file")
     ap.add_argument("--layers", type=int, default=0, help="cut the model to this many layers (small profiling cases)")
     a = ap.parse_args()
     a.warmup = max(a.warmup, 3)
@@ -410,6 +585,9 @@ def main():
     build = importlib.import_module("little-gemma_b200.build")
     if RANK == 0:
         build.build()
+    if a.design:
+        design(a, lg, synth, torch)
+        return
     if a.sweep:
         sweep(a, lg, synth, torch)
         return

@@ -79,6 +79,17 @@ __device__ __forceinline__ void rot_q_rows(const LgRotQ &a, int tok, int first, 
     }
 }
 
+// the same inside the query rows themselves (q == out)
+__device__ __forceinline__ void rot_q_in_place(const LgRotQ &a, int tok, int first, int stride) {
+    const int half = a.rot_dims >> 1;
+    for (int u = first; u < a.H * half; u += stride) {
+        const int h = u / half, i = u % half;
+        uint32_t *p = (uint32_t *)((bf16 *)a.out + (size_t)tok * a.ldq + (size_t)h * a.head_stride + a.rot_at_q) + i;
+        const float2 x = __bfloat1622float2(*(const __nv_bfloat162 *)p), cs = a.tab[(size_t)tok * half + i];
+        *p = pack_bf16(x.x * cs.x - x.y * cs.y, x.y * cs.x + x.x * cs.y);
+    }
+}
+
 // ---------------------------------------------------------------------------------------------
 // small-M matmul: out[tok][row] = W x[tok] for M <= 8 rows at once, bf16 weights streamed once
 // ---------------------------------------------------------------------------------------------
@@ -247,6 +258,7 @@ template <int NT> __host__ __device__ constexpr size_t dn_gemm_smem() {
 }
 struct LgDnGemmArgs {
     int nkb, n_tok, cols;            // blocks of k; valid tokens; stored columns (a multiple of 32)
+    int w_early;                     // the second operand does not depend on earlier kernels
     void *out; int ldo;              // f32 / bf16 rows; GLU: bf16 rows of cols / 2
     int *err;
 };
@@ -263,7 +275,6 @@ __global__ void __launch_bounds__(DN_GEMM_THREADS) lg_dn_gemm_kernel(const __gri
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int row0 = blockIdx.x * NT, tok0 = blockIdx.y * DN_GEMM_BM, nkb = a.nkb;
 
-    pdl_launch();
     if (threadIdx.x == 0) {
         for (int i = 0; i < ST; i++) { mbar_init(full + i, 1); mbar_init(empty + i, 1); }
         mbar_init(acc_full, 1);
@@ -276,15 +287,17 @@ __global__ void __launch_bounds__(DN_GEMM_THREADS) lg_dn_gemm_kernel(const __gri
     __syncthreads();
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
     const uint32_t tmem = *tmem_slot;
+    pdl_launch();                        // only now: a dependant must not take tensor memory a CTA of this grid still waits for
 
     if (warp == 4) {
         if (lane == 0) {
             const int pre = min(ST, nkb);
+            if (!a.w_early) pdl_wait();
             for (int kb = 0; kb < pre; kb++) {
                 mbar_expect_tx(full + kb, A_BYTES + B_BYTES);
                 tma_load_2d(sB + kb * B_BYTES, &tmw, kb * DN_GEMM_BK, row0, full + kb);
             }
-            pdl_wait();
+            if (a.w_early) pdl_wait();
             for (int kb = 0; kb < pre; kb++) tma_load_2d(sA + kb * A_BYTES, &tmx, kb * DN_GEMM_BK, tok0, full + kb);
             bool ok = true;
             int issued = pre;

@@ -3,6 +3,7 @@
 // latent cache; prompts run blocks of up to PLAN_BLOCK tokens through the tcgen05 matmul and the block attention.  In 32-bit
 // mode every product, activation and cache row is f32.
 #include <algorithm>
+#include <tuple>
 #include "lg_engine.h"
 #include "lg_plan.h"
 #include "lg_latent.cuh"
@@ -29,7 +30,7 @@ struct PlanLayer {
     int kv_off, rot_off, g_off;                               // columns of the input projection's row: [query latent | latent | key part | gate]
     int owns, spec;                                           // spec: which rotation table
     int rt;                                                   // row tiles of 16 per CTA of the decode attention (0: the row kernel)
-    DMat in, uq, ukT, ukv, uv, o, gu, down;
+    DMat in, uq, ukT, uk, uv, o, gu, down;             // uk: keys from latents (prompt pass); ukT: the same per head, transposed (decode)
     float *norm1, *norm1b, *norm2 = nullptr, *norm2b = nullptr, *q_norm, *kv_norm = nullptr, *sink;
 };
 
@@ -54,10 +55,10 @@ struct PlanModel {
     // bound to a cache
     int max_seq = 0, seq_alloc = 0, C = 1;
     float *part = nullptr; float2 *part_ml = nullptr;
-    bf16 *ex = nullptr;
+    bf16 *kx = nullptr, *vx = nullptr;                       // one layer's expanded keys [position][H dimp] and values [H vdp][position]
     int *want = nullptr; void *hg = nullptr; float *wlog = nullptr;
     float *logits = nullptr;                                  // 32-bit: rows of a head without F_LOGITS
-    std::map<std::pair<const void *, long long>, CUtensorMap> maps;
+    std::map<std::tuple<const void *, int, int, int>, CUtensorMap> maps;
 };
 
 // ------------------------------------------------------------------------------------------
@@ -147,7 +148,7 @@ void plan_attributes() {
     smem_attr(lg_dn_gemm_kernel<128, DN_G_GLU>, dn_gemm_smem<128>()); smem_attr(lg_dn_gemm_kernel<256, DN_G_GLU>, dn_gemm_smem<256>());
     smem_attr(lg_latent_dec_attn_kernel<1, 2>); smem_attr(lg_latent_dec_attn_kernel<1, 4>); smem_attr(lg_latent_dec_attn_kernel<1, 8>);
     smem_attr(lg_latent_dec_attn_kernel<2, 2>); smem_attr(lg_latent_dec_attn_kernel<2, 4>); smem_attr(lg_latent_dec_attn_kernel<2, 8>);
-    smem_attr(lg_latent_pf_attn_kernel<8>); smem_attr(lg_latent_pf_attn_kernel<16>); smem_attr(lg_latent_pf_attn_kernel<32>);
+    smem_attr(lg_latent_pf_attn_kernel);
     smem_attr(lg_latent_merge_kernel, PLAN_SMEM_SMALL); smem_attr(lg_latent_attn_rows_kernel<float>, PLAN_SMEM_SMALL); smem_attr(lg_latent_attn_rows_kernel<bf16>, PLAN_SMEM_SMALL);
 }
 
@@ -239,12 +240,11 @@ void plan_load(Engine *e) {
             put_groups(b, 0, uv, H, p.vdim, l.vdp);
             l.uv = b.upload(e);
         }
-        if (!e->f32) {   // both expansions, for the prompt pass
-            MatBuild b(e, H * (l.dimp + l.vdp), p.kv_rank);
+        if (!e->f32) {
+            MatBuild b(e, H * l.dimp, p.kv_rank);
             put_groups(b, 0, uk, H, p.dim, l.dimp);
-            put_groups(b, H * l.dimp, uv, H, p.vdim, l.vdp);
             const size_t before = e->weight_bytes;
-            l.ukv = b.upload(e);
+            l.uk = b.upload(e);
             e->weight_bytes = before;                        // a second copy of weights already counted
         }
         {
@@ -279,7 +279,7 @@ void plan_load(Engine *e) {
         }
         l.rt = l.kvp > 512 ? 0 : lg_latent_dec_smem(2, l.ldc) <= PLAN_SMEM_MAX ? 2 : lg_latent_dec_smem(1, l.ldc) <= PLAN_SMEM_MAX ? 1 : 0;
         if (e->f32) l.rt = 0;
-        if (l.vdp > 256 || lg_latent_pf_smem(l.dimp + l.rotp, l.vdp) > PLAN_SMEM_MAX) pm->wide_ok = false;
+        if (l.vdp > 256 || lg_latent_pf_smem(l.dimp, l.rotp, l.vdp) > PLAN_SMEM_MAX) pm->wide_ok = false;
         if ((size_t)(l.ldc + l.kvp + 128) * 4 > PLAN_SMEM_SMALL || (size_t)LG_LM_GROUPS * l.kvp * 4 > PLAN_SMEM_SMALL ||
             (size_t)LG_MAXM * (l.uq.ldk + 8) * 2 > PLAN_SMEM_SMALL) { fprintf(stderr, "lg_b200: layer %d: latent sizes beyond what the kernels hold\n", i); exit(1); }
     }
@@ -300,8 +300,8 @@ void plan_load(Engine *e) {
 
 void dmat_free(DMat &m) { cudaFree(m.w); m = DMat(); }
 void plan_unbind(PlanModel *pm) {
-    cudaFree(pm->part); cudaFree(pm->part_ml); cudaFree(pm->ex); cudaFree(pm->want); cudaFree(pm->hg); cudaFree(pm->wlog);
-    pm->part = nullptr; pm->part_ml = nullptr; pm->ex = nullptr; pm->want = nullptr; pm->hg = nullptr; pm->wlog = nullptr;
+    cudaFree(pm->part); cudaFree(pm->part_ml); cudaFree(pm->kx); cudaFree(pm->vx); cudaFree(pm->want); cudaFree(pm->hg); cudaFree(pm->wlog);
+    pm->part = nullptr; pm->part_ml = nullptr; pm->kx = pm->vx = nullptr; pm->want = nullptr; pm->hg = nullptr; pm->wlog = nullptr;
     if (pm->wb.cap) buf_free(pm->wb, false);
     pm->maps.clear();
 }
@@ -310,7 +310,7 @@ void plan_release(Engine *e) {
     if (!pm) return;
     plan_unbind(pm);
     for (auto &l : pm->L) {
-        for (DMat *m : {&l.in, &l.uq, &l.ukT, &l.ukv, &l.uv, &l.o, &l.gu, &l.down}) dmat_free(*m);
+        for (DMat *m : {&l.in, &l.uq, &l.ukT, &l.uk, &l.uv, &l.o, &l.gu, &l.down}) dmat_free(*m);
         for (float *v : {l.norm1, l.norm1b, l.norm2, l.norm2b, l.q_norm, l.kv_norm, l.sink}) cudaFree(v);
     }
     for (auto &r : pm->rot) cudaFree(r.freq);
@@ -392,21 +392,29 @@ int launch_dn_gemv(Engine *e, const DMat &W, LgDnGemvArgs a, int cap_ctas = 1 <<
     }
     return a.n_main;
 }
+// descriptor of a bf16 activation buffer [rows][ld], of which k columns count; made once per buffer, width and box
+const CUtensorMap &buf_map(PlanModel *pm, const void *x, int k, int ld, int rows, int box_r) {
+    const auto key = std::make_tuple(x, k, ld, box_r);
+    auto it = pm->maps.find(key);
+    if (it == pm->maps.end())
+        it = pm->maps.emplace(key, tiled_map(x, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, std::min(k, ld), rows, (long long)ld * 2, DN_GEMM_BK, box_r)).first;
+    return it->second;
+}
+// out[i][j] = row i of x (n of them count) . row j of w (w_rows, a multiple of 32); maps of w with boxes of 128 / 256 rows
+template <int EPI>
+void launch_gemm_maps(Engine *e, const CUtensorMap &x, int n, const CUtensorMap &w128, const CUtensorMap &w256, int w_rows, int nkb, void *out, int ldo, bool w_early) {
+    LgDnGemmArgs a{};
+    a.nkb = nkb; a.n_tok = n; a.cols = w_rows; a.out = out; a.ldo = ldo; a.err = e->err; a.w_early = w_early;
+    const int ty = (n + DN_GEMM_BM - 1) / DN_GEMM_BM;
+    if ((w_rows + 255) / 256 * ty >= e->sm_count)
+        launch_k(e, lg_dn_gemm_kernel<256, EPI>, dim3((w_rows + 255) / 256, ty), dim3(DN_GEMM_THREADS), dn_gemm_smem<256>(), x, w256, a);
+    else
+        launch_k(e, lg_dn_gemm_kernel<128, EPI>, dim3((w_rows + 127) / 128, ty), dim3(DN_GEMM_THREADS), dn_gemm_smem<128>(), x, w128, a);
+}
 // x: [x_rows][ldx] bf16, of which n rows count
 template <int EPI>
 void launch_dn_gemm(Engine *e, const DMat &W, const void *x, int ldx, int x_rows, int n, void *out, int ldo) {
-    PlanModel *pm = e->plan;
-    const auto key = std::make_pair(x, (long long)ldx << 32 | W.k);
-    auto it = pm->maps.find(key);
-    if (it == pm->maps.end())
-        it = pm->maps.emplace(key, tiled_map(x, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, std::min(W.k, ldx), x_rows, (long long)ldx * 2, DN_GEMM_BK, DN_GEMM_BM)).first;
-    LgDnGemmArgs a{};
-    a.nkb = W.ldk / DN_GEMM_BK; a.n_tok = n; a.cols = W.rows; a.out = out; a.ldo = ldo; a.err = e->err;
-    const int ty = (n + DN_GEMM_BM - 1) / DN_GEMM_BM;
-    if ((W.rows + 255) / 256 * ty >= e->sm_count)
-        launch_k(e, lg_dn_gemm_kernel<256, EPI>, dim3((W.rows + 255) / 256, ty), dim3(DN_GEMM_THREADS), dn_gemm_smem<256>(), it->second, W.map[1], a);
-    else
-        launch_k(e, lg_dn_gemm_kernel<128, EPI>, dim3((W.rows + 127) / 128, ty), dim3(DN_GEMM_THREADS), dn_gemm_smem<128>(), it->second, W.map[0], a);
+    launch_gemm_maps<EPI>(e, buf_map(e->plan, x, W.k, ldx, x_rows, DN_GEMM_BM), n, W.map[0], W.map[1], W.rows, W.ldk / DN_GEMM_BK, out, ldo, true);
 }
 void launch_f32(Engine *e, const DMat &W, const void *x, int ldx, int n, void *out, int ldo, int groups = 1, int group_rows = 0, int x_group = 0, int out_group = 0) {
     LgDnF32Args a{};
@@ -478,21 +486,25 @@ void latent_attention(Engine *e, const struct kvcache *kv, PlanLayer &l, const P
         return;
     }
     if (p.wide) {
-        const int keys = p.pos0 + n, ldx = up(H * (l.dimp + l.vdp), 32);
+        const int keys = p.pos0 + n;
         if (only & C_MISC) launch_k(e, lg_latent_prep_kernel<bf16>, dim3(n), dim3(128), 0, pa);
         if (only & C_QKV) launch_dn_gemm<DN_G_BF16>(e, l.uq, b.cq, l.uq.ldk, b.cap, n, b.q, ldq);
-        if (only & C_PLE) launch_dn_gemm<DN_G_BF16>(e, l.ukv, cache, l.ldc, pm->seq_alloc, keys, pm->ex, ldx);
+        if (only & C_MISC) {
+            rq.out = b.q;
+            launch_k(e, lg_latent_rot_rows_kernel, dim3((unsigned)std::min(16, (H * l.p.rot_dims / 2 + 127) / 128 + 1), n), dim3(128), 0, rq);
+        }
+        if (only & C_PLE) {                        // keys [position][H dimp], values transposed [H vdp][position]
+            launch_dn_gemm<DN_G_BF16>(e, l.uk, cache, l.ldc, pm->seq_alloc, keys, pm->kx, l.uk.rows);
+            launch_gemm_maps<DN_G_BF16>(e, l.uv.map[0], H * l.vdp, buf_map(pm, cache, l.p.kv_rank, l.ldc, pm->seq_alloc, 128),
+                                        buf_map(pm, cache, l.p.kv_rank, l.ldc, pm->seq_alloc, 256), up(keys, 32), l.uv.ldk / DN_GEMM_BK, pm->vx, pm->seq_alloc, false);
+        }
         if (!(only & C_ATTN)) return;
         LgLatentPfArgs a{};
-        a.q = (const bf16 *)b.q; a.ldq = ldq; a.ex = pm->ex; a.ldx = ldx; a.cache = (const bf16 *)cache; a.ldc = l.ldc; a.rot_at = l.kvp;
-        a.H = H; a.dimp = l.dimp; a.rotp = l.rotp; a.rot_dims = l.p.rot_dims; a.vdp = l.vdp; a.n = n;
-        a.tab = b.tab[l.spec]; a.sink = l.sink; a.scale = l.p.scale; a.gate = gate; a.ldg = l.in.rows; a.pos = p.pos;
-        a.out = (bf16 *)b.at; a.ldo = ld_at;
-        const dim3 grid((n + LG_LP_Q - 1) / LG_LP_Q, H), block(LG_LP_THREADS);
-        const size_t sm = lg_latent_pf_smem(qh, l.vdp);
-        if (l.vdp <= 64) launch_k(e, lg_latent_pf_attn_kernel<8>, grid, block, sm, a);
-        else if (l.vdp <= 128) launch_k(e, lg_latent_pf_attn_kernel<16>, grid, block, sm, a);
-        else launch_k(e, lg_latent_pf_attn_kernel<32>, grid, block, sm, a);
+        a.H = H; a.dimp = l.dimp; a.rotp = l.rotp; a.vdp = l.vdp; a.n = n; a.rot_at = l.kvp; a.scale = l.p.scale; a.sink = l.sink;
+        a.gate = gate; a.ldg = l.in.rows; a.pos = p.pos; a.out = (bf16 *)b.at; a.ldo = ld_at; a.err = e->err;
+        launch_k(e, lg_latent_pf_attn_kernel, dim3((n + LG_LP_Q - 1) / LG_LP_Q, H), dim3(LG_LP_THREADS), lg_latent_pf_smem(l.dimp, l.rotp, l.vdp),
+                 buf_map(pm, b.q, ldq, ldq, b.cap, LG_LP_Q), buf_map(pm, pm->kx, l.uk.rows, l.uk.rows, pm->seq_alloc, LG_LP_S),
+                 buf_map(pm, cache, l.ldc, l.ldc, pm->seq_alloc, LG_LP_S), buf_map(pm, pm->vx, pm->seq_alloc, pm->seq_alloc, l.uv.rows, l.vdp), a);
         return;
     }
     if (only & C_QKV) {
@@ -509,19 +521,21 @@ void latent_attention(Engine *e, const struct kvcache *kv, PlanLayer &l, const P
         if (!l.rt) launch_k(e, lg_latent_attn_rows_kernel<bf16>, dim3(H, n), dim3(128), rows_sm, ra);
         else {
             LgLatentDecArgs a{};
-            a.q = (const bf16 *)b.qa; a.cache = (const bf16 *)cache; a.ldc = l.ldc; a.kvp = l.kvp; a.rows = n * H; a.H = H;
+            const CUtensorMap &cm = buf_map(pm, cache, l.ldc, l.ldc, pm->seq_alloc, LG_LD_S);
+            a.err = e->err;
+            a.q = (const bf16 *)b.qa; a.ldc = l.ldc; a.kvp = l.kvp; a.rows = n * H; a.H = H;
             a.scale = l.p.scale; a.pos = p.pos; a.part = pm->part; a.part_ml = pm->part_ml;
             const int rt = n * H > 16 ? l.rt : 1;
             const dim3 grid(pm->C, (n * H + 16 * rt - 1) / (16 * rt)), block(LG_LD_THREADS);
             const size_t sm = lg_latent_dec_smem(rt, l.ldc);
             if (rt == 2) {
-                if (l.kvp <= 128) launch_k(e, lg_latent_dec_attn_kernel<2, 2>, grid, block, sm, a);
-                else if (l.kvp <= 256) launch_k(e, lg_latent_dec_attn_kernel<2, 4>, grid, block, sm, a);
-                else launch_k(e, lg_latent_dec_attn_kernel<2, 8>, grid, block, sm, a);
+                if (l.kvp <= 128) launch_k(e, lg_latent_dec_attn_kernel<2, 2>, grid, block, sm, cm, a);
+                else if (l.kvp <= 256) launch_k(e, lg_latent_dec_attn_kernel<2, 4>, grid, block, sm, cm, a);
+                else launch_k(e, lg_latent_dec_attn_kernel<2, 8>, grid, block, sm, cm, a);
             } else {
-                if (l.kvp <= 128) launch_k(e, lg_latent_dec_attn_kernel<1, 2>, grid, block, sm, a);
-                else if (l.kvp <= 256) launch_k(e, lg_latent_dec_attn_kernel<1, 4>, grid, block, sm, a);
-                else launch_k(e, lg_latent_dec_attn_kernel<1, 8>, grid, block, sm, a);
+                if (l.kvp <= 128) launch_k(e, lg_latent_dec_attn_kernel<1, 2>, grid, block, sm, cm, a);
+                else if (l.kvp <= 256) launch_k(e, lg_latent_dec_attn_kernel<1, 4>, grid, block, sm, cm, a);
+                else launch_k(e, lg_latent_dec_attn_kernel<1, 8>, grid, block, sm, cm, a);
             }
             LgLatentMergeArgs m{};
             m.part = pm->part; m.part_ml = pm->part_ml; m.rows = n * H; m.H = H; m.kvp = l.kvp; m.C = pm->C; m.sink = l.sink; m.pos = p.pos; m.out = (bf16 *)b.ol;
@@ -636,9 +650,9 @@ bool wide_ready(Engine *e) {
     const int ldh = up(pm->plan->width, 64);
     pm->hg = dalloc<uint8_t>((size_t)PLAN_HEAD_ROWS * ldh * (e->f32 ? 4 : 2));
     pm->wlog = dalloc<float>((size_t)PLAN_HEAD_ROWS * pm->embed.rows);
-    size_t ex = 0;
-    for (auto &l : pm->L) ex = std::max(ex, (size_t)up(l.p.heads * (l.dimp + l.vdp), 32));
-    if (!e->f32) pm->ex = dalloc<bf16>((size_t)pm->seq_alloc * ex);
+    size_t kx = 0, vx = 0;
+    for (auto &l : pm->L) { kx = std::max(kx, (size_t)l.uk.rows); vx = std::max(vx, (size_t)l.uv.rows); }
+    if (!e->f32) { pm->kx = dalloc<bf16>((size_t)pm->seq_alloc * kx); pm->vx = dalloc<bf16>((size_t)pm->seq_alloc * vx); }
     return true;
 }
 

@@ -70,7 +70,7 @@ struct lg_plan *lg_plan_read(const struct gguf_context *g) {
         l->q_rank = iv[5][L]; l->kv_rank = iv[6][L]; l->kv_src = iv[7][L]; l->rot_dims = iv[8][L]; l->ff = iv[9][L];
         l->scale = scale[L]; l->rot_base = base[L];
         if (l->mixer != LG_MIX_LATENT) return bad(p, L, "unknown mixer"), NULL;
-        if (l->heads < 1 || l->dim < 1 || l->rot_dim < 0 || l->vdim < 1 || l->q_rank < 1 || l->kv_rank < 1 || l->ff < 0)
+        if (l->heads < 1 || l->dim < 1 || l->rot_dim < 0 || l->vdim < 1 || l->q_rank < 1 || l->kv_rank < 1 || l->ff < 0 || !(l->scale > 0))
             return bad(p, L, "a size is out of range"), NULL;
         if (l->rot_dims < 0 || l->rot_dims > l->rot_dim || l->rot_dims % 2) return bad(p, L, "the rotated dimensions are not an even part of the rotated key part"), NULL;
         if (l->kv_src < 0 || l->kv_src > L) return bad(p, L, "reads the cache of a layer that has not run"), NULL;

@@ -470,3 +470,116 @@ def cached(path_dir: str, name: str, writer, *args, **kw) -> str:
         writer(tmp, *args, **kw)
         os.replace(tmp, path)
     return path
+
+
+# ----------------------------------------------------------------------------
+# checkpoint folders (config.json + model.safetensors) of layer-plan models
+# ----------------------------------------------------------------------------
+
+@dataclass
+class LatentLayer:
+    """One layer of a Mubopel model: latent attention and a gated ReLU feed-forward (ff = 0: none)."""
+    heads: int = 4
+    dim: int = 32                     # unrotated query/key size per head
+    rot_dim: int = 16                 # rotated part, shared by the heads on the key side
+    vdim: int = 32
+    q_rank: int = 48
+    kv_rank: int = 64
+    ff: int = 160
+    kv_from: Optional[int] = None     # layer whose cached rows this one reads
+    base: float = 10000.0
+    scale: Optional[float] = None     # None: (dim + rot_dim) ** -0.5
+
+    def score_scale(self) -> float:
+        return self.scale if self.scale is not None else (self.dim + self.rot_dim) ** -0.5
+
+
+@dataclass
+class LatentShape:
+    width: int
+    vocab: int
+    layers: List[LatentLayer]
+    eps: float = 1e-5
+    residual_mult: float = 0.5
+
+    def config(self) -> dict:
+        out = []
+        for l in self.layers:
+            m = {"heads": l.heads, "dim": l.dim, "rot_dim": l.rot_dim, "vdim": l.vdim, "q_rank": l.q_rank, "kv_rank": l.kv_rank,
+                 "scale": l.score_scale(), "rot": {"base": l.base, "dims": l.rot_dim}}
+            if l.kv_from is not None:
+                m["kv_from"] = l.kv_from
+            out.append({"type": "latent_attention", "mixer": m, "mlp": {"kind": "dense", "ff": l.ff} if l.ff else None})
+        return {"architecture": "Mubopel", "width": self.width, "vocab": self.vocab, "norm": {"eps": self.eps},
+                "residual_mult": self.residual_mult, "layers": out}
+
+    def tensors(self) -> Dict[str, tuple]:
+        """name -> shape, in file order"""
+        W, t = self.width, {"embed": (self.vocab, self.width)}
+        for i, l in enumerate(self.layers):
+            p, H = f"l{i}.", l.heads
+            t[p + "norm1"] = t[p + "norm1b"] = (W,)
+            t[p + "mix.dq"] = (l.q_rank, W); t[p + "mix.dq.norm"] = (l.q_rank,); t[p + "mix.uq"] = (H * (l.dim + l.rot_dim), l.q_rank)
+            if l.kv_from is None:
+                t[p + "mix.dkv"] = (l.kv_rank + l.rot_dim, W); t[p + "mix.dkv.norm"] = (l.kv_rank,)
+            t[p + "mix.uk"] = (H * l.dim, l.kv_rank); t[p + "mix.uv"] = (H * l.vdim, l.kv_rank)
+            t[p + "mix.sink"] = (H,); t[p + "mix.g"] = (H * l.vdim, W); t[p + "mix.o"] = (W, H * l.vdim)
+            if l.ff:
+                t[p + "norm2"] = t[p + "norm2b"] = (W,)
+                t[p + "mlp.gate"] = t[p + "mlp.up"] = (l.ff, W); t[p + "mlp.down"] = (W, l.ff)
+        t["final.norm"] = (W,)
+        return t
+
+
+def to_bf16(x: np.ndarray) -> np.ndarray:
+    """float32 -> bf16 bit patterns (uint16), round to nearest even"""
+    u = np.ascontiguousarray(x, dtype=np.float32).view(np.uint32)
+    return ((u + 0x7FFF + ((u >> 16) & 1)) >> 16).astype(np.uint16)
+
+
+def from_bf16(b: np.ndarray) -> np.ndarray:
+    return (b.astype(np.uint32) << 16).view(np.float32)
+
+
+def random_weights(s: LatentShape, seed: int = 0, fast: bool = False) -> Dict[str, np.ndarray]:
+    """Seeded bf16 weights (bit patterns): matrices N(0, 1/k) so that projections keep their input's size, norm weights around 1,
+    sinks around 1, embeddings N(0, 1).  fast: big matrices repeat one random block (benchmarks, where only the sizes matter)."""
+    rng = np.random.default_rng(seed)
+    pool = to_bf16(rng.standard_normal(1 << 22)) if fast else None
+    w = {}
+    for name, shape in s.tensors().items():
+        n = int(np.prod(shape))
+        if name.endswith("sink"):
+            v = to_bf16(1.0 + 0.5 * rng.standard_normal(shape))
+        elif len(shape) == 1:
+            v = to_bf16(1.0 + 0.2 * rng.standard_normal(shape))
+        else:
+            std = 1.0 if name == "embed" else shape[1] ** -0.5
+            if fast and n > pool.size:
+                v = np.resize(to_bf16(from_bf16(pool) * np.float32(std)), n).reshape(shape)
+            else:
+                v = to_bf16(rng.standard_normal(shape, dtype=np.float32) * np.float32(std))
+        w[name] = v
+    return w
+
+
+def write_checkpoint(path: str, s: LatentShape, seed: int = 0, weights: Optional[Dict[str, np.ndarray]] = None, fast: bool = False) -> str:
+    """A checkpoint folder at `path`: config.json and model.safetensors (bf16)."""
+    import json
+    os.makedirs(path, exist_ok=True)
+    w = weights if weights is not None else random_weights(s, seed, fast)
+    head, off = {}, 0
+    for name, shape in s.tensors().items():
+        n = int(np.prod(shape)) * 2
+        head[name] = {"dtype": "BF16", "shape": list(shape), "data_offsets": [off, off + n]}
+        off += n
+    blob = json.dumps(head).encode()
+    with open(os.path.join(path, "model.safetensors"), "wb") as f:
+        f.write(struct.pack("<Q", len(blob)))
+        f.write(blob)
+        for name, shape in s.tensors().items():
+            assert w[name].shape == tuple(shape) and w[name].dtype == np.uint16, name
+            f.write(np.ascontiguousarray(w[name]).tobytes())
+    with open(os.path.join(path, "config.json"), "w") as f:
+        json.dump(s.config(), f, indent=1)
+    return path
