@@ -468,64 +468,94 @@ struct LgRowNormArgs {
     void *y; int ldy;                // rows of T (norm_w null: not written)
     float *yf; int ldyf;             // optional f32 copy
 };
-template <typename T, int EPT>
+// V consecutive elements as one load / store
+template <int V> struct alignas(V * 4) LgVec { float f[V]; };
+template <int V> __device__ __forceinline__ LgVec<V> vec_load(const float *p) {
+    LgVec<V> r;
+    if (V == 4) *(float4 *)r.f = *(const float4 *)p; else r.f[0] = *p;
+    return r;
+}
+template <int V> __device__ __forceinline__ void vec_store(float *p, const float *f) { if (V == 4) *(float4 *)p = *(const float4 *)f; else *p = *f; }
+template <int V> __device__ __forceinline__ void vec_store(bf16 *p, const float *f) {
+    if (V == 4) *(uint2 *)p = make_uint2(pack_bf16(f[0], f[1]), pack_bf16(f[2], f[V - 1])); else *p = __float2bfloat16_rn(f[0]);
+}
+// item i of a thread: elements (tid + i * blockDim) * V ..
+template <typename T, int IPT, int V>
 __global__ void __launch_bounds__(1024) lg_row_norm_kernel(LgRowNormArgs a) {
-    __shared__ float red[32];
+    __shared__ float red[4][32];
     pdl_launch();
-    float w1[EPT], w2[EPT], v[EPT];
-    const int tid = threadIdx.x, nt = blockDim.x;
-    #pragma unroll
-    for (int i = 0; i < EPT; i++) {              // the weights do not depend on earlier kernels
-        const int c = tid + i * nt;
-        w1[i] = a.add && c < a.n ? a.add_w[c] : 0.0f;
-        w2[i] = a.norm_w && c < a.n ? a.norm_w[c] : 0.0f;
-    }
+    LgVec<V> w1[IPT], w2[IPT], v[IPT], xv[IPT];
+    const int tid = threadIdx.x, nt = blockDim.x, lane = tid & 31, nw = (nt + 31) >> 5;
+    auto zero = [](LgVec<V> &x) {
+        #pragma unroll
+        for (int j = 0; j < V; j++) x.f[j] = 0.0f;
+    };
+    auto fetch = [&](LgVec<V> (&d)[IPT], const float *p) {
+        #pragma unroll
+        for (int i = 0; i < IPT; i++) { const int c = (tid + i * nt) * V; if (p && c < a.n) d[i] = vec_load<V>(p + c); else zero(d[i]); }
+    };
+    fetch(w1, a.add ? a.add_w : nullptr);          // the weights do not depend on earlier kernels
+    fetch(w2, a.norm_w);
     pdl_wait();
     float *x = a.x + (size_t)blockIdx.x * a.ldx;
     const float inv_n = 1.0f / (float)a.n;
-    float xv[EPT];
-    #pragma unroll
-    for (int i = 0; i < EPT; i++) { const int c = tid + i * nt; xv[i] = c < a.n ? x[c] : 0.0f; }
+    fetch(xv, x);
+    fetch(v, a.add ? a.add + (size_t)blockIdx.x * a.ld_add : x);
+    // sum over the row; each call has its own slots, so one barrier is enough
+    auto row_sum = [&](float s, int slot) {
+        s = warp_sum(s);
+        if (lane == 0) red[slot][tid >> 5] = s;
+        __syncthreads();
+        return warp_sum(lane < nw ? red[slot][lane] : 0.0f);
+    };
     // v <- (v - mean) / sqrt(mean of squared deviations + eps), in place
-    auto normalise = [&]() {
+    auto normalise = [&](int slot) {
         if (a.center) {
             float s = 0.0f;
             #pragma unroll
-            for (int i = 0; i < EPT; i++) s += v[i];
-            const float mean = block_sum(s, red) * inv_n;
+            for (int i = 0; i < IPT; i++)
+                #pragma unroll
+                for (int j = 0; j < V; j++) s += v[i].f[j];
+            const float mean = row_sum(s, slot) * inv_n;
             #pragma unroll
-            for (int i = 0; i < EPT; i++) v[i] = tid + i * nt < a.n ? v[i] - mean : 0.0f;
+            for (int i = 0; i < IPT; i++)
+                #pragma unroll
+                for (int j = 0; j < V; j++) v[i].f[j] = (tid + i * nt) * V < a.n ? v[i].f[j] - mean : 0.0f;
         }
         float ss = 0.0f;
         #pragma unroll
-        for (int i = 0; i < EPT; i++) ss += v[i] * v[i];
-        const float inv = 1.0f / sqrtf(block_sum(ss, red) * inv_n + a.eps);
+        for (int i = 0; i < IPT; i++)
+            #pragma unroll
+            for (int j = 0; j < V; j++) ss += v[i].f[j] * v[i].f[j];
+        const float inv = 1.0f / sqrtf(row_sum(ss, slot + 1) * inv_n + a.eps);
         #pragma unroll
-        for (int i = 0; i < EPT; i++) v[i] *= inv;
+        for (int i = 0; i < IPT; i++)
+            #pragma unroll
+            for (int j = 0; j < V; j++) v[i].f[j] *= inv;
     };
     if (a.add) {
-        const float *s = a.add + (size_t)blockIdx.x * a.ld_add;
+        normalise(0);
         #pragma unroll
-        for (int i = 0; i < EPT; i++) { const int c = tid + i * nt; v[i] = c < a.n ? s[c] : 0.0f; }
-        normalise();
-        #pragma unroll
-        for (int i = 0; i < EPT; i++) {
-            const int c = tid + i * nt;
-            xv[i] += a.mult * (v[i] * w1[i]);
-            if (c < a.n) x[c] = xv[i];
+        for (int i = 0; i < IPT; i++) {
+            const int c = (tid + i * nt) * V;
+            #pragma unroll
+            for (int j = 0; j < V; j++) xv[i].f[j] += a.mult * (v[i].f[j] * w1[i].f[j]);
+            if (c < a.n) vec_store<V>(x + c, xv[i].f);
         }
     }
     if (!a.norm_w) return;
     #pragma unroll
-    for (int i = 0; i < EPT; i++) v[i] = xv[i];
-    normalise();
+    for (int i = 0; i < IPT; i++) v[i] = xv[i];
+    normalise(2);
     #pragma unroll
-    for (int i = 0; i < EPT; i++) {
-        const int c = tid + i * nt;
+    for (int i = 0; i < IPT; i++) {
+        const int c = (tid + i * nt) * V;
         if (c >= a.n) continue;
-        const float y = v[i] * w2[i];
-        if (a.y) to_elem(y, ((T *)a.y)[(size_t)blockIdx.x * a.ldy + c]);
-        if (a.yf) a.yf[(size_t)blockIdx.x * a.ldyf + c] = y;
+        alignas(V * 4) float y[V];
+        #pragma unroll
+        for (int j = 0; j < V; j++) y[j] = v[i].f[j] * w2[i].f[j];
+        if (a.y) vec_store<V>((T *)a.y + (size_t)blockIdx.x * a.ldy + c, y);
+        if (a.yf) vec_store<V>(a.yf + (size_t)blockIdx.x * a.ldyf + c, y);
     }
 }
 

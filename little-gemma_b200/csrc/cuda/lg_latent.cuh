@@ -278,25 +278,37 @@ __global__ void __launch_bounds__(LG_LD_THREADS, 1) lg_latent_dec_attn_kernel(co
     if (tid < R && row0 + tid < a.rows) a.part_ml[(size_t)blockIdx.x * a.rows + row0 + tid] = make_float2(sM[tid], sL[tid]);
 }
 
-// Merge of the partials, in ascending split order, with the sink: latent output rows in bf16.  One CTA per query row; four
-// groups of threads take every fourth split.
+// Merge of the partials with the sink: latent output rows in bf16.  One CTA per query row; group g of its threads takes splits
+// g, g + GROUPS, ..., the first LG_LM_PRE of them loaded while the weights are still being made.
 struct LgLatentMergeArgs {
     const float *part; const float2 *part_ml; int rows, H, kvp, C;
     const float *sink; const int *pos;
     bf16 *out;                           // [rows][kvp]
 };
-#define LG_LM_GROUPS 4
-#define LG_LM_THREADS 512
+#define LG_LM_GROUPS 8
+#define LG_LM_THREADS 1024
+#define LG_LM_PRE 4
 #define LG_LM_MAXC 160
 __global__ void __launch_bounds__(LG_LM_THREADS) lg_latent_merge_kernel(LgLatentMergeArgs a) {
     extern __shared__ __align__(16) unsigned char lat_smem[];
     float *sum = (float *)lat_smem;                    // [groups][kvp]
     __shared__ float w[LG_LM_MAXC];
-    __shared__ float red[32];
-    pdl_launch(); pdl_wait();
+    __shared__ float s_inv;
+    pdl_launch();
     const int row = blockIdx.x, tid = threadIdx.x, lane = tid & 31;
     const int n = min(a.C, (*a.pos + row / a.H + LG_LD_S) / LG_LD_S);            // splits that hold keys of this row
     const float sink = a.sink[row % a.H] * LG_LOG2E;
+    constexpr int TPG = LG_LM_THREADS / LG_LM_GROUPS;
+    const int grp = tid / TPG, ti = tid % TPG;
+    pdl_wait();
+    const float *part = a.part + (size_t)row * a.kvp;
+    const size_t stride = (size_t)a.rows * a.kvp;
+    float4 v[LG_LM_PRE];
+    #pragma unroll
+    for (int j = 0; j < LG_LM_PRE; j++) {
+        const int i = grp + j * LG_LM_GROUPS;
+        v[j] = i < n && ti * 4 < a.kvp ? *(const float4 *)(part + i * stride + ti * 4) : make_float4(0, 0, 0, 0);
+    }
     if (tid < 32) {
         float m = sink;
         for (int i = lane; i < n; i += 32) m = fmaxf(m, a.part_ml[(size_t)i * a.rows + row].x);
@@ -309,27 +321,28 @@ __global__ void __launch_bounds__(LG_LM_THREADS) lg_latent_merge_kernel(LgLatent
             l += ml.y * e;
         }
         l = warp_sum(l);
-        if (lane == 0) red[0] = 1.0f / l;
+        if (lane == 0) s_inv = 1.0f / l;
     }
     __syncthreads();
-    const float inv = red[0];
-    const int grp = tid / (LG_LM_THREADS / LG_LM_GROUPS), ti = tid % (LG_LM_THREADS / LG_LM_GROUPS);
-    for (int c = ti * 4; c < a.kvp; c += LG_LM_THREADS / LG_LM_GROUPS * 4) {
+    for (int c = ti * 4; c < a.kvp; c += TPG * 4) {
         float4 o = make_float4(0, 0, 0, 0);
-        #pragma unroll 4
-        for (int i = grp; i < n; i += LG_LM_GROUPS) {
-            const float4 v = *(const float4 *)(a.part + ((size_t)i * a.rows + row) * a.kvp + c);
-            const float wi = w[i];
-            o.x = fmaf(wi, v.x, o.x); o.y = fmaf(wi, v.y, o.y); o.z = fmaf(wi, v.z, o.z); o.w = fmaf(wi, v.w, o.w);
+        auto add = [&](int i, const float4 &x) { const float wi = w[i]; o.x = fmaf(wi, x.x, o.x); o.y = fmaf(wi, x.y, o.y); o.z = fmaf(wi, x.z, o.z); o.w = fmaf(wi, x.w, o.w); };
+        int i0 = grp;
+        if (c == ti * 4) {
+            #pragma unroll
+            for (int j = 0; j < LG_LM_PRE; j++, i0 += LG_LM_GROUPS) if (i0 < n) add(i0, v[j]);
         }
+        #pragma unroll 4
+        for (int i = i0; i < n; i += LG_LM_GROUPS) add(i, *(const float4 *)(part + i * stride + c));
         *(float4 *)(sum + (size_t)grp * a.kvp + c) = o;
     }
     __syncthreads();
+    const float inv = s_inv;
     for (int c = tid; c < a.kvp; c += LG_LM_THREADS) {
-        float v = 0.0f;
+        float o = 0.0f;
         #pragma unroll
-        for (int i = 0; i < LG_LM_GROUPS; i++) v += sum[(size_t)i * a.kvp + c];
-        a.out[(size_t)row * a.kvp + c] = __float2bfloat16_rn(v * inv);
+        for (int i = 0; i < LG_LM_GROUPS; i++) o += sum[(size_t)i * a.kvp + c];
+        a.out[(size_t)row * a.kvp + c] = __float2bfloat16_rn(o * inv);
     }
 }
 

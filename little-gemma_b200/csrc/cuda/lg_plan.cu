@@ -356,7 +356,7 @@ void plan_bind(Engine *e, const struct kvcache *kv) {
     int groups = 1;
     size_t rows = 0;
     for (auto &l : pm->L) {
-        if (l.rt) groups = std::max(groups, (l.p.heads + 16 * l.rt - 1) / (16 * l.rt));
+        if (l.rt) groups = std::max(groups, (l.p.heads + 15) / 16);
         rows = std::max(rows, (size_t)l.p.heads * LG_MAXM * l.kvp);
     }
     pm->C = std::max(1, std::min({e->sm_count / groups, (kv->max_seq + LG_LD_S - 1) / LG_LD_S, LG_LM_MAXC}));
@@ -426,14 +426,17 @@ void launch_f32(Engine *e, const DMat &W, const void *x, int ldx, int n, void *o
 }
 
 void launch_row_norm(Engine *e, int n, LgRowNormArgs a) {
-    // few rows: as many threads as the row has elements, for latency; many rows: fewer threads per row, for throughput
-    const int threads = std::min(1024, std::max(128, up(n > 16 ? a.n / 8 : a.n, 32)));
-    const int ept = (a.n + threads - 1) / threads;
+    // a few elements per thread: barriers among few warps for one row, whole cache lines per warp for many
+    const int vec = a.n % 4 == 0 && a.ldx % 4 == 0 && a.ldy % 4 == 0 && a.ld_add % 4 == 0 ? 4 : 1, items = a.n / vec;
+    const int threads = std::min(1024, std::max(64, up((items + 1) / 2, 32)));
+    const int ipt = (items + threads - 1) / threads;
     auto go = [&](auto kernel) { launch_k(e, kernel, dim3(n), dim3(threads), 0, a); };
     if (e->f32) {
-        if (ept <= 4) go(lg_row_norm_kernel<float, 4>); else if (ept <= 8) go(lg_row_norm_kernel<float, 8>); else go(lg_row_norm_kernel<float, 16>);
+        if (vec == 4) { if (ipt <= 2) go(lg_row_norm_kernel<float, 2, 4>); else go(lg_row_norm_kernel<float, 4, 4>); }
+        else go(lg_row_norm_kernel<float, 16, 1>);
     } else {
-        if (ept <= 4) go(lg_row_norm_kernel<bf16, 4>); else if (ept <= 8) go(lg_row_norm_kernel<bf16, 8>); else go(lg_row_norm_kernel<bf16, 16>);
+        if (vec == 4) { if (ipt <= 2) go(lg_row_norm_kernel<bf16, 2, 4>); else go(lg_row_norm_kernel<bf16, 4, 4>); }
+        else go(lg_row_norm_kernel<bf16, 16, 1>);
     }
 }
 
@@ -525,7 +528,7 @@ void latent_attention(Engine *e, const struct kvcache *kv, PlanLayer &l, const P
             a.err = e->err;
             a.q = (const bf16 *)b.qa; a.ldc = l.ldc; a.kvp = l.kvp; a.rows = n * H; a.H = H;
             a.scale = l.p.scale; a.pos = p.pos; a.part = pm->part; a.part_ml = pm->part_ml;
-            const int rt = n * H > 16 ? l.rt : 1;
+            const int rt = n * H > 2 * 16 * 2 ? l.rt : 1;        // few rows: a row tile per CTA; the arithmetic of a row is the same
             const dim3 grid(pm->C, (n * H + 16 * rt - 1) / (16 * rt)), block(LG_LD_THREADS);
             const size_t sm = lg_latent_dec_smem(rt, l.ldc);
             if (rt == 2) {
