@@ -165,6 +165,22 @@ int  lg_flash_decode_host(const float *q, const float *k, const float *v, int M,
 int  lg_flash_decode_cluster_host(const float *q, const float *k, const float *v, int M, int H, int Hkv, int hd,
                                   int seq, int window, int pos, float *out);
 
+/* Dense matrices and latent attention (models described by a layer plan); f32 != 0 runs the 32-bit kernels, otherwise operands
+ * are rounded to bf16.  Return 0, -1 on bad arguments, -2 where the kernel asked for does not hold the sizes.
+ * out[tok][m] = w x[tok]; with w_up (m a multiple of 8): relu(w x) * (w_up x).  n <= 8 rows take the decode kernel. */
+int  lg_dense_matmul_host(const float *w, const float *w_up, int m, int k, const float *x, int n, int f32, float *out);
+/* x += mult * norm(add) * add_w (add may be NULL), y = norm(x) * norm_w; center != 0 takes the mean off first. */
+int  lg_row_norm_host(float *x, int rows, int n, const float *add, const float *add_w, float mult, const float *norm_w, float eps,
+                      int center, int f32, float *y);
+/* Attention of absorbed queries [n][H][kv_rank + rot_dim] at positions pos.. over latent rows [pos + n][kv_rank + rot_dim], with a
+ * sink per head: latent outputs [n][H][kv_rank].  form 0: split kernel + merge (n <= 8), 1: one (token, head) per CTA. */
+int  lg_latent_attn_host(const float *q, const float *cache, const float *sink, int n, int H, int kv_rank, int rot_dim, int pos, int max_seq,
+                         float scale, int form, int f32, float *out);
+/* Attention of a prompt block: q [n][H][dim + rot_dim], k [pos + n][H][dim], k_rot [pos + n][rot_dim], v [pos + n][H][vdim],
+ * gate [n][H][vdim]; out [n][H][vdim] = sigmoid(gate) * attention. */
+int  lg_latent_prompt_attn_host(const float *q, const float *k, const float *k_rot, const float *v, const float *gate, const float *sink,
+                                int n, int H, int dim, int rot_dim, int vdim, int pos, float scale, float *out);
+
 /* Split-KV flash-decode for callers that cannot allocate device memory (a captured stream, a
  * serving loop whose memory was fixed at start-up, a process whose allocator owns the device).
  * Same kernel as lg_flash_decode_host, but every pointer is a DEVICE pointer supplied by the

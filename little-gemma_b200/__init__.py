@@ -32,6 +32,7 @@ ABI_SYMBOLS = [
     "lg_bench_matmul_pass", "lg_bench_prefill_pass", "lg_set_attn_deep", "lg_flash_decode_noalloc",
     "lg_debug_bounded_wait", "lg_debug_stamps", "lg_debug_clear_stamps", "lg_matmul_resid_host",
     "lg_dequant_host", "lg_gemv_host", "lg_flash_decode_host", "lg_flash_decode_cluster_host", "lg_prefill_matmul_host",
+    "lg_dense_matmul_host", "lg_row_norm_host", "lg_latent_attn_host", "lg_latent_prompt_attn_host",
 ]
 
 _lib = None
@@ -107,6 +108,13 @@ def load() -> C.CDLL:
     L.lgs_host_syncs.argtypes = [C.c_void_p]; L.lgs_host_syncs.restype = C.c_longlong
     L.lg_set_round_width.argtypes = [C.c_int]; L.lg_set_round_width.restype = None
     L.lg_set_replay_origin.argtypes = [C.c_void_p, C.c_int, C.c_int]; L.lg_set_replay_origin.restype = None
+    f, i, vp, fl = _f32p, C.c_int, C.c_void_p, C.c_float
+    for name, args in (("lg_dense_matmul_host", [f, vp, i, i, f, i, i, f]),
+                       ("lg_row_norm_host", [f, i, i, vp, vp, fl, f, fl, i, i, f]),
+                       ("lg_latent_attn_host", [f, f, f, i, i, i, i, i, i, fl, i, i, f]),
+                       ("lg_latent_prompt_attn_host", [f, f, f, f, f, f, i, i, i, i, i, i, fl, f])):
+        getattr(L, name).argtypes = args
+        getattr(L, name).restype = i
     _lib = L
     return L
 
@@ -170,6 +178,57 @@ def prefill_matmul(ggml_type: int, raw: np.ndarray, m: int, k: int, x: np.ndarra
     if rc:
         raise ValueError(f"lg_prefill_matmul_host failed ({rc})")
     return y
+
+
+def _f32(a) -> np.ndarray:
+    return np.ascontiguousarray(a, dtype=np.float32)
+
+
+def _ptr(a):
+    return None if a is None else a.ctypes.data_as(C.c_void_p)
+
+
+def _ok(rc: int, what: str) -> None:
+    if rc:
+        raise ValueError(f"{what} failed ({rc})")
+
+
+def dense_matmul(w, x, w_up=None, f32: bool = False) -> np.ndarray:
+    """y[tok] = w x[tok] through the dense matmul kernels (up to 8 rows: the decode kernel, more: the tcgen05 one, f32: the
+    32-bit one); with w_up, relu(w x) * (w_up x) through their gated epilogues."""
+    w, x, u = _f32(w), _f32(x), None if w_up is None else _f32(w_up)
+    y = np.empty((x.shape[0], w.shape[0]), dtype=np.float32)
+    _ok(load().lg_dense_matmul_host(w.reshape(-1), _ptr(u), w.shape[0], w.shape[1], x.reshape(-1), x.shape[0], int(f32), y.reshape(-1)), "dense_matmul")
+    return y
+
+
+def row_norm(x, norm_w, eps: float, add=None, add_w=None, mult: float = 1.0, center: bool = True, f32: bool = False):
+    """(x + mult norm(add) add_w, norm of that times norm_w) through the residual / norm kernel."""
+    x, nw = np.array(x, dtype=np.float32, order="C", copy=True), _f32(norm_w)
+    a, aw = (None, None) if add is None else (_f32(add), _f32(add_w))
+    y = np.empty_like(x)
+    _ok(load().lg_row_norm_host(x.reshape(-1), x.shape[0], x.shape[1], _ptr(a), _ptr(aw), mult, nw, eps, int(center), int(f32), y.reshape(-1)), "row_norm")
+    return x, y
+
+
+def latent_attn(q, cache, sink, kv_rank: int, pos: int, scale: float, max_seq: int = 0, rows_form: bool = False, f32: bool = False) -> np.ndarray:
+    """Absorbed queries q [n, H, kv_rank + rot] at positions pos.. over latent rows cache [pos + n, kv_rank + rot]: [n, H, kv_rank]."""
+    q, cache, sink = _f32(q), _f32(cache), _f32(sink)
+    n, H, d = q.shape
+    out = np.empty((n, H, kv_rank), dtype=np.float32)
+    _ok(load().lg_latent_attn_host(q.reshape(-1), cache.reshape(-1), sink, n, H, kv_rank, d - kv_rank, pos, max(max_seq, pos + n), scale,
+                                   int(rows_form), int(f32), out.reshape(-1)), "latent_attn")
+    return out
+
+
+def latent_prompt_attn(q, k, k_rot, v, gate, sink, pos: int, scale: float) -> np.ndarray:
+    """A prompt block's attention: q [n, H, dim + rot], k [pos + n, H, dim], k_rot [pos + n, rot], v [pos + n, H, vdim]: [n, H, vdim]."""
+    q, k, k_rot, v, gate, sink = map(_f32, (q, k, k_rot, v, gate, sink))
+    n, H, _ = q.shape
+    out = np.empty((n, H, v.shape[2]), dtype=np.float32)
+    _ok(load().lg_latent_prompt_attn_host(q.reshape(-1), k.reshape(-1), k_rot.reshape(-1), v.reshape(-1), gate.reshape(-1), sink, n, H, k.shape[2],
+                                          k_rot.shape[1], v.shape[2], pos, scale, out.reshape(-1)), "latent_prompt_attn")
+    return out
 
 
 def set_attn_deep(min_seq: int = 4096, force_g: int = 0) -> None:

@@ -58,7 +58,7 @@ struct PlanModel {
     bf16 *kx = nullptr, *vx = nullptr;                       // one layer's expanded keys [position][H dimp] and values [H vdp][position]
     int *want = nullptr; void *hg = nullptr; float *wlog = nullptr;
     float *logits = nullptr;                                  // 32-bit: rows of a head without F_LOGITS
-    std::map<std::tuple<const void *, int, int, int>, CUtensorMap> maps;
+    std::map<std::tuple<const void *, int, int, int, int>, CUtensorMap> maps;
 };
 
 // ------------------------------------------------------------------------------------------
@@ -346,20 +346,19 @@ int plan_kv_init(struct kvcache *kv, const struct model *m, bool f32) {
     return 0;
 }
 
+int latent_splits(const Engine *e, int heads, int max_seq);
 void plan_bind(Engine *e, const struct kvcache *kv) {
     PlanModel *pm = e->plan;
     plan_unbind(pm);
     pm->max_seq = kv->max_seq; pm->seq_alloc = cache_rows(kv->max_seq);
     if (e->f32) return;
-    // Splits of the decode attention: as many CTAs as there are SMs for the row groups of one token, a property of the cache
-    // length and the head counts alone (never of the block's width or the position).
-    int groups = 1;
     size_t rows = 0;
+    int most = 1;
     for (auto &l : pm->L) {
-        if (l.rt) groups = std::max(groups, (l.p.heads + 15) / 16);
+        most = std::max(most, l.p.heads);
         rows = std::max(rows, (size_t)l.p.heads * LG_MAXM * l.kvp);
     }
-    pm->C = std::max(1, std::min({e->sm_count / groups, (kv->max_seq + LG_LD_S - 1) / LG_LD_S, LG_LM_MAXC}));
+    pm->C = latent_splits(e, most, kv->max_seq);
     size_t heads = 0;
     for (auto &l : pm->L) heads = std::max(heads, (size_t)l.p.heads);
     pm->part = dalloc<float>(rows * pm->C);
@@ -378,8 +377,8 @@ int gemv_ks(const Engine *e, const DMat &W) {
     return ks;
 }
 template <int EPI, bool RMSX>
-int launch_dn_gemv(Engine *e, const DMat &W, LgDnGemvArgs a, int cap_ctas = 1 << 20) {
-    a.w = (const bf16 *)W.w; a.ldk = W.ldk; a.n_tiles = W.rows / 16;
+int launch_dn_gemv(Engine *e, const DMat &W, LgDnGemvArgs a, int groups = 0, int cap_ctas = 1 << 20) {
+    a.w = (const bf16 *)W.w; a.ldk = W.ldk; a.n_tiles = groups ? groups * a.tiles_per_group : W.rows / 16;   // (rows behind the last group are padding)
     const int ks = gemv_ks(e, W), tpc = 8 / ks;
     a.n_main = std::min((a.n_tiles + tpc - 1) / tpc, cap_ctas);
     const dim3 grid(a.n_main + (a.job ? a.M : 0));
@@ -392,9 +391,9 @@ int launch_dn_gemv(Engine *e, const DMat &W, LgDnGemvArgs a, int cap_ctas = 1 <<
     }
     return a.n_main;
 }
-// descriptor of a bf16 activation buffer [rows][ld], of which k columns count; made once per buffer, width and box
+// descriptor of a bf16 activation buffer [rows][ld], of which k columns count; made once per buffer, shape and box
 const CUtensorMap &buf_map(PlanModel *pm, const void *x, int k, int ld, int rows, int box_r) {
-    const auto key = std::make_tuple(x, k, ld, box_r);
+    const auto key = std::make_tuple(x, k, ld, rows, box_r);
     auto it = pm->maps.find(key);
     if (it == pm->maps.end())
         it = pm->maps.emplace(key, tiled_map(x, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, std::min(k, ld), rows, (long long)ld * 2, DN_GEMM_BK, box_r)).first;
@@ -457,6 +456,52 @@ void plan_embed_rows(Engine *e, const int *toks, int n, float *x) {
     else launch_k(e, lg_dn_embed_rows<bf16>, dim3(n), dim3(256), 0, (const bf16 *)E.w, E.ldk, e->plan->plan->vocab, toks, x, W);
 }
 
+// Splits of the decode attention: as many CTAs as there are SMs for the row tiles of one token, a property of the cache length
+// and the head count alone (never of the block's width or the position).
+int latent_splits(const Engine *e, int heads, int max_seq) {
+    return std::max(1, std::min({e->sm_count / ((heads + 15) / 16), (max_seq + LG_LD_S - 1) / LG_LD_S, LG_LM_MAXC}));
+}
+void launch_latent_rows(Engine *e, const PlanLayer &l, int n, const LgLatentRowsArgs &a) {
+    const size_t sm = (size_t)(l.ldc + l.kvp + 128) * 4;
+    if (e->f32) launch_k(e, lg_latent_attn_rows_kernel<float>, dim3(l.p.heads, n), dim3(128), sm, a);
+    else launch_k(e, lg_latent_attn_rows_kernel<bf16>, dim3(l.p.heads, n), dim3(128), sm, a);
+}
+// absorbed queries q [n * H][ldc] over the cache -> latent rows out [n * H][kvp]
+void launch_latent_dec(Engine *e, const PlanLayer &l, int n, const void *q, const void *cache, const int *pos, void *out) {
+    PlanModel *pm = e->plan;
+    const int H = l.p.heads;
+    LgLatentDecArgs a{};
+    const CUtensorMap &cm = buf_map(pm, cache, l.ldc, l.ldc, pm->seq_alloc, LG_LD_S);
+    a.q = (const bf16 *)q; a.ldc = l.ldc; a.kvp = l.kvp; a.rows = n * H; a.H = H;
+    a.scale = l.p.scale; a.pos = pos; a.part = pm->part; a.part_ml = pm->part_ml; a.err = e->err;
+    const int rt = n * H > 64 ? l.rt : 1;                      // few rows: a row tile per CTA; the arithmetic of a row is the same
+    const dim3 grid(pm->C, (n * H + 16 * rt - 1) / (16 * rt)), block(LG_LD_THREADS);
+    const size_t sm = lg_latent_dec_smem(rt, l.ldc);
+    if (rt == 2) {
+        if (l.kvp <= 128) launch_k(e, lg_latent_dec_attn_kernel<2, 2>, grid, block, sm, cm, a);
+        else if (l.kvp <= 256) launch_k(e, lg_latent_dec_attn_kernel<2, 4>, grid, block, sm, cm, a);
+        else launch_k(e, lg_latent_dec_attn_kernel<2, 8>, grid, block, sm, cm, a);
+    } else {
+        if (l.kvp <= 128) launch_k(e, lg_latent_dec_attn_kernel<1, 2>, grid, block, sm, cm, a);
+        else if (l.kvp <= 256) launch_k(e, lg_latent_dec_attn_kernel<1, 4>, grid, block, sm, cm, a);
+        else launch_k(e, lg_latent_dec_attn_kernel<1, 8>, grid, block, sm, cm, a);
+    }
+    LgLatentMergeArgs m{};
+    m.part = pm->part; m.part_ml = pm->part_ml; m.rows = n * H; m.H = H; m.kvp = l.kvp; m.C = pm->C; m.sink = l.sink; m.pos = pos; m.out = (bf16 *)out;
+    launch_k(e, lg_latent_merge_kernel, dim3(n * H), dim3(LG_LM_THREADS), (size_t)LG_LM_GROUPS * l.kvp * 4, m);
+}
+// rotated queries q [n][ldq] over the expanded keys and values of the block's context -> gated rows out [n][ldo]
+void launch_latent_prompt(Engine *e, const PlanLayer &l, int n, int q_rows, const void *q, int ldq, const void *cache, const float *gate, int ldg,
+                          const int *pos, void *out, int ldo) {
+    PlanModel *pm = e->plan;
+    LgLatentPfArgs a{};
+    a.H = l.p.heads; a.dimp = l.dimp; a.rotp = l.rotp; a.vdp = l.vdp; a.n = n; a.rot_at = l.kvp; a.scale = l.p.scale; a.sink = l.sink;
+    a.gate = gate; a.ldg = ldg; a.pos = pos; a.out = (bf16 *)out; a.ldo = ldo; a.err = e->err;
+    launch_k(e, lg_latent_pf_attn_kernel, dim3((n + LG_LP_Q - 1) / LG_LP_Q, l.p.heads), dim3(LG_LP_THREADS), lg_latent_pf_smem(l.dimp, l.rotp, l.vdp),
+             buf_map(pm, q, ldq, ldq, q_rows, LG_LP_Q), buf_map(pm, pm->kx, l.uk.rows, l.uk.rows, pm->seq_alloc, LG_LP_S),
+             buf_map(pm, cache, l.ldc, l.ldc, pm->seq_alloc, LG_LP_S), buf_map(pm, pm->vx, pm->seq_alloc, pm->seq_alloc, l.uv.rows, l.vdp), a);
+}
+
 void latent_attention(Engine *e, const struct kvcache *kv, PlanLayer &l, const Pass &p, int only) {
     PlanModel *pm = e->plan;
     PlanBuf &b = *p.b;
@@ -476,14 +521,13 @@ void latent_attention(Engine *e, const struct kvcache *kv, PlanLayer &l, const P
     pa.cq = b.cq; pa.ldcq = l.uq.ldk; pa.owns = l.owns; pa.cr = cr;
     LgLatentRowsArgs ra{};
     ra.q = b.qa; ra.cache = cache; ra.ldc = l.ldc; ra.kvp = l.kvp; ra.H = H; ra.sink = l.sink; ra.scale = l.p.scale; ra.pos = p.pos; ra.out = b.ol;
-    const size_t rows_sm = (size_t)(l.ldc + l.kvp + 128) * 4;
 
     if (e->f32) {
         launch_k(e, lg_latent_prep_kernel<float>, dim3(n), dim3(128), 0, pa);
         launch_f32(e, l.uq, b.cq, l.uq.ldk, n, b.q, ldq);
         launch_f32(e, l.ukT, b.q, ldq, n, b.qa, H * l.ldc, H, l.kvp, qh, l.ldc);
         launch_k(e, lg_latent_rot_q_kernel<float>, dim3(1, n), dim3(128), 0, rq);
-        launch_k(e, lg_latent_attn_rows_kernel<float>, dim3(H, n), dim3(128), rows_sm, ra);
+        launch_latent_rows(e, l, n, ra);
         launch_f32(e, l.uv, b.ol, H * l.kvp, n, b.at, ld_at, H, l.vdp, l.kvp, l.vdp);
         launch_k(e, lg_dn_gate_rows, dim3((H * l.vdp + 255) / 256, n), dim3(256), 0, (float *)b.at, ld_at, gate, l.in.rows, H * l.vdp);
         return;
@@ -501,13 +545,7 @@ void latent_attention(Engine *e, const struct kvcache *kv, PlanLayer &l, const P
             launch_gemm_maps<DN_G_BF16>(e, l.uv.map[0], H * l.vdp, buf_map(pm, cache, l.p.kv_rank, l.ldc, pm->seq_alloc, 128),
                                         buf_map(pm, cache, l.p.kv_rank, l.ldc, pm->seq_alloc, 256), up(keys, 32), l.uv.ldk / DN_GEMM_BK, pm->vx, pm->seq_alloc, false);
         }
-        if (!(only & C_ATTN)) return;
-        LgLatentPfArgs a{};
-        a.H = H; a.dimp = l.dimp; a.rotp = l.rotp; a.vdp = l.vdp; a.n = n; a.rot_at = l.kvp; a.scale = l.p.scale; a.sink = l.sink;
-        a.gate = gate; a.ldg = l.in.rows; a.pos = p.pos; a.out = (bf16 *)b.at; a.ldo = ld_at; a.err = e->err;
-        launch_k(e, lg_latent_pf_attn_kernel, dim3((n + LG_LP_Q - 1) / LG_LP_Q, H), dim3(LG_LP_THREADS), lg_latent_pf_smem(l.dimp, l.rotp, l.vdp),
-                 buf_map(pm, b.q, ldq, ldq, b.cap, LG_LP_Q), buf_map(pm, pm->kx, l.uk.rows, l.uk.rows, pm->seq_alloc, LG_LP_S),
-                 buf_map(pm, cache, l.ldc, l.ldc, pm->seq_alloc, LG_LP_S), buf_map(pm, pm->vx, pm->seq_alloc, pm->seq_alloc, l.uv.rows, l.vdp), a);
+        if (only & C_ATTN) launch_latent_prompt(e, l, n, b.cap, b.q, ldq, cache, gate, l.in.rows, p.pos, b.at, ld_at);
         return;
     }
     if (only & C_QKV) {
@@ -518,38 +556,17 @@ void latent_attention(Engine *e, const struct kvcache *kv, PlanLayer &l, const P
         LgDnGemvArgs k{};                          // per head onto the latent; beside it, the rotated parts
         k.x = (const bf16 *)b.q; k.ldx = ldq; k.tiles_per_group = l.kvp / 16; k.x_group = qh; k.out_group = l.ldc; k.M = n;
         k.outh = (bf16 *)b.qa; k.ldoh = H * l.ldc; k.job = DN_JOB_ROT_Q; k.rq = rq;
-        launch_dn_gemv<DN_STORE, false>(e, l.ukT, k);
+        launch_dn_gemv<DN_STORE, false>(e, l.ukT, k, H);
     }
     if (only & C_ATTN) {
-        if (!l.rt) launch_k(e, lg_latent_attn_rows_kernel<bf16>, dim3(H, n), dim3(128), rows_sm, ra);
-        else {
-            LgLatentDecArgs a{};
-            const CUtensorMap &cm = buf_map(pm, cache, l.ldc, l.ldc, pm->seq_alloc, LG_LD_S);
-            a.err = e->err;
-            a.q = (const bf16 *)b.qa; a.ldc = l.ldc; a.kvp = l.kvp; a.rows = n * H; a.H = H;
-            a.scale = l.p.scale; a.pos = p.pos; a.part = pm->part; a.part_ml = pm->part_ml;
-            const int rt = n * H > 2 * 16 * 2 ? l.rt : 1;        // few rows: a row tile per CTA; the arithmetic of a row is the same
-            const dim3 grid(pm->C, (n * H + 16 * rt - 1) / (16 * rt)), block(LG_LD_THREADS);
-            const size_t sm = lg_latent_dec_smem(rt, l.ldc);
-            if (rt == 2) {
-                if (l.kvp <= 128) launch_k(e, lg_latent_dec_attn_kernel<2, 2>, grid, block, sm, cm, a);
-                else if (l.kvp <= 256) launch_k(e, lg_latent_dec_attn_kernel<2, 4>, grid, block, sm, cm, a);
-                else launch_k(e, lg_latent_dec_attn_kernel<2, 8>, grid, block, sm, cm, a);
-            } else {
-                if (l.kvp <= 128) launch_k(e, lg_latent_dec_attn_kernel<1, 2>, grid, block, sm, cm, a);
-                else if (l.kvp <= 256) launch_k(e, lg_latent_dec_attn_kernel<1, 4>, grid, block, sm, cm, a);
-                else launch_k(e, lg_latent_dec_attn_kernel<1, 8>, grid, block, sm, cm, a);
-            }
-            LgLatentMergeArgs m{};
-            m.part = pm->part; m.part_ml = pm->part_ml; m.rows = n * H; m.H = H; m.kvp = l.kvp; m.C = pm->C; m.sink = l.sink; m.pos = p.pos; m.out = (bf16 *)b.ol;
-            launch_k(e, lg_latent_merge_kernel, dim3(n * H), dim3(LG_LM_THREADS), (size_t)LG_LM_GROUPS * l.kvp * 4, m);
-        }
+        if (l.rt) launch_latent_dec(e, l, n, b.qa, cache, p.pos, b.ol);
+        else launch_latent_rows(e, l, n, ra);
     }
     if (only & C_O) {
         LgDnGemvArgs v{};                          // latent outputs -> gated head values
         v.x = (const bf16 *)b.ol; v.ldx = H * l.kvp; v.tiles_per_group = l.vdp / 16; v.x_group = l.kvp; v.out_group = l.vdp; v.M = n;
         v.outh = (bf16 *)b.at; v.ldoh = ld_at; v.gate = gate; v.ld_gate = l.in.rows;
-        launch_dn_gemv<DN_SIGMOID_GATE, false>(e, l.uv, v);
+        launch_dn_gemv<DN_SIGMOID_GATE, false>(e, l.uv, v, H);
     }
 }
 
@@ -638,7 +655,7 @@ int plan_forward(Engine *e, const struct kvcache *kv, int M, int flags, int only
     LgDnGemvArgs a{};
     a.x = (const bf16 *)pm->nb.h; a.ldx = ldh; a.M = M; a.rows = pm->plan->vocab; a.out = lg; a.ldo = e->head.ldo;
     a.amax_val = e->amax_val; a.amax_idx = e->amax_idx;
-    return launch_dn_gemv<DN_HEAD, false>(e, pm->embed, a, e->head_ctas);
+    return launch_dn_gemv<DN_HEAD, false>(e, pm->embed, a, 0, e->head_ctas);
 }
 
 // buffers of the wide pass, at its first use
@@ -708,3 +725,195 @@ const LgFamily plan_family = {"layer plan", plan_load, plan_release, plan_kv_ini
 }  // namespace lg
 
 extern "C" const lg::LgFamily *lg_family_for(const struct gguf_context *ctx) { return lg_plan_present(ctx) ? &lg::plan_family : nullptr; }
+
+// ==========================================================================================
+// kernel-level entry points of the parity tests (host buffers in, host buffers out)
+// ==========================================================================================
+namespace lg {
+
+// an engine without a model: stream, status word, launch settings, and the descriptor store of the launch helpers
+struct Scratch {
+    Engine e;
+    PlanModel pm;
+    std::vector<void *> mem;
+    explicit Scratch(bool f32) {
+        plan_attributes();
+        int dev = 0;
+        LG_CHECK(cudaGetDevice(&dev));
+        LG_CHECK(cudaDeviceGetAttribute(&e.sm_count, cudaDevAttrMultiProcessorCount, dev));
+        LG_CHECK(cudaStreamCreateWithFlags(&e.stream, cudaStreamNonBlocking));
+        e.err = dalloc<int>(1); mem.push_back(e.err);
+        e.f32 = f32; e.plan = &pm;
+    }
+    ~Scratch() {
+        cudaStreamSynchronize(e.stream);
+        for (void *p : mem) cudaFree(p);
+        cudaStreamDestroy(e.stream);
+    }
+    size_t es() const { return e.f32 ? 4 : 2; }
+    // rows x n f32 values as [rows_alloc][ld] elements of the mode's type (plus slack), zero elsewhere
+    void *rows(const float *src, int rows, int n, int rows_alloc, int ld) {
+        std::vector<uint8_t> h(((size_t)rows_alloc * ld + 256) * es(), 0);
+        for (int r = 0; r < rows; r++)
+            for (int i = 0; i < n; i++) {
+                const float v = src[(size_t)r * n + i];
+                if (e.f32) memcpy(&h[((size_t)r * ld + i) * 4], &v, 4);
+                else { const uint16_t b = bf16_bits(v); memcpy(&h[((size_t)r * ld + i) * 2], &b, 2); }
+            }
+        void *d = dalloc<uint8_t>(h.size());
+        h2d_sync(d, h.data(), h.size());
+        mem.push_back(d);
+        return d;
+    }
+    template <typename T> T *put(const T *src, size_t n) {
+        T *d = dalloc<T>(n);
+        if (src) h2d_sync(d, src, n * sizeof(T));
+        mem.push_back(d);
+        return d;
+    }
+    // n elements of a device buffer, as f32
+    std::vector<float> get(const void *d, size_t n, bool f32) {
+        std::vector<float> out(n);
+        check_err(&e);
+        if (f32) { LG_CHECK(cudaMemcpy(out.data(), d, n * 4, cudaMemcpyDeviceToHost)); return out; }
+        std::vector<uint16_t> b(n);
+        LG_CHECK(cudaMemcpy(b.data(), d, n * 2, cudaMemcpyDeviceToHost));
+        for (size_t i = 0; i < n; i++) { const uint32_t u = (uint32_t)b[i] << 16; memcpy(&out[i], &u, 4); }
+        return out;
+    }
+};
+
+}  // namespace lg
+
+using namespace lg;
+
+extern "C" int lg_dense_matmul_host(const float *w, const float *w_up, int m, int k, const float *x, int n, int f32, float *out) {
+    if (m < 1 || k < 1 || n < 1 || (w_up && m % 8)) return -1;
+    Scratch s(f32 != 0);
+    Engine *e = &s.e;
+    MatBuild b(e, w_up ? 2 * up(m, 16) : m, k);
+    for (int r = 0; r < m; r++)
+        for (int i = 0; i < k; i++) {
+            b.put((size_t)(w_up ? r / 8 * 16 + r % 8 : r) * b.ldk + i, w[(size_t)r * k + i]);
+            if (w_up) b.put((size_t)(r / 8 * 16 + 8 + r % 8) * b.ldk + i, w_up[(size_t)r * k + i]);
+        }
+    DMat W = b.upload(e);
+    s.mem.push_back(W.w);
+    const int xr = up(n, 128);
+    PlanLayer l;
+    l.gu = W; l.ffp = up(m, 16); l.down.ldk = up(l.ffp, 64);
+    s.pm.nb.cap = xr;
+    s.pm.nb.gu = s.put<float>(nullptr, (size_t)xr * W.rows);
+    s.pm.nb.act = s.put<uint8_t>(nullptr, ((size_t)xr * l.down.ldk + 64) * s.es());
+    float *o = s.put<float>(nullptr, (size_t)xr * W.rows);
+    void *dx = s.rows(x, n, k, xr, W.ldk);
+    Pass p{&s.pm.nb, n, n > LG_MAXM, nullptr, nullptr, 0};
+    if (w_up) gated(e, l, dx, W.ldk, p); else project(e, W, dx, W.ldk, p, o);
+    const int ld = w_up ? l.down.ldk : W.rows;
+    const std::vector<float> r = s.get(w_up ? s.pm.nb.act : (void *)o, (size_t)n * ld, !w_up || f32);
+    for (int i = 0; i < n; i++) memcpy(out + (size_t)i * m, &r[(size_t)i * ld], (size_t)m * 4);
+    s.pm.nb = PlanBuf();
+    return 0;
+}
+
+extern "C" int lg_row_norm_host(float *x, int rows, int n, const float *add, const float *add_w, float mult, const float *norm_w, float eps,
+                                int center, int f32, float *y) {
+    if (rows < 1 || n < 1 || n > 16 * 1024 || (add && !add_w)) return -1;
+    Scratch s(f32 != 0);
+    LgRowNormArgs a{};
+    a.x = s.put(x, (size_t)rows * n); a.ldx = a.n = n;
+    if (add) { a.add = s.put(add, (size_t)rows * n); a.ld_add = n; a.add_w = s.put(add_w, n); }
+    a.mult = mult; a.norm_w = s.put(norm_w, n); a.eps = eps; a.center = center;
+    a.ldy = up(n, 64);
+    a.y = s.put<uint8_t>(nullptr, (size_t)rows * a.ldy * s.es());
+    launch_row_norm(&s.e, rows, a);
+    const std::vector<float> r = s.get(a.y, (size_t)rows * a.ldy, f32 != 0);
+    for (int i = 0; i < rows; i++) memcpy(y + (size_t)i * n, &r[(size_t)i * a.ldy], (size_t)n * 4);
+    LG_CHECK(cudaMemcpy(x, a.x, (size_t)rows * n * 4, cudaMemcpyDeviceToHost));
+    return 0;
+}
+
+// Attention over latent rows in the absorbed form: q [n][H][kv_rank + rot_dim], cache [pos + n][kv_rank + rot_dim] -> latent
+// outputs [n][H][kv_rank].  form 0: the split kernel and its merge (bf16, n <= 8), 1: the row kernel.
+extern "C" int lg_latent_attn_host(const float *q, const float *cache, const float *sink, int n, int H, int kv_rank, int rot_dim, int pos, int max_seq,
+                                   float scale, int form, int f32, float *out) {
+    if (n < 1 || H < 1 || kv_rank < 1 || rot_dim < 0 || pos < 0 || pos + n > max_seq || (form == 0 && (n > LG_MAXM || f32))) return -1;
+    Scratch s(f32 != 0);
+    Engine *e = &s.e;
+    PlanLayer l;
+    l.p = lg_plan_layer{};
+    l.p.heads = H; l.p.kv_rank = kv_rank; l.p.rot_dim = rot_dim; l.p.scale = scale; l.p.dim = l.p.vdim = 16; l.p.ff = 0;
+    layer_sizes(l);
+    l.rt = l.kvp > 512 || lg_latent_dec_smem(1, l.ldc) > PLAN_SMEM_MAX ? 0 : lg_latent_dec_smem(2, l.ldc) <= PLAN_SMEM_MAX ? 2 : 1;
+    if (form == 0 && !l.rt) return -2;
+    auto padded = [&](const float *src, int rows) {            // [latent | 0 | key part | 0]
+        std::vector<float> p((size_t)rows * l.ldc, 0.0f);
+        for (int r = 0; r < rows; r++) {
+            memcpy(&p[(size_t)r * l.ldc], src + (size_t)r * (kv_rank + rot_dim), (size_t)kv_rank * 4);
+            memcpy(&p[(size_t)r * l.ldc + l.kvp], src + (size_t)r * (kv_rank + rot_dim) + kv_rank, (size_t)rot_dim * 4);
+        }
+        return p;
+    };
+    const int seq = cache_rows(max_seq);
+    const std::vector<float> pq = padded(q, n * H), pc = padded(cache, pos + n);
+    void *dq = s.rows(pq.data(), n * H, l.ldc, n * H, l.ldc), *dc = s.rows(pc.data(), pos + n, l.ldc, seq, l.ldc);
+    int *dpos = s.put(&pos, 1);
+    l.sink = s.put(sink, H);
+    void *ol = s.put<uint8_t>(nullptr, (size_t)n * H * l.kvp * s.es());
+    if (form == 1) {
+        LgLatentRowsArgs ra{};
+        ra.q = dq; ra.cache = dc; ra.ldc = l.ldc; ra.kvp = l.kvp; ra.H = H; ra.sink = l.sink; ra.scale = scale; ra.pos = dpos; ra.out = ol;
+        launch_latent_rows(e, l, n, ra);
+    } else {
+        s.pm.seq_alloc = seq;
+        s.pm.C = latent_splits(e, H, max_seq);
+        s.pm.part = s.put<float>(nullptr, (size_t)n * H * l.kvp * s.pm.C);
+        s.pm.part_ml = s.put<float2>(nullptr, (size_t)n * H * s.pm.C);
+        launch_latent_dec(e, l, n, dq, dc, dpos, ol);
+        s.pm.part = nullptr; s.pm.part_ml = nullptr;
+    }
+    const std::vector<float> r = s.get(ol, (size_t)n * H * l.kvp, f32 != 0);
+    for (int i = 0; i < n * H; i++) memcpy(out + (size_t)i * kv_rank, &r[(size_t)i * l.kvp], (size_t)kv_rank * 4);
+    return 0;
+}
+
+// The prompt block's attention: q [n][H][dim + rot_dim] (rotated), k [pos + n][H][dim], k_rot [pos + n][rot_dim],
+// v [pos + n][H][vdim], gate [n][H][vdim] -> [n][H][vdim].
+extern "C" int lg_latent_prompt_attn_host(const float *q, const float *k, const float *k_rot, const float *v, const float *gate, const float *sink,
+                                          int n, int H, int dim, int rot_dim, int vdim, int pos, float scale, float *out) {
+    if (n < 1 || H < 1 || dim < 1 || rot_dim < 1 || vdim < 1 || vdim > 256 || pos < 0) return -1;
+    Scratch s(false);
+    Engine *e = &s.e;
+    PlanLayer l;
+    l.p = lg_plan_layer{};
+    l.p.heads = H; l.p.dim = dim; l.p.rot_dim = rot_dim; l.p.vdim = vdim; l.p.kv_rank = 16; l.p.scale = scale; l.p.ff = 0;
+    layer_sizes(l);
+    if (lg_latent_pf_smem(l.dimp, l.rotp, l.vdp) > PLAN_SMEM_MAX) return -2;
+    const int keys = pos + n, seq = cache_rows(keys), cap = up(n, 128), qh = l.dimp + l.rotp, ldq = up(H * qh, 32), ldk = up(H * l.dimp, 32), ldo = up(H * l.vdp, 64);
+    std::vector<float> hq((size_t)n * ldq), hk((size_t)keys * ldk), hc((size_t)keys * l.ldc), hv((size_t)H * l.vdp * seq), hg((size_t)n * H * l.vdp);
+    for (int h = 0; h < H; h++) {
+        for (int t = 0; t < n; t++) {
+            memcpy(&hq[(size_t)t * ldq + h * qh], q + ((size_t)t * H + h) * (dim + rot_dim), (size_t)dim * 4);
+            memcpy(&hq[(size_t)t * ldq + h * qh + l.dimp], q + ((size_t)t * H + h) * (dim + rot_dim) + dim, (size_t)rot_dim * 4);
+            memcpy(&hg[((size_t)t * H + h) * l.vdp], gate + ((size_t)t * H + h) * vdim, (size_t)vdim * 4);
+        }
+        for (int t = 0; t < keys; t++) {
+            memcpy(&hk[(size_t)t * ldk + h * l.dimp], k + ((size_t)t * H + h) * dim, (size_t)dim * 4);
+            for (int j = 0; j < vdim; j++) hv[((size_t)h * l.vdp + j) * seq + t] = v[((size_t)t * H + h) * vdim + j];
+        }
+    }
+    for (int t = 0; t < keys; t++) memcpy(&hc[(size_t)t * l.ldc + l.kvp], k_rot + (size_t)t * rot_dim, (size_t)rot_dim * 4);
+    s.pm.seq_alloc = seq;
+    l.uk.rows = ldk; l.uv.rows = up(H * l.vdp, 32);
+    s.pm.kx = (bf16 *)s.rows(hk.data(), keys, ldk, seq, ldk);
+    s.pm.vx = (bf16 *)s.rows(hv.data(), H * l.vdp, seq, l.uv.rows, seq);
+    l.sink = s.put(sink, H);
+    void *at = s.put<bf16>(nullptr, (size_t)cap * ldo);
+    launch_latent_prompt(e, l, n, cap, s.rows(hq.data(), n, ldq, cap, ldq), ldq, s.rows(hc.data(), keys, l.ldc, seq, l.ldc), s.put(hg.data(), hg.size()), H * l.vdp,
+                         s.put(&pos, 1), at, ldo);
+    const std::vector<float> r = s.get(at, (size_t)n * ldo, false);
+    for (int t = 0; t < n; t++)
+        for (int h = 0; h < H; h++) memcpy(out + ((size_t)t * H + h) * vdim, &r[(size_t)t * ldo + h * l.vdp], (size_t)vdim * 4);
+    s.pm.kx = s.pm.vx = nullptr;
+    return 0;
+}
