@@ -135,6 +135,18 @@ def test_long_decoding(lg):
         c.check(run(s, c.toks, [700, 1]), "bfloat16")             # 600 single steps across nine key tiles
 
 
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_prompts_longer_than_a_block(lg, dtype):
+    c = Case("mixed", 2310, seed=12)
+    places = np.unique(np.concatenate([np.arange(0, 2310, 13), np.arange(2040, 2060), [2309]]))       # around the border of two blocks
+    with lg.Session(c.path, None, 2400, dtype=dtype) as s:
+        c.check(s.prefill_logits(c.toks, 0, places), dtype, places)
+        # a portion that starts inside a block and a last stretch of a few tokens
+        s.prefill(c.toks[:250], 0)
+        c.check(s.prefill_logits(c.toks[250:2303], 250, places[places > 250][:150] - 250), dtype, places[places > 250][:150])
+        c.check(s.prefill_logits(c.toks[2303:], 2303, range(7)), dtype, slice(2303, 2310))
+
+
 def test_prefix_rows_and_embedding_rows(lg):
     c = Case("mixed", 120, seed=21)
     toks = c.toks
