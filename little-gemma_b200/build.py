@@ -21,7 +21,7 @@ NVCC = os.environ.get("NVCC", "/usr/local/cuda/bin/nvcc")
 
 HOST_SRC = ["lg_gguf.c", "lg_ckpt.c", "lg_quant.c", "lg_plan.c", "lg_setup.c", "lg_session.c"]
 CUDA_SRC = {"lg_engine.cu": ["lg_engine.h", "lg_device.cuh", "lg_kernels.cuh", "lg_capi.cuh", "lg_prefill.cuh", "lg_attn_deep.cuh", "lg_attn_cluster.cuh"],
-            "lg_plan.cu": ["lg_engine.h", "lg_device.cuh", "lg_dense.cuh", "lg_latent.cuh"]}
+            "lg_plan.cu": ["lg_engine.h", "lg_device.cuh", "lg_dense.cuh", "lg_latent.cuh", "lg_seq.cuh", "lg_ssd.cuh", "lg_window.cuh", "lg_plan_seq.cuh"]}
 HEADERS = [os.path.join(INC, f) for f in ("lg_abi.h", "lg_b200.h", "lg_plan.h")] + [os.path.join(HOST, f) for f in ("lg_host.h", "lg_formats.h")]
 SELF = os.path.abspath(__file__)
 

@@ -16,8 +16,9 @@ __device__ __forceinline__ float from_elem(float v) { return v; }
 __device__ __forceinline__ float from_elem(bf16 v) { return __bfloat162float(v); }
 __device__ __forceinline__ uint32_t pack_bf16(float a, float b) { __nv_bfloat162 v = __floats2bfloat162_rn(a, b); return *(uint32_t *)&v; }
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + __expf(-z)); }
-// value * gate of a gated feed-forward unit; the activation is one of enum lg_act (only ReLU so far)
+// activations of enum lg_act: value * gate of a gated unit, and the square of ReLU
 __device__ __forceinline__ float gated_unit(float gate, float up) { return fmaxf(gate, 0.0f) * up; }
+__device__ __forceinline__ float relu2_unit(float up) { const float r = fmaxf(up, 0.0f); return r * r; }
 
 __device__ __forceinline__ void mma_bf16(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
     asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
@@ -98,7 +99,9 @@ __device__ __forceinline__ void rot_q_in_place(const LgRotQ &a, int tok, int fir
 // 8-column B operand) are read with the same permutation, 16 contiguous bytes of token g.  The weight loads of a warp's first
 // batch are issued before the dependency wait.  A row's products are added in an order that depends on the matrix only,
 // never on M.
-enum { DN_STORE = 0, DN_GLU = 1, DN_HEAD = 2, DN_SIGMOID_GATE = 3 };
+// PAIR: two matrices of equal width stacked, the second (from tile split_tile on) with activations x2 and the ReLU-square
+// epilogue into bf16 rows of its own -- the two input projections of a layer whose mixer and feed-forward run side by side.
+enum { DN_STORE = 0, DN_GLU = 1, DN_HEAD = 2, DN_SIGMOID_GATE = 3, DN_PAIR = 4 };
 enum { DN_JOB_NONE = 0, DN_JOB_CACHE_ROW = 1, DN_JOB_ROT_Q = 2 };
 #define DN_GEMV_THREADS 256
 #define DN_GEMV_U 8                 // chunks of a batch: 16 loads of 16 bytes per lane in flight
@@ -115,6 +118,8 @@ struct LgDnGemvArgs {
     const float *gate; int ld_gate;             // SIGMOID_GATE: outh = acc * sigmoid(gate)
     float *amax_val; int *amax_idx;             // HEAD: [n_main][LG_MAXM] best logit and row of each CTA
     int job; LgCacheRow cr; LgRotQ rq;
+    const bf16 *x2; int split_tile;             // PAIR
+    float out_scale = 1.0f;                     // HEAD: logits = out_scale * W x
 };
 
 template <int EPI, int KS, bool RMSX>
@@ -172,6 +177,7 @@ __global__ void __launch_bounds__(DN_GEMV_THREADS, 2) lg_dn_gemv_kernel(LgDnGemv
         float c[4] = {0.0f, 0.0f, 0.0f, 0.0f};
         if (tile < a.n_tiles) {
             const bf16 *xp = RMSX ? xs + g * ldxs : a.x + (size_t)g * a.ldx + (a.tiles_per_group ? (size_t)(tile / a.tiles_per_group) * a.x_group : 0);
+            if (EPI == DN_PAIR && tile >= a.split_tile) xp = a.x2 + (size_t)g * a.ldx;
             for (int c0 = lo; c0 < hi; c0 += U) {
                 if (!first) load_batch(tile, c0);
                 first = false;
@@ -204,12 +210,16 @@ __global__ void __launch_bounds__(DN_GEMV_THREADS, 2) lg_dn_gemv_kernel(LgDnGemv
             }
             if (EPI == DN_GLU) {
                 if (r < 8) a.outh[(size_t)tok * a.ldoh + tt * 8 + r] = __float2bfloat16_rn(gated_unit(v, v8));
+            } else if (EPI == DN_PAIR) {
+                if (tt < a.split_tile) a.out[(size_t)tok * a.ldo + tt * 16 + r] = v;
+                else a.outh[(size_t)tok * a.ldoh + (tt - a.split_tile) * 16 + r] = __float2bfloat16_rn(relu2_unit(v));
             } else {
                 int row = tt * 16 + r;
                 if (a.tiles_per_group) row = (tt % a.tiles_per_group) * 16 + r + (tt / a.tiles_per_group) * a.out_group;
                 if (EPI == DN_SIGMOID_GATE) a.outh[(size_t)tok * a.ldoh + row] = __float2bfloat16_rn(v * sigmoid_f(a.gate[(size_t)tok * a.ld_gate + row]));
                 else if (EPI == DN_HEAD) {
                     if (row < a.rows) {
+                        v *= a.out_scale;
                         if (a.out) a.out[(size_t)tok * a.ldo + row] = v;
                         if (v > best || (v == best && row < besti)) { best = v; besti = row; }
                     }
@@ -248,7 +258,7 @@ __global__ void __launch_bounds__(DN_GEMV_THREADS, 2) lg_dn_gemv_kernel(LgDnGemv
 //                        weight tiles of the first stages are requested before the dependency wait;
 //   warp 5 (one thread)  issues four tcgen05.mma (M = 128, N = NT, K = 16) per block and commits the stage back;
 //   warps 0-3            read the accumulator (lane = token) and store 32 columns at a time with 16-byte stores.
-enum { DN_G_F32 = 0, DN_G_BF16 = 1, DN_G_GLU = 2 };
+enum { DN_G_F32 = 0, DN_G_BF16 = 1, DN_G_GLU = 2, DN_G_RELU2 = 3 };
 #define DN_GEMM_BM 128
 #define DN_GEMM_BK 64
 #define DN_GEMM_THREADS 192
@@ -261,6 +271,8 @@ struct LgDnGemmArgs {
     int w_early;                     // the second operand does not depend on earlier kernels
     void *out; int ldo;              // f32 / bf16 rows; GLU: bf16 rows of cols / 2
     int *err;
+    float out_scale = 1.0f;          // F32: out = out_scale * W x
+    int f32_from = 0x7fffffff; float *out2 = nullptr; int ldo2 = 0;      // BF16: columns from here on (a multiple of 32) go to f32 rows of their own
 };
 
 template <int NT, int EPI>
@@ -346,7 +358,20 @@ __global__ void __launch_bounds__(DN_GEMM_THREADS) lg_dn_gemm_kernel(const __gri
                 if (EPI == DN_G_F32) {
                     float4 *o = (float4 *)((float *)a.out + (size_t)tok * a.ldo + col);
                     #pragma unroll
+                    for (int j = 0; j < 8; j++) o[j] = make_float4(__uint_as_float(v[4 * j]) * a.out_scale, __uint_as_float(v[4 * j + 1]) * a.out_scale, __uint_as_float(v[4 * j + 2]) * a.out_scale, __uint_as_float(v[4 * j + 3]) * a.out_scale);
+                } else if (EPI == DN_G_BF16 && col >= a.f32_from) {
+                    float4 *o = (float4 *)(a.out2 + (size_t)tok * a.ldo2 + col - a.f32_from);
+                    #pragma unroll
                     for (int j = 0; j < 8; j++) o[j] = make_float4(__uint_as_float(v[4 * j]), __uint_as_float(v[4 * j + 1]), __uint_as_float(v[4 * j + 2]), __uint_as_float(v[4 * j + 3]));
+                } else if (EPI == DN_G_RELU2) {
+                    uint4 *o = (uint4 *)((bf16 *)a.out + (size_t)tok * a.ldo + col);
+                    #pragma unroll
+                    for (int j = 0; j < 4; j++) {
+                        uint32_t p[4];
+                        #pragma unroll
+                        for (int i = 0; i < 4; i++) p[i] = pack_bf16(relu2_unit(__uint_as_float(v[8 * j + 2 * i])), relu2_unit(__uint_as_float(v[8 * j + 2 * i + 1])));
+                        o[j] = make_uint4(p[0], p[1], p[2], p[3]);
+                    }
                 } else if (EPI == DN_G_BF16) {
                     uint4 *o = (uint4 *)((bf16 *)a.out + (size_t)tok * a.ldo + col);
                     #pragma unroll
@@ -386,6 +411,7 @@ struct LgDnF32Args {
     const float *x; int ldx, n;
     float *out; int ldo;
     size_t w_group; int x_group, out_group;      // blockIdx.z selects a group of rows with its own activations
+    float out_scale = 1.0f;
 };
 __global__ void __launch_bounds__(256) lg_dn_gemm_f32_kernel(LgDnF32Args a) {
     __shared__ float sx[16][68], sw[16][68];
@@ -420,7 +446,7 @@ __global__ void __launch_bounds__(256) lg_dn_gemm_f32_kernel(LgDnF32Args a) {
         #pragma unroll
         for (int j = 0; j < 4; j++) {
             const int tok = t0 + ty * 4 + i, row = r0 + tx * 4 + j;
-            if (tok < a.n && row < a.rows) O[(size_t)tok * a.ldo + row] = acc[i][j];
+            if (tok < a.n && row < a.rows) O[(size_t)tok * a.ldo + row] = acc[i][j] * a.out_scale;
         }
 }
 // the 32-bit path's epilogues as kernels of their own
@@ -429,6 +455,11 @@ __global__ void lg_dn_glu_rows(const float *gu, int ld, int n_ff, float *out, in
     const float *s = gu + (size_t)blockIdx.y * ld;
     for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < n_ff; i += gridDim.x * blockDim.x)
         out[(size_t)blockIdx.y * ldo + i] = gated_unit(s[(i >> 3) * 16 + (i & 7)], s[(i >> 3) * 16 + 8 + (i & 7)]);
+}
+__global__ void lg_dn_relu2_rows(const float *u, int ld, int n_ff, float *out, int ldo) {
+    pdl_launch(); pdl_wait();
+    for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < n_ff; i += gridDim.x * blockDim.x)
+        out[(size_t)blockIdx.y * ldo + i] = relu2_unit(u[(size_t)blockIdx.y * ld + i]);
 }
 __global__ void lg_dn_gate_rows(float *x, int ldx, const float *gate, int ldg, int n) {
     pdl_launch(); pdl_wait();
@@ -461,12 +492,15 @@ __global__ void lg_dn_argmax_rows(const float *logits, int ld, int n, float *val
 // ---------------------------------------------------------------------------------------------
 // x += mult * norm(add) * add_w (add may be null), then y = norm(x) * norm_w.  The norm divides by the root of the mean square
 // plus eps, after taking the mean off when `center` is set.  Every value of a row stays in registers between the passes.
+// PAR (layers whose branches run side by side): x += add [+ bias] as they are, and two outputs with weights of their own.
 struct LgRowNormArgs {
     float *x; int ldx, n;
     const float *add; int ld_add; const float *add_w; float mult;
     const float *norm_w; float eps; int center;
     void *y; int ldy;                // rows of T (norm_w null: not written)
     float *yf; int ldyf;             // optional f32 copy
+    const float *bias;               // PAR: a vector added to the row, or null
+    const float *norm_w2; void *y2;  // PAR: second output (null: none), leading dimension ldy
 };
 // V consecutive elements as one load / store
 template <int V> struct alignas(V * 4) LgVec { float f[V]; };
@@ -480,7 +514,7 @@ template <int V> __device__ __forceinline__ void vec_store(bf16 *p, const float 
     if (V == 4) *(uint2 *)p = make_uint2(pack_bf16(f[0], f[1]), pack_bf16(f[2], f[V - 1])); else *p = __float2bfloat16_rn(f[0]);
 }
 // item i of a thread: elements (tid + i * blockDim) * V ..
-template <typename T, int IPT, int V>
+template <typename T, int IPT, int V, bool PAR = false>
 __global__ void __launch_bounds__(1024) lg_row_norm_kernel(LgRowNormArgs a) {
     __shared__ float red[4][32];
     pdl_launch();
@@ -494,7 +528,7 @@ __global__ void __launch_bounds__(1024) lg_row_norm_kernel(LgRowNormArgs a) {
         #pragma unroll
         for (int i = 0; i < IPT; i++) { const int c = (tid + i * nt) * V; if (p && c < a.n) d[i] = vec_load<V>(p + c); else zero(d[i]); }
     };
-    fetch(w1, a.add ? a.add_w : nullptr);          // the weights do not depend on earlier kernels
+    fetch(w1, PAR ? a.norm_w2 : a.add ? a.add_w : nullptr);          // the weights do not depend on earlier kernels
     fetch(w2, a.norm_w);
     pdl_wait();
     float *x = a.x + (size_t)blockIdx.x * a.ldx;
@@ -533,7 +567,17 @@ __global__ void __launch_bounds__(1024) lg_row_norm_kernel(LgRowNormArgs a) {
             #pragma unroll
             for (int j = 0; j < V; j++) v[i].f[j] *= inv;
     };
-    if (a.add) {
+    if (PAR) {
+        LgVec<V> b[IPT];
+        fetch(b, a.bias);
+        #pragma unroll
+        for (int i = 0; i < IPT; i++) {
+            const int c = (tid + i * nt) * V;
+            #pragma unroll
+            for (int j = 0; j < V; j++) xv[i].f[j] += (a.add ? v[i].f[j] : 0.0f) + b[i].f[j];
+            if (c < a.n && (a.add || a.bias)) vec_store<V>(x + c, xv[i].f);
+        }
+    } else if (a.add) {
         normalise(0);
         #pragma unroll
         for (int i = 0; i < IPT; i++) {
@@ -556,6 +600,11 @@ __global__ void __launch_bounds__(1024) lg_row_norm_kernel(LgRowNormArgs a) {
         for (int j = 0; j < V; j++) y[j] = v[i].f[j] * w2[i].f[j];
         if (a.y) vec_store<V>((T *)a.y + (size_t)blockIdx.x * a.ldy + c, y);
         if (a.yf) vec_store<V>(a.yf + (size_t)blockIdx.x * a.ldyf + c, y);
+        if (PAR && a.y2) {
+            #pragma unroll
+            for (int j = 0; j < V; j++) y[j] = v[i].f[j] * w1[i].f[j];
+            vec_store<V>((T *)a.y2 + (size_t)blockIdx.x * a.ldy + c, y);
+        }
     }
 }
 

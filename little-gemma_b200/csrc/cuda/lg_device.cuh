@@ -13,6 +13,7 @@
 
 // error bits a kernel may raise in the engine's status word
 #define LG_ERR_MBAR_TIMEOUT 1
+#define LG_ERR_SEQ_POS 256       // a block at a position whose sequence state is gone
 
 struct LgPanel {               // quantised activations of <= 8 tokens, k = 32*nsb columns
     int8_t *q;                 // [2][nsb][256]

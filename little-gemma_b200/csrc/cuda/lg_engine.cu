@@ -1232,6 +1232,7 @@ void lg::check_err(Engine *e) {
     int err = 0;
     LG_CHECK(cudaMemcpyAsync(&err, e->err, sizeof(int), cudaMemcpyDeviceToHost, e->stream));
     LG_CHECK(cudaStreamSynchronize(e->stream));
+    if (err == LG_ERR_SEQ_POS) { fprintf(stderr, "lg_b200: a block started at a position whose sequence state is gone\n"); exit(1); }
     if (err) { fprintf(stderr, "lg_b200: device status %d (a bounded wait inside a kernel gave up)\n", err); exit(1); }
 }
 namespace {
@@ -1406,9 +1407,16 @@ bool pos_in_cache(const struct kvcache *kv, int pos, int n, const char *what) {
     return false;
 }
 
+// The same for a family whose layers carry state from token to token: a block can only start where the state is.
+bool can_start(Engine *e, const struct kvcache *kv, int pos, int n, bool wide, const char *what) {
+    if (!e->fam || e->fam->start(e, kv, pos, n, wide)) return true;
+    fprintf(stderr, "lg_b200: %s at position %d: the sequence's state is elsewhere\n", what, pos);
+    return false;
+}
+
 int spec_n(struct model *m, struct kvcache *kv, int n, const int *toks, int pos, int *out) {
     Engine *e = engine_for(m);
-    if (!pos_in_cache(kv, pos, n, "a forward")) exit(1);
+    if (!pos_in_cache(kv, pos, n, "a forward") || !can_start(e, kv, pos, n, false, "a forward")) exit(1);
     if (e->lazy.valid) {
         // the round this verify belongs to has already run (mtp_draft_device): if the caller verifies exactly the tokens it
         // was handed, the outcome is on the host already -- no launch, no wait
@@ -1494,14 +1502,17 @@ extern "C" {
 
 int kvcache_init(struct kvcache *kv, const struct model *m, int max_seq) {
     const struct config *c = &m->cfg;
-    kv->n_layer = c->n_layer; kv->max_seq = max_seq; kv->px_k = kv->px_v = nullptr;
-    kv->kv_dim = (int *)calloc(c->n_layer, sizeof(int));
-    kv->seq = (int *)calloc(c->n_layer, sizeof(int));
-    kv->f16 = (int *)calloc(c->n_layer, sizeof(int));
-    kv->k = (void **)calloc(c->n_layer, sizeof(void *));
-    kv->v = (void **)calloc(c->n_layer, sizeof(void *));
+    const LgFamily *fam = lg_family_for ? lg_family_for(m->ctx) : nullptr;
+    const int slots = fam ? fam->kv_slots(m) : c->n_layer;
+    if (slots <= 0) return -1;
+    kv->n_layer = slots; kv->max_seq = max_seq; kv->px_k = kv->px_v = nullptr;
+    kv->kv_dim = (int *)calloc(slots, sizeof(int));
+    kv->seq = (int *)calloc(slots, sizeof(int));
+    kv->f16 = (int *)calloc(slots, sizeof(int));
+    kv->k = (void **)calloc(slots, sizeof(void *));
+    kv->v = (void **)calloc(slots, sizeof(void *));
     if (!kv->kv_dim || !kv->seq || !kv->f16 || !kv->k || !kv->v) return -1;
-    if (const LgFamily *fam = lg_family_for ? lg_family_for(m->ctx) : nullptr) {
+    if (fam) {
         if (fam->kv_init(kv, m, g_compute_f32) != 0) return -1;
         LG_CHECK(cudaDeviceSynchronize());
         return 0;
@@ -1546,13 +1557,15 @@ void kvcache_save_prefix(struct kvcache *kv, int n) {
     kv->px_v = (void **)calloc(kv->n_layer, sizeof(void *));
     if (!kv->px_k || !kv->px_v) return;
     if (g_eng) LG_CHECK(cudaStreamSynchronize(g_eng->stream));
+    const LgFamily *fam = g_eng ? g_eng->fam : nullptr;
+    if (fam) fam->prefix(kv, n, false, 0);
     for (int L = 0; L < kv->n_layer; L++) {
         if (!kv->k[L]) continue;
         int rows = n < kv->seq[L] ? n : kv->seq[L];
         size_t bytes = (size_t)rows * kv->kv_dim[L] * kv_elem(kv, L);
         LG_CHECK(cudaMalloc(&kv->px_k[L], bytes));
         LG_CHECK(cudaMemcpy(kv->px_k[L], kv->k[L], bytes, cudaMemcpyDeviceToDevice));
-        if (!kv->v[L]) continue;                     // one row per position holds keys and values (latent rows)
+        if (fam || !kv->v[L]) continue;              // one row per position holds keys and values
         LG_CHECK(cudaMalloc(&kv->px_v[L], bytes));
         LG_CHECK(cudaMemcpy(kv->px_v[L], kv->v[L], bytes, cudaMemcpyDeviceToDevice));
     }
@@ -1562,19 +1575,21 @@ void kvcache_save_prefix(struct kvcache *kv, int n) {
 void kvcache_restore_prefix(struct kvcache *kv, int n) {
     if (!kv->px_k) return;
     cudaStream_t s = g_eng ? g_eng->stream : 0;
+    const LgFamily *fam = g_eng ? g_eng->fam : nullptr;
+    if (fam) { fam->prefix(kv, n, true, s); fam->start(g_eng, kv, 0, -1, false); }
     for (int L = 0; L < kv->n_layer; L++) {
         if (!kv->px_k[L]) continue;
         int rows = n < kv->seq[L] ? n : kv->seq[L];
         size_t bytes = (size_t)rows * kv->kv_dim[L] * kv_elem(kv, L);
         LG_CHECK(cudaMemcpyAsync(kv->k[L], kv->px_k[L], bytes, cudaMemcpyDeviceToDevice, s));
-        if (kv->px_v[L]) LG_CHECK(cudaMemcpyAsync(kv->v[L], kv->px_v[L], bytes, cudaMemcpyDeviceToDevice, s));
+        if (!fam && kv->px_v[L]) LG_CHECK(cudaMemcpyAsync(kv->v[L], kv->px_v[L], bytes, cudaMemcpyDeviceToDevice, s));
     }
 }
 
 void model_forward(struct model *m, struct kvcache *kv, int token, int pos, float *logits) {
     Engine *e = engine_for(m);
     e->lazy.valid = false;
-    if (!pos_in_cache(kv, pos, 1, "model_forward")) exit(1);
+    if (!pos_in_cache(kv, pos, 1, "model_forward") || !can_start(e, kv, pos, 1, false, "model_forward")) exit(1);
     upload_round(e, &token, 1, pos);
     run_forward(e, kv, 1, logits ? (F_HEAD | F_LOGITS | F_ACCEPT) : 0);
     if (logits) LG_CHECK(cudaMemcpyAsync(logits, e->logits, (size_t)m->cfg.n_vocab * 4, cudaMemcpyDeviceToHost, e->stream));
@@ -1598,7 +1613,7 @@ static void prefill_impl(struct model *m, struct kvcache *kv, const float *rows,
     const int ne = m->cfg.n_embd;
     if (n <= 0) return;
     e->lazy.valid = false;
-    if (!pos_in_cache(kv, pos0, n, "a prompt pass")) exit(1);
+    if (!pos_in_cache(kv, pos0, n, "a prompt pass") || !can_start(e, kv, pos0, 0, false, "a prompt pass")) exit(1);
     std::vector<int> toks(n), ridx(n, -1);
     bool media = false;
     for (int i = 0; i < n; i++) {
@@ -1610,6 +1625,7 @@ static void prefill_impl(struct model *m, struct kvcache *kv, const float *rows,
     if (e->fam && !media && n > LG_MAXM) {
         bind_kv(e, kv);
         i = e->fam->prefill(e, kv, toks.data(), n, pos0, want, n_want, logits);
+        if (i) e->fam->start(e, kv, pos0, i, true);
     }
     // the wide pass leaves no logits: with places asked for, it ends before the first of them
     const int n_all = n, n_wide = n_want > 0 ? std::min(n, want[0]) : n;
@@ -1661,6 +1677,7 @@ static void prefill_impl(struct model *m, struct kvcache *kv, const float *rows,
     while (w < n_want && want[w] < i) w++;
     for (; i < n; i += LG_MAXM) {
         int b = n - i < LG_MAXM ? n - i : LG_MAXM;
+        if (e->fam) e->fam->start(e, kv, pos0 + i, b, false);
         upload_round(e, toks.data() + i, b, pos0 + i);
         bool blk_media = false;
         for (int j = 0; j < b; j++) blk_media |= ids[i + j] < 0;
@@ -1703,6 +1720,7 @@ int lg_prefill_logits(struct model *m, struct kvcache *kv, const int *tokens, in
         if (want[i] < 0 || want[i] >= n || (i && want[i] <= want[i - 1])) return -1;
     for (int i = 0; i < n; i++)
         if (tokens[i] < 0 || tokens[i] >= m->cfg.n_vocab) return -1;
+    if (!can_start(engine_for(m), kv, pos0, 0, false, "lg_prefill_logits")) return -1;
     prefill_impl(m, kv, nullptr, tokens, n, pos0, want, n_want, logits);
     return 0;
 }
@@ -1714,7 +1732,7 @@ int model_forward_spec(struct model *m, struct kvcache *kv, const int *toks, int
 
 int lg_forward_spec_n(struct model *m, struct kvcache *kv, int n, const int *toks, int pos, int *out) {
     if (n < 1 || n > LG_MAXM) return -1;
-    if (!pos_in_cache(kv, pos, n, "lg_forward_spec_n")) return -2;
+    if (!pos_in_cache(kv, pos, n, "lg_forward_spec_n") || !can_start(engine_for(m), kv, pos, 0, false, "lg_forward_spec_n")) return -2;
     return spec_n(m, kv, n, toks, pos, out);
 }
 
@@ -1896,6 +1914,11 @@ int lg_rounds_enqueue(struct model *m, struct kvcache *kv, struct mtp *t, int n,
     if (n_rounds < 0 || (long long)e->pos_hi + (long long)n_rounds * n > kv->max_seq) {
         fprintf(stderr, "lg_b200: %d rounds of width %d from position <= %d could leave the cache of %d rows\n", n_rounds, n, e->pos_hi, kv->max_seq);
         return -2;
+    }
+    if (e->fam && n_rounds > 0) {
+        // (only the first rounds behind lg_rounds_begin start at a position the host knows; the device checks the others)
+        const int pos = e->pos_hi == e->st_host->pos ? e->pos_hi : 0;
+        if (!can_start(e, kv, pos, -1, false, "lg_rounds_enqueue")) return -2;
     }
     e->pos_hi += n_rounds * n;
     cudaGraphExec_t g = round_graph(e, kv, d, n, mode == 2, true);

@@ -38,6 +38,7 @@ struct LgFamily {
     const char *name;
     void (*load)(Engine *e);                                       // weights + activations (e->m, e->ctx, e->stream are set)
     void (*release)(Engine *e);
+    int  (*kv_slots)(const struct model *m);                       // cache entries (a layer that runs several times has one per run)
     int  (*kv_init)(struct kvcache *kv, const struct model *m, bool f32);   // fills kv_dim / seq / f16 and allocates; 0 / -1
     void (*bind)(Engine *e, const struct kvcache *kv);             // scratch that depends on the cache's geometry
     // M <= LG_MAXM rows at st->pos from st->toks (captured into graphs); with F_HEAD: e->hidden, argmax candidates in
@@ -48,6 +49,10 @@ struct LgFamily {
     // (host, [n_want][n_vocab]).  Returns the number of tokens it took (the rest goes through `forward`).
     int  (*prefill)(Engine *e, const struct kvcache *kv, const int *toks, int n, int pos0, const int *want, int n_want, float *logits);
     int  (*bench_block)(Engine *e, const struct kvcache *kv, int n, int pos0, int only);   // kernels of one wide block, timing only
+    // Told before n tokens run at pos (wide: as a prompt block; n < 0: rounds that only the device follows); false: the cache holds no state
+    // for that position.
+    bool (*start)(Engine *e, const struct kvcache *kv, int pos, int n, bool wide);
+    bool (*prefix)(struct kvcache *kv, int n, bool restore, cudaStream_t s);               // what a saved prefix needs besides cache rows
 };
 
 struct WMat {

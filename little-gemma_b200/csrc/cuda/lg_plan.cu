@@ -1,12 +1,15 @@
-// lg_plan.cu -- the family of models described by a layer plan (lg_plan.h): dense bf16 weights, per-layer mixers (latent
-// attention so far), f32 residual rows.  Decode and verify steps run the small-M matmuls and the split attention over the
-// latent cache; prompts run blocks of up to PLAN_BLOCK tokens through the tcgen05 matmul and the block attention.  In 32-bit
-// mode every product, activation and cache row is f32.
+// lg_plan.cu -- the family of models described by a layer plan (lg_plan.h): dense bf16 weights, per-layer mixers (latent attention,
+// grouped windowed attention, state-space), f32 residual rows.  Decode and verify steps run the small-M matmuls, the split attention
+// over the cache and the state-space step; prompts run blocks of up to PLAN_BLOCK tokens through the tcgen05 matmul, block attention
+// and chunked state-space kernels.  In 32-bit mode every product, activation and cache row is f32.
 #include <algorithm>
 #include <tuple>
 #include "lg_engine.h"
 #include "lg_plan.h"
 #include "lg_latent.cuh"
+#include "lg_seq.cuh"
+#include "lg_ssd.cuh"
+#include "lg_window.cuh"
 
 namespace lg {
 
@@ -31,7 +34,15 @@ struct PlanLayer {
     int owns, spec;                                           // spec: which rotation table
     int rt;                                                   // row tiles of 16 per CTA of the decode attention (0: the row kernel)
     DMat in, uq, ukT, uk, uv, o, gu, down;             // uk: keys from latents (prompt pass); ukT: the same per head, transposed (decode)
-    float *norm1, *norm1b, *norm2 = nullptr, *norm2b = nullptr, *q_norm, *kv_norm = nullptr, *sink;
+    // grouped attention and state-space layers (lg_plan_seq.cuh)
+    int np = 0, npl = 0, nst = 0, vs = 0;                     // state columns padded to 16; per lane of the step kernel; of a stored state row; value columns per chunk CTA
+    int in_rows = 0, ch0 = 0, nch = 0, dt_off = 0, q_cols = 0, k_cols = 0;   // projection row: [q | k | v] or [z | x | B | C | step sizes]; convolved columns ch0 .. ch0 + nch
+    int at_cols = 0, act_off = 0, mask = 0, C = 1;            // output product's columns: mixer rows, feed-forward rows from act_off on; ring of projected rows; key splits
+    int chunked = 1;                                          // the prompt kernels hold the sizes
+    float lambda = 0.0f, out_mult = 1.0f, eps = 0.0f;
+    float *conv_w = nullptr, *conv_b = nullptr, *dt_bias = nullptr, *a_log = nullptr, *d = nullptr, *gnorm = nullptr;
+    DMat inup;                                                // input projection over the feed-forward's; `in` and `gu` are its parts
+    float *norm1 = nullptr, *norm1b = nullptr, *norm2 = nullptr, *norm2b = nullptr, *q_norm = nullptr, *kv_norm = nullptr, *sink = nullptr;
 };
 
 // Activations of up to `cap` token rows.
@@ -39,6 +50,8 @@ struct PlanBuf {
     int cap = 0;
     float *x = nullptr, *pj = nullptr, *o = nullptr, *gu = nullptr;
     void *h = nullptr, *cq = nullptr, *q = nullptr, *qa = nullptr, *ol = nullptr, *at = nullptr, *act = nullptr;
+    void *h2 = nullptr, *cv = nullptr, *y = nullptr;          // second norm; convolved rows; state-space outputs
+    float *dt = nullptr, *ds = nullptr, *decay = nullptr; bf16 *s_hi = nullptr, *s_lo = nullptr;    // raw step sizes; chunk sums, decays and states
     std::vector<float2 *> tab;
     int *toks = nullptr, *pos = nullptr;                      // of the block (narrow: the engine's round state)
 };
@@ -50,6 +63,10 @@ struct PlanModel {
     float *out_norm = nullptr;
     struct Rot { float base; int dims; double *freq; };
     std::vector<Rot> rot;
+    struct Run { int layer, slot; const float *step; };       // a looped layer runs once per pass, with cache and state of its own
+    std::vector<Run> runs;
+    float *step = nullptr;                                    // [times][width]
+    const struct kvcache *st_kv = nullptr; int st_lo = -1, st_hi = -1;       // positions a block may start at, as far as the host knows (-1: ask the device)
     PlanBuf nb, wb;
     bool wide_ok = false;
     // bound to a cache
@@ -103,14 +120,14 @@ struct MatBuild {
         else { const uint16_t b = bf16_bits(v); memcpy(&buf[i * 2], &b, 2); }
     }
     // row `src` of t; its columns come in segments of seg that start every seg_to columns here (0: one piece)
-    void row(int dst, const struct gguf_tensor *t, int src, int seg = 0, int seg_to = 0) {
+    void row(int dst, const struct gguf_tensor *t, int src, int seg = 0, int seg_to = 0, int col0 = 0) {
         const int n = (int)t->dims[0];
         if (!f32 && t->type == GGML_TYPE_BF16 && seg == seg_to) {
-            memcpy(&buf[(size_t)dst * ldk * 2], (const uint8_t *)t->data + (size_t)src * n * 2, (size_t)n * 2);
+            memcpy(&buf[((size_t)dst * ldk + col0) * 2], (const uint8_t *)t->data + (size_t)src * n * 2, (size_t)n * 2);
             return;
         }
         const std::vector<float> f = row_f32(t, src);
-        for (int i = 0; i < n; i++) put((size_t)dst * ldk + (seg ? i / seg * seg_to + i % seg : i), f[i]);
+        for (int i = 0; i < n; i++) put((size_t)dst * ldk + col0 + (seg ? i / seg * seg_to + i % seg : i), f[i]);
     }
     DMat upload(Engine *e) {
         DMat m;
@@ -136,6 +153,7 @@ template <int EPI, bool RMSX> void gemv_attrs() {
     smem_attr(lg_dn_gemv_kernel<EPI, 1, RMSX>, PLAN_SMEM_SMALL); smem_attr(lg_dn_gemv_kernel<EPI, 2, RMSX>, PLAN_SMEM_SMALL);
     smem_attr(lg_dn_gemv_kernel<EPI, 4, RMSX>, PLAN_SMEM_SMALL); smem_attr(lg_dn_gemv_kernel<EPI, 8, RMSX>, PLAN_SMEM_SMALL);
 }
+void seq_attributes();
 void plan_attributes() {
     static bool done[64] = {false};
     int dev = 0;
@@ -149,11 +167,14 @@ void plan_attributes() {
     smem_attr(lg_latent_dec_attn_kernel<1, 2>); smem_attr(lg_latent_dec_attn_kernel<1, 4>); smem_attr(lg_latent_dec_attn_kernel<1, 8>);
     smem_attr(lg_latent_dec_attn_kernel<2, 2>); smem_attr(lg_latent_dec_attn_kernel<2, 4>); smem_attr(lg_latent_dec_attn_kernel<2, 8>);
     smem_attr(lg_latent_pf_attn_kernel);
+    seq_attributes();
     smem_attr(lg_latent_merge_kernel, PLAN_SMEM_SMALL); smem_attr(lg_latent_attn_rows_kernel<float>, PLAN_SMEM_SMALL); smem_attr(lg_latent_attn_rows_kernel<bf16>, PLAN_SMEM_SMALL);
 }
 
+void seq_buf_alloc(Engine *e, PlanBuf &b, int cap, bool narrow);
 void buf_alloc(Engine *e, PlanBuf &b, int cap, bool narrow) {
     PlanModel *pm = e->plan;
+    if (pm->plan->form == LG_FORM_PARALLEL) { seq_buf_alloc(e, b, cap, narrow); return; }
     const size_t es = e->f32 ? 4 : 2;
     size_t pj = 0, o = up(pm->plan->width, 32), gu = 0, cq = 0, q = 0, qa = 0, ol = 0, at = 0, act = 0;
     for (auto &l : pm->L) {
@@ -176,6 +197,7 @@ void buf_alloc(Engine *e, PlanBuf &b, int cap, bool narrow) {
 void buf_free(PlanBuf &b, bool narrow) {
     if (!narrow) cudaFree(b.x);
     cudaFree(b.pj); cudaFree(b.o); cudaFree(b.gu); cudaFree(b.h); cudaFree(b.cq); cudaFree(b.q); cudaFree(b.qa); cudaFree(b.ol); cudaFree(b.at); cudaFree(b.act);
+    cudaFree(b.h2); cudaFree(b.cv); cudaFree(b.y); cudaFree(b.dt); cudaFree(b.ds); cudaFree(b.decay); cudaFree(b.s_hi); cudaFree(b.s_lo);
     for (auto t : b.tab) cudaFree(t);
     cudaFree(b.toks); cudaFree(b.pos);
     b = PlanBuf();
@@ -185,6 +207,98 @@ void layer_sizes(PlanLayer &l) {
     const struct lg_plan_layer &p = l.p;
     l.dimp = up(p.dim, 16); l.rotp = up(p.rot_dim, 16); l.kvp = up(p.kv_rank, 16); l.vdp = up(p.vdim, 16); l.ffp = up(p.ff, 16);
     l.ldc = l.kvp + l.rotp;
+}
+
+void seq_layer_sizes(PlanLayer &l);
+void seq_layer_load(Engine *e, int L, PlanLayer &l);
+void seq_layer_free(PlanLayer &l);
+float *vec_offset(Engine *e, int L, const char *leaf, int n, float offset);
+
+void latent_layer_load(Engine *e, int i, PlanLayer &l) {
+    PlanModel *pm = e->plan;
+    const int W = pm->plan->width;
+    layer_sizes(l);
+    const struct lg_plan_layer &p = l.p;
+    const int H = p.heads;
+    l.owns = p.kv_src == i;
+    l.kv_off = up(p.q_rank, 16);
+    l.rot_off = l.kv_off + (l.owns ? l.kvp : 0);
+    l.g_off = l.rot_off + (l.owns ? l.rotp : 0);
+    {   // everything that reads the layer's input: query latent, cached latent and key part, output gate
+        MatBuild b(e, l.g_off + H * l.vdp, W);
+        put_groups(b, 0, need(e, i, "attn_q_a", p.q_rank, W), 1, p.q_rank, 0);
+        if (l.owns) {
+            const struct gguf_tensor *t = need(e, i, "attn_kv_a", p.kv_rank + p.rot_dim, W);
+            for (int r = 0; r < p.kv_rank + p.rot_dim; r++) b.row(r < p.kv_rank ? l.kv_off + r : l.rot_off + r - p.kv_rank, t, r);
+        }
+        put_groups(b, l.g_off, need(e, i, "attn_gate", H * p.vdim, W), H, p.vdim, l.vdp);
+        l.in = b.upload(e);
+    }
+    {   // queries: per head [unrotated | rotated]
+        const struct gguf_tensor *t = need(e, i, "attn_q_b", H * (p.dim + p.rot_dim), p.q_rank);
+        MatBuild b(e, H * (l.dimp + l.rotp), p.q_rank);
+        for (int h = 0; h < H; h++)
+            for (int r = 0; r < p.dim + p.rot_dim; r++)
+                b.row(h * (l.dimp + l.rotp) + (r < p.dim ? r : l.dimp + r - p.dim), t, h * (p.dim + p.rot_dim) + r);
+        l.uq = b.upload(e);
+    }
+    const struct gguf_tensor *uk = need(e, i, "attn_k_b", H * p.dim, p.kv_rank), *uv = need(e, i, "attn_v_b", H * p.vdim, p.kv_rank);
+    {   // the key expansion transposed per head: rows = latent columns, contraction over the head's dimensions
+        MatBuild b(e, H * l.kvp, p.dim);
+        for (int h = 0; h < H; h++)
+            for (int d = 0; d < p.dim; d++) {
+                const std::vector<float> f = row_f32(uk, h * p.dim + d);
+                for (int r = 0; r < p.kv_rank; r++) b.put((size_t)(h * l.kvp + r) * b.ldk + d, f[r]);
+            }
+        l.ukT = b.upload(e);
+    }
+    {
+        MatBuild b(e, H * l.vdp, p.kv_rank);
+        put_groups(b, 0, uv, H, p.vdim, l.vdp);
+        l.uv = b.upload(e);
+    }
+    if (!e->f32) {
+        MatBuild b(e, H * l.dimp, p.kv_rank);
+        put_groups(b, 0, uk, H, p.dim, l.dimp);
+        const size_t before = e->weight_bytes;
+        l.uk = b.upload(e);
+        e->weight_bytes = before;                        // a second copy of weights already counted
+    }
+    {
+        const struct gguf_tensor *t = need(e, i, "attn_output", W, H * p.vdim);
+        MatBuild b(e, W, H * l.vdp);
+        for (int r = 0; r < W; r++) b.row(r, t, r, p.vdim, l.vdp);
+        l.o = b.upload(e);
+    }
+    if (p.ff) {
+        const struct gguf_tensor *g = need(e, i, "ffn_gate", p.ff, W), *u = need(e, i, "ffn_up", p.ff, W), *d = need(e, i, "ffn_down", W, p.ff);
+        MatBuild b(e, 2 * l.ffp, W);
+        for (int r = 0; r < p.ff; r++) { b.row(r / 8 * 16 + r % 8, g, r); b.row(r / 8 * 16 + 8 + r % 8, u, r); }   // 8 gate rows, their 8 up rows
+        l.gu = b.upload(e);
+        MatBuild c(e, W, l.ffp);
+        for (int r = 0; r < W; r++) c.row(r, d, r);
+        l.down = c.upload(e);
+        l.norm2 = vec(e, i, "ffn_norm", W); l.norm2b = vec(e, i, "post_ffw_norm", W);
+    }
+    l.norm1 = vec(e, i, "attn_norm", W); l.norm1b = vec(e, i, "post_attention_norm", W);
+    l.q_norm = vec(e, i, "attn_q_a_norm", p.q_rank);
+    if (l.owns) l.kv_norm = vec(e, i, "attn_kv_a_norm", p.kv_rank);
+    l.sink = vec(e, i, "attn_sinks", H);
+    l.spec = -1;
+    for (size_t s = 0; s < pm->rot.size(); s++) if (pm->rot[s].base == p.rot_base && pm->rot[s].dims == p.rot_dims) l.spec = (int)s;
+    if (l.spec < 0) {
+        std::vector<double> f(p.rot_dims / 2 + 1);
+        for (int j = 0; j < p.rot_dims / 2; j++) f[j] = pow((double)p.rot_base, -2.0 * j / p.rot_dims);
+        double *d = dalloc<double>(f.size());
+        h2d_sync(d, f.data(), f.size() * 8);
+        l.spec = (int)pm->rot.size();
+        pm->rot.push_back({p.rot_base, p.rot_dims, d});
+    }
+    l.rt = l.kvp > 512 ? 0 : lg_latent_dec_smem(2, l.ldc) <= PLAN_SMEM_MAX ? 2 : lg_latent_dec_smem(1, l.ldc) <= PLAN_SMEM_MAX ? 1 : 0;
+    if (e->f32) l.rt = 0;
+    if (l.vdp > 256 || lg_latent_pf_smem(l.dimp, l.rotp, l.vdp) > PLAN_SMEM_MAX) pm->wide_ok = false;
+    if ((size_t)(l.ldc + l.kvp + 128) * 4 > PLAN_SMEM_SMALL || (size_t)LG_LM_GROUPS * l.kvp * 4 > PLAN_SMEM_SMALL ||
+        (size_t)LG_MAXM * (l.uq.ldk + 8) * 2 > PLAN_SMEM_SMALL) { fprintf(stderr, "lg_b200: layer %d: latent sizes beyond what the kernels hold\n", i); exit(1); }
 }
 
 void plan_load(Engine *e) {
@@ -200,88 +314,9 @@ void plan_load(Engine *e) {
     for (int i = 0; i < P->n_layer; i++) {
         PlanLayer &l = pm->L[i];
         l.p = P->layer[i];
-        layer_sizes(l);
-        const struct lg_plan_layer &p = l.p;
-        const int H = p.heads;
-        l.owns = p.kv_src == i;
-        l.kv_off = up(p.q_rank, 16);
-        l.rot_off = l.kv_off + (l.owns ? l.kvp : 0);
-        l.g_off = l.rot_off + (l.owns ? l.rotp : 0);
-        {   // everything that reads the layer's input: query latent, cached latent and key part, output gate
-            MatBuild b(e, l.g_off + H * l.vdp, W);
-            put_groups(b, 0, need(e, i, "attn_q_a", p.q_rank, W), 1, p.q_rank, 0);
-            if (l.owns) {
-                const struct gguf_tensor *t = need(e, i, "attn_kv_a", p.kv_rank + p.rot_dim, W);
-                for (int r = 0; r < p.kv_rank + p.rot_dim; r++) b.row(r < p.kv_rank ? l.kv_off + r : l.rot_off + r - p.kv_rank, t, r);
-            }
-            put_groups(b, l.g_off, need(e, i, "attn_gate", H * p.vdim, W), H, p.vdim, l.vdp);
-            l.in = b.upload(e);
-        }
-        {   // queries: per head [unrotated | rotated]
-            const struct gguf_tensor *t = need(e, i, "attn_q_b", H * (p.dim + p.rot_dim), p.q_rank);
-            MatBuild b(e, H * (l.dimp + l.rotp), p.q_rank);
-            for (int h = 0; h < H; h++)
-                for (int r = 0; r < p.dim + p.rot_dim; r++)
-                    b.row(h * (l.dimp + l.rotp) + (r < p.dim ? r : l.dimp + r - p.dim), t, h * (p.dim + p.rot_dim) + r);
-            l.uq = b.upload(e);
-        }
-        const struct gguf_tensor *uk = need(e, i, "attn_k_b", H * p.dim, p.kv_rank), *uv = need(e, i, "attn_v_b", H * p.vdim, p.kv_rank);
-        {   // the key expansion transposed per head: rows = latent columns, contraction over the head's dimensions
-            MatBuild b(e, H * l.kvp, p.dim);
-            for (int h = 0; h < H; h++)
-                for (int d = 0; d < p.dim; d++) {
-                    const std::vector<float> f = row_f32(uk, h * p.dim + d);
-                    for (int r = 0; r < p.kv_rank; r++) b.put((size_t)(h * l.kvp + r) * b.ldk + d, f[r]);
-                }
-            l.ukT = b.upload(e);
-        }
-        {
-            MatBuild b(e, H * l.vdp, p.kv_rank);
-            put_groups(b, 0, uv, H, p.vdim, l.vdp);
-            l.uv = b.upload(e);
-        }
-        if (!e->f32) {
-            MatBuild b(e, H * l.dimp, p.kv_rank);
-            put_groups(b, 0, uk, H, p.dim, l.dimp);
-            const size_t before = e->weight_bytes;
-            l.uk = b.upload(e);
-            e->weight_bytes = before;                        // a second copy of weights already counted
-        }
-        {
-            const struct gguf_tensor *t = need(e, i, "attn_output", W, H * p.vdim);
-            MatBuild b(e, W, H * l.vdp);
-            for (int r = 0; r < W; r++) b.row(r, t, r, p.vdim, l.vdp);
-            l.o = b.upload(e);
-        }
-        if (p.ff) {
-            const struct gguf_tensor *g = need(e, i, "ffn_gate", p.ff, W), *u = need(e, i, "ffn_up", p.ff, W), *d = need(e, i, "ffn_down", W, p.ff);
-            MatBuild b(e, 2 * l.ffp, W);
-            for (int r = 0; r < p.ff; r++) { b.row(r / 8 * 16 + r % 8, g, r); b.row(r / 8 * 16 + 8 + r % 8, u, r); }   // 8 gate rows, their 8 up rows
-            l.gu = b.upload(e);
-            MatBuild c(e, W, l.ffp);
-            for (int r = 0; r < W; r++) c.row(r, d, r);
-            l.down = c.upload(e);
-            l.norm2 = vec(e, i, "ffn_norm", W); l.norm2b = vec(e, i, "post_ffw_norm", W);
-        }
-        l.norm1 = vec(e, i, "attn_norm", W); l.norm1b = vec(e, i, "post_attention_norm", W);
-        l.q_norm = vec(e, i, "attn_q_a_norm", p.q_rank);
-        if (l.owns) l.kv_norm = vec(e, i, "attn_kv_a_norm", p.kv_rank);
-        l.sink = vec(e, i, "attn_sinks", H);
-        l.spec = -1;
-        for (size_t s = 0; s < pm->rot.size(); s++) if (pm->rot[s].base == p.rot_base && pm->rot[s].dims == p.rot_dims) l.spec = (int)s;
-        if (l.spec < 0) {
-            std::vector<double> f(p.rot_dims / 2 + 1);
-            for (int j = 0; j < p.rot_dims / 2; j++) f[j] = pow((double)p.rot_base, -2.0 * j / p.rot_dims);
-            double *d = dalloc<double>(f.size());
-            h2d_sync(d, f.data(), f.size() * 8);
-            l.spec = (int)pm->rot.size();
-            pm->rot.push_back({p.rot_base, p.rot_dims, d});
-        }
-        l.rt = l.kvp > 512 ? 0 : lg_latent_dec_smem(2, l.ldc) <= PLAN_SMEM_MAX ? 2 : lg_latent_dec_smem(1, l.ldc) <= PLAN_SMEM_MAX ? 1 : 0;
-        if (e->f32) l.rt = 0;
-        if (l.vdp > 256 || lg_latent_pf_smem(l.dimp, l.rotp, l.vdp) > PLAN_SMEM_MAX) pm->wide_ok = false;
-        if ((size_t)(l.ldc + l.kvp + 128) * 4 > PLAN_SMEM_SMALL || (size_t)LG_LM_GROUPS * l.kvp * 4 > PLAN_SMEM_SMALL ||
-            (size_t)LG_MAXM * (l.uq.ldk + 8) * 2 > PLAN_SMEM_SMALL) { fprintf(stderr, "lg_b200: layer %d: latent sizes beyond what the kernels hold\n", i); exit(1); }
+        l.eps = P->norm_eps;
+        if (P->form == LG_FORM_PARALLEL) { seq_layer_sizes(l); seq_layer_load(e, i, l); }
+        else latent_layer_load(e, i, l);
     }
     if (e->f32) pm->wide_ok = true;
     static const int wide = env_int("LG_PREFILL_WIDE", 1);
@@ -293,7 +328,18 @@ void plan_load(Engine *e) {
         pm->embed = b.upload(e);
     }
     e->head.ldo = pm->embed.rows;
-    pm->out_norm = vec(e, -1, "output_norm", W);
+    pm->out_norm = vec_offset(e, -1, "output_norm", W, P->norm_offset);
+    if (P->loop_times) {
+        const struct gguf_tensor *t = need(e, -1, "loop_step", P->loop_times, W);
+        std::vector<float> f;
+        for (int r = 0; r < P->loop_times; r++) { const std::vector<float> row = row_f32(t, r); f.insert(f.end(), row.begin(), row.end()); }
+        pm->step = upload_f32(f.data(), f.size());
+    }
+    for (int r = 0; r < lg_plan_runs(P); r++) {
+        int pass = -1;
+        const int L = lg_plan_run_layer(P, r, &pass);
+        pm->runs.push_back({L, r, pass < 0 ? nullptr : pm->step + (size_t)pass * W});
+    }
     buf_alloc(e, pm->nb, LG_MAXM, true);
     if (e->f32) pm->logits = dalloc<float>((size_t)LG_MAXM * e->head.ldo);
 }
@@ -310,12 +356,14 @@ void plan_release(Engine *e) {
     if (!pm) return;
     plan_unbind(pm);
     for (auto &l : pm->L) {
-        for (DMat *m : {&l.in, &l.uq, &l.ukT, &l.uk, &l.uv, &l.o, &l.gu, &l.down}) dmat_free(*m);
+        if (l.inup.w) l.in = l.gu = DMat();                  // parts of it
+        for (DMat *m : {&l.in, &l.uq, &l.ukT, &l.uk, &l.uv, &l.o, &l.gu, &l.down, &l.inup}) dmat_free(*m);
+        seq_layer_free(l);
         for (float *v : {l.norm1, l.norm1b, l.norm2, l.norm2b, l.q_norm, l.kv_norm, l.sink}) cudaFree(v);
     }
     for (auto &r : pm->rot) cudaFree(r.freq);
     dmat_free(pm->embed);
-    cudaFree(pm->out_norm); cudaFree(pm->logits);
+    cudaFree(pm->out_norm); cudaFree(pm->logits); cudaFree(pm->step);
     buf_free(pm->nb, true);
     lg_plan_free(pm->plan);
     delete pm;
@@ -327,9 +375,21 @@ void plan_release(Engine *e) {
 // ------------------------------------------------------------------------------------------
 int cache_rows(int max_seq) { return up(max_seq, 128); }      // whole boxes of the tiled copies
 
+int plan_kv_slots(const struct model *m) {
+    struct lg_plan *P = lg_plan_read(m->ctx);
+    const int n = P ? lg_plan_runs(P) : 0;
+    lg_plan_free(P);
+    return n;
+}
+int seq_kv_init(struct kvcache *kv, const struct lg_plan *P, bool f32);
 int plan_kv_init(struct kvcache *kv, const struct model *m, bool f32) {
     struct lg_plan *P = lg_plan_read(m->ctx);
     if (!P) return -1;
+    if (P->form == LG_FORM_PARALLEL) {
+        const int rc = seq_kv_init(kv, P, f32);
+        lg_plan_free(P);
+        return rc;
+    }
     for (int i = 0; i < P->n_layer; i++) {
         PlanLayer l;
         l.p = P->layer[i];
@@ -347,10 +407,12 @@ int plan_kv_init(struct kvcache *kv, const struct model *m, bool f32) {
 }
 
 int latent_splits(const Engine *e, int heads, int max_seq);
+void seq_bind(Engine *e, const struct kvcache *kv);
 void plan_bind(Engine *e, const struct kvcache *kv) {
     PlanModel *pm = e->plan;
     plan_unbind(pm);
     pm->max_seq = kv->max_seq; pm->seq_alloc = cache_rows(kv->max_seq);
+    if (pm->plan->form == LG_FORM_PARALLEL) { seq_bind(e, kv); return; }
     if (e->f32) return;
     size_t rows = 0;
     int most = 1;
@@ -401,8 +463,7 @@ const CUtensorMap &buf_map(PlanModel *pm, const void *x, int k, int ld, int rows
 }
 // out[i][j] = row i of x (n of them count) . row j of w (w_rows, a multiple of 32); maps of w with boxes of 128 / 256 rows
 template <int EPI>
-void launch_gemm_maps(Engine *e, const CUtensorMap &x, int n, const CUtensorMap &w128, const CUtensorMap &w256, int w_rows, int nkb, void *out, int ldo, bool w_early) {
-    LgDnGemmArgs a{};
+void launch_gemm_maps(Engine *e, const CUtensorMap &x, int n, const CUtensorMap &w128, const CUtensorMap &w256, int w_rows, int nkb, void *out, int ldo, bool w_early, LgDnGemmArgs a = LgDnGemmArgs{}) {
     a.nkb = nkb; a.n_tok = n; a.cols = w_rows; a.out = out; a.ldo = ldo; a.err = e->err; a.w_early = w_early;
     const int ty = (n + DN_GEMM_BM - 1) / DN_GEMM_BM;
     if ((w_rows + 255) / 256 * ty >= e->sm_count)
@@ -412,11 +473,12 @@ void launch_gemm_maps(Engine *e, const CUtensorMap &x, int n, const CUtensorMap 
 }
 // x: [x_rows][ldx] bf16, of which n rows count
 template <int EPI>
-void launch_dn_gemm(Engine *e, const DMat &W, const void *x, int ldx, int x_rows, int n, void *out, int ldo) {
-    launch_gemm_maps<EPI>(e, buf_map(e->plan, x, W.k, ldx, x_rows, DN_GEMM_BM), n, W.map[0], W.map[1], W.rows, W.ldk / DN_GEMM_BK, out, ldo, true);
+void launch_dn_gemm(Engine *e, const DMat &W, const void *x, int ldx, int x_rows, int n, void *out, int ldo, LgDnGemmArgs a = LgDnGemmArgs{}) {
+    launch_gemm_maps<EPI>(e, buf_map(e->plan, x, W.k, ldx, x_rows, DN_GEMM_BM), n, W.map[0], W.map[1], W.rows, W.ldk / DN_GEMM_BK, out, ldo, true, a);
 }
-void launch_f32(Engine *e, const DMat &W, const void *x, int ldx, int n, void *out, int ldo, int groups = 1, int group_rows = 0, int x_group = 0, int out_group = 0) {
+void launch_f32(Engine *e, const DMat &W, const void *x, int ldx, int n, void *out, int ldo, int groups = 1, int group_rows = 0, int x_group = 0, int out_group = 0, float scale = 1.0f) {
     LgDnF32Args a{};
+    a.out_scale = scale;
     a.w = (const float *)W.w; a.ldk = W.ldk; a.rows = groups > 1 ? group_rows : W.rows; a.k = W.k;
     if (groups == 1 && group_rows) a.rows = group_rows;
     a.x = (const float *)x; a.ldx = ldx; a.n = n; a.out = (float *)out; a.ldo = ldo;
@@ -439,6 +501,20 @@ void launch_row_norm(Engine *e, int n, LgRowNormArgs a) {
     }
 }
 
+void launch_row_norm_par(Engine *e, int n, LgRowNormArgs a) {
+    const int vec = a.n % 4 == 0 && a.ldx % 4 == 0 && a.ldy % 4 == 0 && a.ld_add % 4 == 0 ? 4 : 1, items = a.n / vec;
+    const int threads = std::min(1024, std::max(64, up((items + 1) / 2, 32)));
+    const int ipt = (items + threads - 1) / threads;
+    auto go = [&](auto kernel) { launch_k(e, kernel, dim3(n), dim3(threads), 0, a); };
+    if (e->f32) {
+        if (vec == 4) { if (ipt <= 2) go(lg_row_norm_kernel<float, 2, 4, true>); else go(lg_row_norm_kernel<float, 4, 4, true>); }
+        else go(lg_row_norm_kernel<float, 16, 1, true>);
+    } else {
+        if (vec == 4) { if (ipt <= 2) go(lg_row_norm_kernel<bf16, 2, 4, true>); else go(lg_row_norm_kernel<bf16, 4, 4, true>); }
+        else go(lg_row_norm_kernel<bf16, 16, 1, true>);
+    }
+}
+
 // ------------------------------------------------------------------------------------------
 // a pass over the layers
 // ------------------------------------------------------------------------------------------
@@ -447,6 +523,7 @@ struct Pass {
     int n; bool wide;
     const int *toks, *pos;                        // device
     int pos0;                                     // wide: the host's copy of *pos
+    bool first = true;                            // wide: the first block of a prompt pass
 };
 
 void plan_embed_rows(Engine *e, const int *toks, int n, float *x) {
@@ -594,12 +671,15 @@ void gated(Engine *e, PlanLayer &l, const void *x, int ldx, const Pass &p) {
     }
 }
 
+#include "lg_plan_seq.cuh"
+
 // x in place -> every layer -> (with final_norm) the normed rows in b->h and, narrow, in e->hidden
 void plan_layers(Engine *e, const struct kvcache *kv, const Pass &p, bool final_norm, int only) {
     PlanModel *pm = e->plan;
     PlanBuf &b = *p.b;
     const struct lg_plan *P = pm->plan;
     const int W = P->width, ldh = up(W, 64);
+    if (P->form == LG_FORM_PARALLEL) { seq_layers(e, kv, p, final_norm, only); return; }
     if (only & C_MISC)
         for (size_t s0 = 0; s0 < pm->rot.size(); s0 += 8) {
             LgRotTables a{};
@@ -648,13 +728,13 @@ int plan_forward(Engine *e, const struct kvcache *kv, int M, int flags, int only
     const int ldh = up(pm->plan->width, 64);
     if (e->f32) {
         if (!lg) lg = pm->logits;
-        launch_f32(e, pm->embed, pm->nb.h, ldh, M, lg, e->head.ldo);
+        launch_f32(e, pm->embed, pm->nb.h, ldh, M, lg, e->head.ldo, 1, 0, 0, 0, pm->plan->logit_scale);
         launch_k(e, lg_dn_argmax_rows, dim3(32, M), dim3(256), 0, (const float *)lg, e->head.ldo, pm->plan->vocab, e->amax_val, e->amax_idx);
         return 32;
     }
     LgDnGemvArgs a{};
     a.x = (const bf16 *)pm->nb.h; a.ldx = ldh; a.M = M; a.rows = pm->plan->vocab; a.out = lg; a.ldo = e->head.ldo;
-    a.amax_val = e->amax_val; a.amax_idx = e->amax_idx;
+    a.amax_val = e->amax_val; a.amax_idx = e->amax_idx; a.out_scale = pm->plan->logit_scale;
     return launch_dn_gemv<DN_HEAD, false>(e, pm->embed, a, 0, e->head_ctas);
 }
 
@@ -670,6 +750,7 @@ bool wide_ready(Engine *e) {
     const int ldh = up(pm->plan->width, 64);
     pm->hg = dalloc<uint8_t>((size_t)PLAN_HEAD_ROWS * ldh * (e->f32 ? 4 : 2));
     pm->wlog = dalloc<float>((size_t)PLAN_HEAD_ROWS * pm->embed.rows);
+    if (pm->plan->form == LG_FORM_PARALLEL) return true;
     size_t kx = 0, vx = 0;
     for (auto &l : pm->L) { kx = std::max(kx, (size_t)l.uk.rows); vx = std::max(vx, (size_t)l.uv.rows); }
     if (!e->f32) { pm->kx = dalloc<bf16>((size_t)pm->seq_alloc * kx); pm->vx = dalloc<bf16>((size_t)pm->seq_alloc * vx); }
@@ -691,7 +772,7 @@ int plan_prefill(Engine *e, const struct kvcache *kv, const int *toks, int n, in
         const int m = std::min(b.cap, n - i);
         starts.push_back(pos0 + i);
         LG_CHECK(cudaMemcpyAsync(b.pos, &starts.back(), 4, cudaMemcpyHostToDevice, e->stream));
-        Pass p{&b, m, true, b.toks + i, b.pos, pos0 + i};
+        Pass p{&b, m, true, b.toks + i, b.pos, pos0 + i, i == 0};
         int hi = w;
         while (hi < n_want && want[hi] < i + m) hi++;
         plan_embed_rows(e, p.toks, m, b.x);
@@ -699,8 +780,12 @@ int plan_prefill(Engine *e, const struct kvcache *kv, const int *toks, int n, in
         for (; w < hi; w += PLAN_HEAD_ROWS) {
             const int c = std::min(PLAN_HEAD_ROWS, hi - w);
             launch_k(e, lg_dn_gather_rows, dim3(c), dim3(128), 0, (const void *)b.h, (const int *)(pm->want + w), pm->hg, row_bytes);
-            if (e->f32) launch_f32(e, pm->embed, pm->hg, ldh, c, pm->wlog, pm->embed.rows);
-            else launch_dn_gemm<DN_G_F32>(e, pm->embed, pm->hg, ldh, PLAN_HEAD_ROWS, c, pm->wlog, pm->embed.rows);
+            if (e->f32) launch_f32(e, pm->embed, pm->hg, ldh, c, pm->wlog, pm->embed.rows, 1, 0, 0, 0, pm->plan->logit_scale);
+            else {
+                LgDnGemmArgs g{};
+                g.out_scale = pm->plan->logit_scale;
+                launch_dn_gemm<DN_G_F32>(e, pm->embed, pm->hg, ldh, PLAN_HEAD_ROWS, c, pm->wlog, pm->embed.rows, g);
+            }
             LG_CHECK(cudaMemcpy2DAsync(logits + (size_t)w * V, (size_t)V * 4, pm->wlog, (size_t)pm->embed.rows * 4, (size_t)V * 4, c, cudaMemcpyDeviceToHost, e->stream));
         }
         w = hi;
@@ -720,7 +805,8 @@ int plan_bench_block(Engine *e, const struct kvcache *kv, int n, int pos0, int o
     return 0;
 }
 
-const LgFamily plan_family = {"layer plan", plan_load, plan_release, plan_kv_init, plan_bind, plan_forward, plan_embed, plan_prefill, plan_bench_block};
+const LgFamily plan_family = {"layer plan", plan_load, plan_release, plan_kv_slots, plan_kv_init, plan_bind, plan_forward, plan_embed, plan_prefill, plan_bench_block,
+                              plan_start, plan_prefix};
 
 }  // namespace lg
 

@@ -234,8 +234,81 @@ static const struct rename mubopel_layer[] = {
     {"mlp.gate", "ffn_gate"}, {"mlp.up", "ffn_up"}, {"mlp.down", "ffn_down"}, {NULL, NULL}};
 static const struct rename mubopel_model[] = {{"embed", "token_embd"}, {"final.norm", "output_norm"}, {NULL, NULL}};
 
+/* Baporax: layers that add a mixer and a feed-forward (square of ReLU) of the same x, RMS norms stored as distances from 1; mixers are
+ * Mamba-2 state-space layers and sliding-window differential attention with short convolutions on q, k and v; a stretch of layers
+ * runs several times with a vector added before each pass; tied output head with scaled logits. */
+enum { BAPORAX_MAPS = 2 };
+static int jstr_is(const struct json *v, const char *s) { return v && v->type == J_STR && !strcmp(v->str, s); }
+static int jset(const struct json *o, const char *key) { const struct json *v = jget(o, key); return v && v->type != J_NULL; }
+static int baporax_configure(struct gguf_context *g, const char *prefix, const struct json *cfg) {
+    int ok = 1, n = 0;
+    const struct json *layers = jget(cfg, "layers"), *loop = jget(cfg, "loop");
+    if (layers && layers->type == J_ARR) for (const struct json *l = layers->child; l; l = l->next) n++;
+    if (!n) { fprintf(stderr, "checkpoint: config.json lists no layers\n"); return -1; }
+    meta_u32(g, prefix, "block_count", (uint32_t)n);
+    meta_u32(g, prefix, "embedding_length", (uint32_t)jint(cfg, "width", "config.json", &ok));
+    meta_u32(g, prefix, "vocab_size", (uint32_t)jint(cfg, "vocab", "config.json", &ok));
+    meta_f32(g, prefix, "logit_scale", jnum(cfg, "logit_scale", "config.json", &ok));
+    meta_f32(g, prefix, "norm.epsilon", jnum(jget(cfg, "norm"), "eps", "norm", &ok));
+    meta_f32(g, prefix, "norm.weight_offset", 1.0);
+    meta_str(g, prefix, "norm.kind", "rms");
+    meta_str(g, prefix, "block.form", "parallel");
+    meta_str(g, prefix, "feed_forward.activation", "relu2");
+    if (loop && loop->type == J_OBJ) {
+        meta_u32(g, prefix, "loop.start", (uint32_t)jint(loop, "start", "loop", &ok));
+        meta_u32(g, prefix, "loop.stop", (uint32_t)jint(loop, "stop", "loop", &ok));
+        meta_u32(g, prefix, "loop.times", (uint32_t)jint(loop, "times", "loop", &ok));
+    }
+    enum { HEADS, DIM, VDIM, KV, MAPS, WINDOW, TAPS, S_HEADS, S_VDIM, S_STATE, S_GROUPS, S_NORM, MIXER, FF, NI };
+    static const char *const leaf[NI] = {"attention.head_count", "attention.key_length", "attention.value_length", "attention.head_count_kv",
+        "attention.maps", "attention.window", "conv.taps", "ssm.head_count", "ssm.value_length", "ssm.state_size", "ssm.group_count",
+        "ssm.norm_groups", "layer.mixer", "feed_forward_length"};
+    int32_t *iv[NI];
+    for (int i = 0; i < NI; i++) iv[i] = meta_arr(g, prefix, leaf[i], GGUF_TYPE_INT32, n);
+    float *scale = meta_arr(g, prefix, "attention.scale", GGUF_TYPE_FLOAT32, n), *diff = meta_arr(g, prefix, "attention.diff", GGUF_TYPE_FLOAT32, n);
+    int L = 0;
+    for (const struct json *l = layers->child; l; l = l->next, L++) {
+        char where[32];
+        snprintf(where, sizeof where, "layer %d", L);
+        const struct json *type = jget(l, "type"), *mx = jget(l, "mixer"), *mlp = jget(l, "mlp");
+        static const struct { const char *key; int to; } attn[] = {{"heads", HEADS}, {"dim", DIM}, {"vdim", VDIM}, {"kv_heads", KV}, {"conv", TAPS}, {NULL, 0}},
+            ssm[] = {{"heads", S_HEADS}, {"vdim", S_VDIM}, {"state", S_STATE}, {"groups", S_GROUPS}, {"norm_groups", S_NORM}, {"conv", TAPS}, {NULL, 0}}, *f;
+        if (jstr_is(type, "attention")) {
+            iv[MIXER][L] = LG_MIX_GROUPED;
+            iv[MAPS][L] = BAPORAX_MAPS;
+            if (jset(mx, "mask")) {
+                iv[WINDOW][L] = jint(jget(mx, "mask"), "size", where, &ok);
+                if (iv[WINDOW][L] < 1) { fprintf(stderr, "checkpoint: %s sees no position\n", where); return -1; }
+            }
+            scale[L] = (float)jnum(mx, "scale", where, &ok);
+            diff[L] = (float)jnum(mx, "diff", where, &ok);
+            f = attn;
+        } else if (jstr_is(type, "mamba2")) {
+            iv[MIXER][L] = LG_MIX_SSM;
+            f = ssm;
+        } else {
+            fprintf(stderr, "checkpoint: %s has a mixer this library does not know: '%s'\n", where, type && type->type == J_STR ? type->str : "?");
+            return -1;
+        }
+        for (; f->key; f++) iv[f->to][L] = jint(mx, f->key, where, &ok);
+        if (mlp && mlp->type == J_OBJ) {
+            if (!jstr_is(jget(mlp, "kind"), "dense")) { fprintf(stderr, "checkpoint: %s has an unknown kind of feed-forward\n", where); return -1; }
+            iv[FF][L] = jint(mlp, "ff", where, &ok);
+        }
+    }
+    return ok ? 0 : -1;
+}
+static const struct rename baporax_layer[] = {
+    {"norm1", "attn_norm"}, {"norm2", "ffn_norm"}, {"mlp.up", "ffn_up"}, {"mlp.down", "ffn_down"}, {"mix.o", "attn_output"},
+    {"mix.q", "attn_q"}, {"mix.k", "attn_k"}, {"mix.v", "attn_v"}, {"mix.q.conv", "attn_q_conv"}, {"mix.k.conv", "attn_k_conv"},
+    {"mix.v.conv", "attn_v_conv"}, {"mix.lq1", "attn_lambda_q1"}, {"mix.lk1", "attn_lambda_k1"}, {"mix.lq2", "attn_lambda_q2"},
+    {"mix.lk2", "attn_lambda_k2"}, {"mix.in", "ssm_in"}, {"mix.conv", "ssm_conv1d"}, {"mix.conv.b", "ssm_conv1d_bias"},
+    {"mix.dt_bias", "ssm_dt_bias"}, {"mix.A_log", "ssm_a_log"}, {"mix.D", "ssm_d"}, {"mix.norm", "ssm_norm"}, {NULL, NULL}};
+static const struct rename baporax_model[] = {{"embed", "token_embd"}, {"final.norm", "output_norm"}, {"loop.step", "loop_step"}, {NULL, NULL}};
+
 static const struct ckpt_arch archs[] = {
     {"Mubopel", "mubopel", mubopel_configure, "l", mubopel_layer, mubopel_model},
+    {"Baporax", "baporax", baporax_configure, "l", baporax_layer, baporax_model},
 };
 
 /* the library's name of a checkpoint tensor (caller frees), or NULL for one the architecture does not have */

@@ -87,14 +87,16 @@ static const struct gguf_tensor *layer_tensor(const struct gguf_context *g, int 
     return gguf_find_tensor(g, name);
 }
 
-/* geometry of a model described by a layer plan: one latent row per position and layer, read by every head */
+/* geometry of a model described by a layer plan: latent rows are one per position, read by every head; a state-space layer caches
+ * no rows */
 static int plan_geometry(struct model *m, const struct gguf_context *g) {
     struct lg_plan *p = lg_plan_read(g);
     if (!p) return -1;
     for (int L = 0; L < p->n_layer; L++) {
         m->ffn_len[L] = p->layer[L].ff;
         m->head_dim[L] = p->layer[L].dim + p->layer[L].rot_dim;
-        m->n_head_kv[L] = 1;
+        m->n_head_kv[L] = p->layer[L].mixer == LG_MIX_GROUPED ? p->layer[L].kv_heads : p->layer[L].mixer == LG_MIX_SSM ? 0 : 1;
+        m->is_local[L] = p->layer[L].window > 0;
     }
     lg_plan_free(p);
     return 0;
