@@ -4,7 +4,7 @@
     python bench.py [--gpus N] [--steps K] [--warmup W] [--impl ours|reference]
                     [--config b12|b12k|e4b|tiny|c5] [--depth D] [--p P] [--mtp-n M]
     python bench.py --sweep e4b|b12|b12k [--sweep-out FILE.md]
-    python bench.py --design mubopel [--design-out FILE.md]
+    python bench.py --design mubopel|baporax [--design-out FILE.md]
 
 One "step" is one MTP round at batch 1: M-1 draft-head forwards, one M-token verify forward of
 the target (every weight streamed once), greedy acceptance and position advance -- all on the
@@ -462,6 +462,137 @@ def design(a, lg, synth, torch):
     print(json.dumps({"design": "mubopel", "results": out}), flush=True)
 
 
+# ---------------------------------------------------------------------------------------------
+# the state-space / windowed-attention design beside the latent-attention one
+# ---------------------------------------------------------------------------------------------
+def hybrid_shapes(synth, name):
+    """({kind of layer: shape of a model of such layers}, latent-attention shape) of equal width, feed-forward, layers and vocabulary"""
+    ls = design_shapes(synth, name)[0]
+    W, ff, n = ls.width, ls.layers[0].ff, len(ls.layers)
+    H, G, win = {"2b": (16, 4, 1024), "8b": (32, 8, 2048), "16b": (64, 8, 2048)}[name]
+    ssm = synth.SsmLayer(heads=2 * W // 64, vdim=64, state=128, groups=8, norm_groups=8, conv=4, ff=ff)
+    att = synth.DiffLayer(heads=H, kv_heads=G, dim=64, vdim=128, window=win, conv=4, ff=ff)
+    return {k: synth.HybridShape(width=W, vocab=ls.vocab, layers=[l] * n) for k, l in (("state-space", ssm), ("windowed", att))}, ls
+
+
+def hybrid_model(lg, synth, torch, path, shape, n_pf, depths, peaks):
+    """One model of one kind of layer: whole-step and per-class device times with algorithmic bytes or operations."""
+    l, L, W, V = shape.layers[0], len(shape.layers), shape.width, shape.vocab
+    hbm, tc = float(peaks.get("hbm_gbs", 6650.0)) * 1e9, float(peaks.get("bf16_tflops_sustained", 1400.0)) * 1e12
+    ssm = l.type == "mamba2"
+    t = l.tensors(W)
+    in_cols = t["in"][0] if ssm else t["q"][0] + t["k"][0] + t["v"][0]
+    at = t["o"][1]
+    state = l.heads * l.vdim * l.state * 4 if ssm else 0
+    conv_ch = at + 2 * l.groups * l.state if ssm else in_cols
+    row = 0 if ssm else 2 * (t["k"][0] + t["v"][0])
+    seen = lambda d: 0 if ssm else min(d, l.window)
+    par = {"in + up": (W * (in_cols + l.ff), C_QKV), "o + down": (W * (at + l.ff), C_O)}
+    res = {"decode": {}, "prefill": {}}
+    with lg.Session(path, None, max(depths) + 1024) as s:
+        tm = DesignTimer(torch, s)
+        prompt = synth.prompt_ids(max(depths), V, seed=11)
+        for d in depths:
+            s.prefill(prompt[:d - 1], 0)
+            first = s.next(int(prompt[d - 1]), d - 1)
+            s.rounds_begin(first, d, 1)
+            s.rounds_enqueue(1, 0, 16)
+            s.rounds_collect()
+            clk = ClockSampler()
+            clk.start()
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            torch.cuda.synchronize()
+            e0.record(tm.stream)
+            s.rounds_enqueue(1, 0, 256)
+            e1.record(tm.stream)
+            e1.synchronize()
+            ms = e0.elapsed_time(e1) / 256
+            mix = 2 * state + seen(d) * row
+            byts = 2.0 * (L * sum(p for p, _ in par.values()) + W * V) + L * mix
+            r = {"step": {"us": ms * 1e3, "tok_s": 1e3 / ms, "frac": byts / (ms * 1e-3) / hbm}, "clocks": clk.stop()}
+            s.rounds_collect()
+            for name, (p, c) in par.items():
+                us = tm(lambda c=c: s.matmul_pass(1, c)) * 1e3 / L
+                r[name] = {"us": us, "frac": 2.0 * p / (us * 1e-6) / hbm}
+            us = tm(lambda: s.matmul_pass(1, C_HEAD)) * 1e3
+            r["head"] = {"us": us, "frac": 2.0 * W * V / (us * 1e-6) / hbm}
+            us = tm(lambda: s.matmul_pass(1, C_ATTN)) * 1e3 / L
+            r["mixer"] = {"us": us, "frac": mix / (us * 1e-6) / hbm}
+            us = tm(lambda: s.matmul_pass(1, C_EXPAND)) * 1e3 / L
+            r["gated norm" if ssm else "conv"] = {"us": us}
+            r["norms"] = {"us": tm(lambda: s.matmul_pass(1, C_NORM)) * 1e3 / L}
+            res["decode"][d] = r
+        for n in n_pf:
+            s.prefill(prompt[:n], 0)
+            torch.cuda.synchronize()
+            t0 = time.perf_counter()
+            for _ in range(3):
+                s.prefill(prompt[:n], 0)
+            torch.cuda.synchronize()
+            ms = (time.perf_counter() - t0) / 3 * 1e3
+            if ssm:                                            # the recurrence itself: update and read of the state
+                mixer_fl, mixer_by = 4.0 * n * l.heads * l.vdim * l.state, 2.0 * n * (2 * at + 2 * l.groups * l.state)
+            else:
+                w = min(n, l.window)
+                mixer_fl, mixer_by = (n * w - w * (w - 1) / 2) * 4 * l.heads * (l.dim + l.vdim), 0.0
+            fl = 2.0 * L * n * W * (in_cols + l.ff + at + l.ff) + L * mixer_fl
+            r = {"prompt": {"ms": ms, "tok_s": n / ms * 1e3, "frac": fl / (ms * 1e-3) / tc}}
+            for name, c, p in (("in", C_QKV, W * in_cols), ("up", C_GATEUP, W * l.ff), ("o + down", C_O, W * (at + l.ff))):
+                us = tm(lambda c=c: s.prefill_pass(n, c)) * 1e3 / L
+                r[name] = {"us": us, "frac": 2.0 * n * p / (us * 1e-6) / tc}
+            us = tm(lambda: s.prefill_pass(n, C_ATTN)) * 1e3 / L
+            r["mixer"] = {"us": us, "frac": mixer_by / (us * 1e-6) / hbm if ssm else mixer_fl / (us * 1e-6) / tc}
+            us = tm(lambda: s.prefill_pass(n, C_EXPAND)) * 1e3 / L
+            r["conv + gated norm" if ssm else "conv"] = {"us": us, "frac": 2.0 * n * (2 * conv_ch + (3 * at if ssm else 0)) / (us * 1e-6) / hbm}
+            r["norms"] = {"us": tm(lambda: s.prefill_pass(n, C_NORM)) * 1e3 / L}
+            res["prefill"][n] = r
+    return res
+
+
+def hybrid(a, lg, synth, torch):
+    peaks = load_peaks()
+    lines = ["# The state-space / windowed-attention design beside the latent-attention one", "",
+             "`python bench.py --design baporax`: random weights, batch 1, one model of each kind of layer (`state-space`, `windowed`) and a Mubopel model",
+             "(`latent`) of equal width, feed-forward, layers and vocabulary, all bf16.  `frac` = algorithmic bytes (decode; state-space prompts, the",
+             "convolution and the gated norm) or operations (prefill) over device time, of the measured copy bandwidth",
+             f"({peaks.get('hbm_gbs')} GB/s) or sustained bf16 throughput ({peaks.get('bf16_tflops_sustained')} TFLOP/s).  Times are per layer, all layers' launches",
+             "of a class back to back, L2 overwritten before each pass; the prompt is one block of 2048 tokens from position 0.", ""]
+    out = {}
+    show = lambda x: "" if not x else (f"{x['tok_s']:.0f} tok/s ({x.get('ms', x.get('us', 0) / 1e3):.2f} ms)" if "tok_s" in x else f"{x['us']:.1f} us") + \
+        (f", {x['frac']:.3f}" if "frac" in x else "")
+    for name in a.design_sizes.split(","):
+        hs, ls = hybrid_shapes(synth, name)
+        depths, n_pf = [1024, 8192], [2048]
+        both = {}
+        for k, sh in hs.items():
+            path = os.path.join(CACHE, f"baporax_{k}_{name}")
+            if not os.path.exists(os.path.join(path, "config.json")):
+                synth.write_checkpoint(path, sh, 0, fast=True)
+            both[k] = hybrid_model(lg, synth, torch, path, sh, n_pf, depths, peaks)
+        if not a.design_alone:
+            path = os.path.join(CACHE, f"mubopel_{name}")
+            if not os.path.exists(os.path.join(path, "config.json")):
+                synth.write_checkpoint(path, ls, 0, fast=True)
+            both["latent"] = design_model(a, lg, synth, torch, path, True, ls, n_pf, depths, peaks)
+        out[name] = both
+        sl, wl = hs["state-space"].layers[0], hs["windowed"].layers[0]
+        lines += [f"## {name}: width {ls.width}, ff {sl.ff}, {len(ls.layers)} layers; state-space {sl.heads} x {sl.vdim}, state {sl.state}; "
+                  f"windowed {wl.heads} heads over {wl.kv_heads}, 2 x {wl.dim} / {wl.vdim}, window {wl.window}", ""]
+        for kind in ("decode", "prefill"):
+            for d in (depths if kind == "decode" else n_pf):
+                lines += [f"### {kind} {d}", "", "| model | " + " | ".join(["class: time, frac"]) + " |", "|---|---|"]
+                for k, v in both.items():
+                    lines.append(f"| {k} | " + "; ".join(f"{c}: {show(x)}" for c, x in v[kind][d].items() if c != "clocks") + " |")
+                lines.append("")
+        lines += [f"clocks ({k}): {v['decode'][1024]['clocks']}" for k, v in both.items()] + [""]
+    text = "\n".join(lines)
+    if a.design_out:
+        with open(a.design_out, "w") as f:
+            f.write(text + "\n")
+    print(text, flush=True)
+    print(json.dumps({"design": "baporax", "results": out}), flush=True)
+
+
 def load_peaks():
     try:
         return json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json")))
@@ -527,9 +658,9 @@ def main():
     ap.add_argument("--profile-prefill", type=int, default=None, metavar="CLASSES",
                     help="short path for profilers: load, model_prefill of 512 tokens, 3 wide prompt blocks of 256 tokens "
                          "restricted to kernel classes (4 = gate/up matmul, 1023 = everything), exit")
-    ap.add_argument("--design", default=None, choices=["mubopel"], help="time a design beside the block-quantised family instead of the benchmark line")
+    ap.add_argument("--design", default=None, choices=["mubopel", "baporax"], help="time a design beside its closest one instead of the benchmark line")
     ap.add_argument("--design-sizes", default="2b,8b,16b")
-    ap.add_argument("--design-alone", action="store_true", help="with --design: leave the block-quantised family out")
+    ap.add_argument("--design-alone", action="store_true", help="with --design: leave the other family out")
     ap.add_argument("--design-out", default=None, help="with --design: also write the table to this file")
     ap.add_argument("--layers", type=int, default=0, help="cut the model to this many layers (small profiling cases)")
     a = ap.parse_args()
@@ -586,7 +717,7 @@ def main():
     if RANK == 0:
         build.build()
     if a.design:
-        design(a, lg, synth, torch)
+        (hybrid if a.design == "baporax" else design)(a, lg, synth, torch)
         return
     if a.sweep:
         sweep(a, lg, synth, torch)

@@ -181,6 +181,17 @@ int  lg_latent_attn_host(const float *q, const float *cache, const float *sink, 
 int  lg_latent_prompt_attn_host(const float *q, const float *k, const float *k_rot, const float *v, const float *gate, const float *sink,
                                 int n, int H, int dim, int rot_dim, int vdim, int pos, float scale, float *out);
 
+/* Layers whose mixer and feed-forward run side by side.  The stacked input projections: out = w x [n][m], act = relu(w_up x_up)^2
+ * [n][m_up]; x += add + bias (either may be NULL) and the RMS norms of x with two weights; a mixer between its projections, run
+ * block by block on projected rows (see lg_plan.cu; -2: sizes the kernels do not hold). */
+struct lg_plan_layer;
+int  lg_dense_pair_host(const float *w, int m, const float *w_up, int m_up, int k, const float *x, const float *x_up, int n, int f32,
+                        float *out, float *act);
+int  lg_row_norm_pair_host(float *x, int rows, int n, const float *add, const float *bias, const float *norm_w, const float *norm_w2, float eps,
+                           int f32, float *y, float *y2);
+int  lg_mixer_blocks_host(const struct lg_plan_layer *layer, float eps, int max_seq, const float *const *w, const float *rows, int total,
+                          const int *pos, const int *m, int n_blocks, int plain, int f32, float *out);
+
 /* Split-KV flash-decode for callers that cannot allocate device memory (a captured stream, a
  * serving loop whose memory was fixed at start-up, a process whose allocator owns the device).
  * Same kernel as lg_flash_decode_host, but every pointer is a DEVICE pointer supplied by the

@@ -33,7 +33,17 @@ ABI_SYMBOLS = [
     "lg_debug_bounded_wait", "lg_debug_stamps", "lg_debug_clear_stamps", "lg_matmul_resid_host",
     "lg_dequant_host", "lg_gemv_host", "lg_flash_decode_host", "lg_flash_decode_cluster_host", "lg_prefill_matmul_host",
     "lg_dense_matmul_host", "lg_row_norm_host", "lg_latent_attn_host", "lg_latent_prompt_attn_host",
+    "lg_dense_pair_host", "lg_row_norm_pair_host", "lg_mixer_blocks_host",
 ]
+
+class PlanLayer(C.Structure):
+    """struct lg_plan_layer of include/lg_plan.h"""
+    _fields_ = [(n, C.c_int) for n in ("mixer", "heads", "dim", "rot_dim", "vdim", "q_rank", "kv_rank", "kv_src", "rot_dims")] + \
+               [("scale", C.c_float), ("rot_base", C.c_float)] + [(n, C.c_int) for n in ("ff", "kv_heads", "maps", "window", "taps")] + \
+               [("diff", C.c_float)] + [(n, C.c_int) for n in ("state", "groups", "norm_groups")]
+
+
+MIX_LATENT, MIX_GROUPED, MIX_SSM = 1, 2, 3
 
 _lib = None
 
@@ -112,7 +122,10 @@ def load() -> C.CDLL:
     for name, args in (("lg_dense_matmul_host", [f, vp, i, i, f, i, i, f]),
                        ("lg_row_norm_host", [f, i, i, vp, vp, fl, f, fl, i, i, f]),
                        ("lg_latent_attn_host", [f, f, f, i, i, i, i, i, i, fl, i, i, f]),
-                       ("lg_latent_prompt_attn_host", [f, f, f, f, f, f, i, i, i, i, i, i, fl, f])):
+                       ("lg_latent_prompt_attn_host", [f, f, f, f, f, f, i, i, i, i, i, i, fl, f]),
+                       ("lg_dense_pair_host", [f, i, f, i, i, f, f, i, i, f, f]),
+                       ("lg_row_norm_pair_host", [f, i, i, vp, vp, f, f, fl, i, f, f]),
+                       ("lg_mixer_blocks_host", [C.POINTER(PlanLayer), fl, i, C.POINTER(vp), f, i, _i32p, _i32p, i, i, i, f])):
         getattr(L, name).argtypes = args
         getattr(L, name).restype = i
     _lib = L
@@ -228,6 +241,37 @@ def latent_prompt_attn(q, k, k_rot, v, gate, sink, pos: int, scale: float) -> np
     out = np.empty((n, H, v.shape[2]), dtype=np.float32)
     _ok(load().lg_latent_prompt_attn_host(q.reshape(-1), k.reshape(-1), k_rot.reshape(-1), v.reshape(-1), gate.reshape(-1), sink, n, H, k.shape[2],
                                           k_rot.shape[1], v.shape[2], pos, scale, out.reshape(-1)), "latent_prompt_attn")
+    return out
+
+
+def dense_pair(w, w_up, x, x_up, f32: bool = False):
+    """(w x[tok], relu(w_up x_up[tok])^2) as the stacked input projections of a layer compute them."""
+    w, u, x, xu = map(_f32, (w, w_up, x, x_up))
+    out, act = np.empty((len(x), len(w)), np.float32), np.empty((len(x), len(u)), np.float32)
+    _ok(load().lg_dense_pair_host(w.reshape(-1), len(w), u.reshape(-1), len(u), w.shape[1], x.reshape(-1), xu.reshape(-1), len(x), int(f32),
+                                  out.reshape(-1), act.reshape(-1)), "dense_pair")
+    return out, act
+
+
+def row_norm_pair(x, norm_w, norm_w2, eps: float, add=None, bias=None, f32: bool = False):
+    """(x + add + bias, its RMS norm times norm_w, times norm_w2) through the residual / norm kernel."""
+    x, w1, w2 = np.array(x, dtype=np.float32, order="C", copy=True), _f32(norm_w), _f32(norm_w2)
+    a, b = None if add is None else _f32(add), None if bias is None else _f32(bias)
+    y, y2 = np.empty_like(x), np.empty_like(x)
+    _ok(load().lg_row_norm_pair_host(x.reshape(-1), x.shape[0], x.shape[1], _ptr(a), _ptr(b), w1, w2, eps, int(f32), y.reshape(-1), y2.reshape(-1)), "row_norm_pair")
+    return x, y, y2
+
+
+def mixer_blocks(layer: PlanLayer, weights, rows, blocks, eps: float, max_seq: int = 0, plain: bool = False, f32: bool = False) -> np.ndarray:
+    """A grouped-attention or state-space mixer on projected rows [total, columns], run in blocks [(position, tokens), ...]: what its
+    output product reads, [total, heads * vdim] (positions run more than once: of the last time)."""
+    rows = _f32(rows)
+    weights = [_f32(w) for w in weights]
+    ptrs = (C.c_void_p * len(weights))(*[w.ctypes.data for w in weights])
+    pos, m = (np.ascontiguousarray([b[i] for b in blocks], dtype=np.int32) for i in (0, 1))
+    out = np.zeros((len(rows), layer.heads * layer.vdim), dtype=np.float32)
+    _ok(load().lg_mixer_blocks_host(C.byref(layer), eps, max(max_seq, len(rows)), ptrs, rows.reshape(-1), len(rows), pos, m, len(pos), int(plain), int(f32),
+                                    out.reshape(-1)), "mixer_blocks")
     return out
 
 

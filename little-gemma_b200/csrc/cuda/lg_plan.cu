@@ -1003,3 +1003,147 @@ extern "C" int lg_latent_prompt_attn_host(const float *q, const float *k, const 
     s.pm.kx = s.pm.vx = nullptr;
     return 0;
 }
+
+// Input projections of a layer whose branches run side by side: out = w x [n][m], act = relu(w_up x_up)^2 [n][m_up].
+extern "C" int lg_dense_pair_host(const float *w, int m, const float *w_up, int m_up, int k, const float *x, const float *x_up, int n, int f32,
+                                  float *out, float *act) {
+    if (m < 1 || m_up < 1 || k < 1 || n < 1) return -1;
+    Scratch s(f32 != 0);
+    Engine *e = &s.e;
+    const int r0 = up(m, 32), r1 = up(m_up, 32), xr = up(n, 128), ld = up(k, 64);
+    MatBuild b(e, r0 + r1, k);
+    for (int r = 0; r < m; r++) for (int i = 0; i < k; i++) b.put((size_t)r * b.ldk + i, w[(size_t)r * k + i]);
+    for (int r = 0; r < m_up; r++) for (int i = 0; i < k; i++) b.put((size_t)(r0 + r) * b.ldk + i, w_up[(size_t)r * k + i]);
+    const DMat both = b.upload(e), a = rows_of(e, both, 0, r0), u = rows_of(e, both, r0, r1);
+    s.mem.push_back(both.w);
+    void *dx = s.rows(x, n, k, xr, ld), *du = s.rows(x_up, n, k, xr, ld);
+    float *o = s.put<float>(nullptr, (size_t)xr * r0), *g = s.put<float>(nullptr, (size_t)xr * r1);
+    void *ac = s.put<uint8_t>(nullptr, (size_t)xr * r1 * s.es());
+    if (f32) {
+        launch_f32(e, a, dx, ld, n, o, r0);
+        launch_f32(e, u, du, ld, n, g, r1);
+        launch_k(e, lg_dn_relu2_rows, dim3((r1 + 255) / 256, n), dim3(256), 0, (const float *)g, r1, r1, (float *)ac, r1);
+    } else if (n > LG_MAXM) {
+        launch_dn_gemm<DN_G_F32>(e, a, dx, ld, xr, n, o, r0);
+        launch_dn_gemm<DN_G_RELU2>(e, u, du, ld, xr, n, ac, r1);
+    } else {
+        LgDnGemvArgs v{};
+        v.x = (const bf16 *)dx; v.x2 = (const bf16 *)du; v.ldx = ld; v.M = n; v.split_tile = r0 / 16; v.out = o; v.ldo = r0; v.outh = (bf16 *)ac; v.ldoh = r1;
+        launch_dn_gemv<DN_PAIR, false>(e, both, v);
+    }
+    const std::vector<float> ro = s.get(o, (size_t)n * r0, true), ra = s.get(ac, (size_t)n * r1, f32 != 0);
+    for (int i = 0; i < n; i++) {
+        memcpy(out + (size_t)i * m, &ro[(size_t)i * r0], (size_t)m * 4);
+        memcpy(act + (size_t)i * m_up, &ra[(size_t)i * r1], (size_t)m_up * 4);
+    }
+    return 0;
+}
+
+// x += add + bias (either may be null), then the RMS norms of x with two weights.
+extern "C" int lg_row_norm_pair_host(float *x, int rows, int n, const float *add, const float *bias, const float *norm_w, const float *norm_w2, float eps,
+                                     int f32, float *y, float *y2) {
+    if (rows < 1 || n < 1 || n > 16 * 1024 || !norm_w || !norm_w2) return -1;
+    Scratch s(f32 != 0);
+    LgRowNormArgs a{};
+    a.x = s.put(x, (size_t)rows * n); a.ldx = a.n = n;
+    if (add) { a.add = s.put(add, (size_t)rows * n); a.ld_add = n; }
+    if (bias) a.bias = s.put(bias, n);
+    a.norm_w = s.put(norm_w, n); a.norm_w2 = s.put(norm_w2, n); a.eps = eps; a.ldy = up(n, 64);
+    a.y = s.put<uint8_t>(nullptr, (size_t)rows * a.ldy * s.es()); a.y2 = s.put<uint8_t>(nullptr, (size_t)rows * a.ldy * s.es());
+    launch_row_norm_par(&s.e, rows, a);
+    const std::vector<float> r = s.get(a.y, (size_t)rows * a.ldy, f32 != 0), r2 = s.get(a.y2, (size_t)rows * a.ldy, f32 != 0);
+    for (int i = 0; i < rows; i++) {
+        memcpy(y + (size_t)i * n, &r[(size_t)i * a.ldy], (size_t)n * 4);
+        memcpy(y2 + (size_t)i * n, &r2[(size_t)i * a.ldy], (size_t)n * 4);
+    }
+    LG_CHECK(cudaMemcpy(x, a.x, (size_t)rows * n * 4, cudaMemcpyDeviceToHost));
+    return 0;
+}
+
+// A mixer between its projections, block by block: rows [total][projected columns without padding] (grouped: q | k | v; state-space:
+// z | x | B | C | step sizes) -> out [total][heads vdim], what the output product would read.  Block b runs tokens pos[b] .. pos[b] + m[b]
+// (more than 8: as a prompt block), in the order given, so that positions can be run again.  w: grouped { q, k, v filters, lq1, lk1,
+// lq2, lk2 }, state-space { filters, filter bias, dt_bias, A_log, D, norm weight }.  plain != 0: the kernels that hold every size.
+extern "C" int lg_mixer_blocks_host(const struct lg_plan_layer *layer, float eps, int max_seq, const float *const *w, const float *rows, int total,
+                                    const int *pos, const int *m, int n_blocks, int plain, int f32, float *out) {
+    if (layer->mixer != LG_MIX_GROUPED && layer->mixer != LG_MIX_SSM) return -1;
+    Scratch s(f32 != 0);
+    Engine *e = &s.e;
+    struct lg_plan plan{};
+    struct lg_plan_layer pl = *layer;
+    pl.ff = 0;
+    plan.n_layer = 1; plan.width = 32; plan.vocab = 1; plan.layer = &pl; plan.form = LG_FORM_PARALLEL; plan.norm_eps = eps;
+    s.pm.plan = &plan;
+    s.pm.L.resize(1);
+    PlanLayer &l = s.pm.L[0];
+    l.p = pl; l.eps = eps;
+    seq_layer_sizes(l);
+    SeqWeights sw;
+    auto take = [](const float *p, size_t n) { return std::vector<float>(p, p + n); };
+    const int H = pl.heads, G = pl.kv_heads, M = pl.maps, inner = H * pl.vdim, gn = pl.groups * pl.state;
+    const bool attn = pl.mixer == LG_MIX_GROUPED;
+    if (attn) {
+        const int ch[3] = {H * M * pl.dim, G * M * pl.dim, G * pl.vdim};
+        for (int i = 0; i < 3; i++) sw.conv[i] = take(w[i], (size_t)ch[i] * pl.taps);
+        if (M == 2) for (int i = 0; i < 4; i++) sw.lam[i] = take(w[3 + i], pl.dim);
+    } else {
+        sw.conv[0] = take(w[0], (size_t)(inner + 2 * gn) * pl.taps); sw.conv_b = take(w[1], inner + 2 * gn);
+        sw.dt_bias = take(w[2], H); sw.a_log = take(w[3], H); sw.d = take(w[4], H); sw.norm = take(w[5], inner);
+    }
+    if (!seq_layer_weights(e, 0, l, sw)) { seq_layer_free(l); return -2; }
+    if (plain) { l.chunked = 0; l.rt = 0; }
+    l.act_off = up(l.at_cols, 64);
+    l.in.rows = l.in_rows; l.in.ldk = 64; l.o.ldk = l.act_off;
+    int cap = 128, bad = 0;
+    for (int b = 0; b < n_blocks; b++) { cap = std::max(cap, up(m[b], 128)); bad |= m[b] < 1 || m[b] > PLAN_BLOCK || pos[b] < 0 || pos[b] + m[b] > std::min(total, max_seq); }
+    if (bad) { seq_layer_free(l); return -1; }
+    int kv_dim = 0, seq = 0, f16 = 0;
+    void *k = nullptr, *v = nullptr;
+    struct kvcache kv{};
+    kv.n_layer = 1; kv.max_seq = max_seq; kv.kv_dim = &kv_dim; kv.seq = &seq; kv.f16 = &f16; kv.k = &k; kv.v = &v;
+    seq_kv_init(&kv, &plan, f32 != 0);
+    LG_CHECK(cudaDeviceSynchronize());
+    s.pm.seq_alloc = up(max_seq, 128);
+    seq_bind(e, &kv);
+    e->x = nullptr;
+    PlanBuf nb, wb;
+    seq_buf_alloc(e, nb, LG_MAXM, true);
+    seq_buf_alloc(e, wb, cap, false);
+    // where unpadded column c of a projection row goes
+    std::vector<int> at;
+    auto sections = [&](int first, int n, int per, int to) { for (int i = 0; i < n; i++) for (int j = 0; j < per; j++) at.push_back(first + i * to + j); };
+    if (attn) { sections(0, H * M, pl.dim, l.dimp); sections(l.q_cols, G * M, pl.dim, l.dimp); sections(l.q_cols + l.k_cols, G, pl.vdim, l.vdp); }
+    else { sections(0, H, pl.vdim, l.vdp); sections(l.ch0, H, pl.vdim, l.vdp); sections(l.ch0 + H * l.vdp, 2 * pl.groups, pl.state, l.np); sections(l.dt_off, 1, H, H); }
+    const int cols = (int)at.size();
+    int *d_pos = s.put<int>(nullptr, 1);
+    for (int b = 0; b < n_blocks; b++) {
+        const bool wide = m[b] > LG_MAXM;
+        PlanBuf &pb = wide ? wb : nb;
+        std::vector<float> pad((size_t)m[b] * l.in_rows, 0.0f), dt((size_t)m[b] * std::max(1, l.in_rows - l.dt_off), 0.0f);
+        for (int t = 0; t < m[b]; t++)
+            for (int c = 0; c < cols; c++) {
+                const float x = rows[(size_t)(pos[b] + t) * cols + c];
+                pad[(size_t)t * l.in_rows + at[c]] = x;
+                if (at[c] >= l.dt_off) dt[(size_t)t * (l.in_rows - l.dt_off) + at[c] - l.dt_off] = x;
+            }
+        if (wide && !f32) {
+            std::vector<uint16_t> h(pad.size());
+            for (size_t i = 0; i < pad.size(); i++) h[i] = bf16_bits(pad[i]);
+            h2d_sync(pb.pj, h.data(), h.size() * 2);
+            if (!attn) h2d_sync(pb.dt, dt.data(), dt.size() * 4);
+        } else h2d_sync(pb.pj, pad.data(), pad.size() * 4);
+        h2d_sync(d_pos, &pos[b], 4);
+        Pass p{&pb, m[b], wide, nullptr, d_pos, pos[b]};
+        launch_k(e, lg_seq_begin_kernel, dim3(1), dim3(32), 0, seq_ctl(&kv), (const int *)d_pos, m[b], wide ? 1 : 0, e->err);
+        seq_mixer(e, &kv, l, 0, p, C_ALL);
+        const std::vector<float> r = s.get(pb.at, (size_t)m[b] * l.o.ldk, f32 != 0);
+        for (int t = 0; t < m[b]; t++)
+            for (int h = 0; h < H; h++)
+                memcpy(out + ((size_t)(pos[b] + t) * H + h) * pl.vdim, &r[(size_t)t * l.o.ldk + h * l.vdp], (size_t)pl.vdim * 4);
+    }
+    seq_layer_free(l);
+    buf_free(nb, true); buf_free(wb, false);
+    cudaFree(k); cudaFree(v); cudaFree(s.pm.part); cudaFree(s.pm.part_ml);
+    s.pm.part = nullptr; s.pm.part_ml = nullptr; s.pm.plan = nullptr;
+    return 0;
+}

@@ -17,13 +17,16 @@ void put_sections(std::vector<float> &dst, size_t at, const std::vector<float> &
     for (int s = 0; s < sections; s++)
         for (int i = 0; i < per; i++) dst[at + (size_t)s * to + i] = src[from + (size_t)s * per + i];
 }
-// filter rows of a convolution [channels][taps], channels first_ch .. in padded sections, as [taps][nch]
-void put_taps(std::vector<float> &dst, int nch, int at, const struct gguf_tensor *t, int from, int sections, int per, int to, int taps) {
+// filters [channels][taps], channels from .. in padded sections, as [taps][nch]
+void put_taps(std::vector<float> &dst, int nch, int at, const std::vector<float> &f, int from, int sections, int per, int to, int taps) {
     for (int s = 0; s < sections; s++)
-        for (int i = 0; i < per; i++) {
-            const std::vector<float> f = row_f32(t, from + s * per + i);
-            for (int j = 0; j < taps; j++) dst[(size_t)j * nch + at + s * to + i] = f[j];
-        }
+        for (int i = 0; i < per; i++)
+            for (int j = 0; j < taps; j++) dst[(size_t)j * nch + at + s * to + i] = f[(size_t)(from + s * per + i) * taps + j];
+}
+std::vector<float> mat_f32(const struct gguf_tensor *t) {
+    std::vector<float> f;
+    for (int r = 0; r < (int)t->dims[1]; r++) { const std::vector<float> row = row_f32(t, r); f.insert(f.end(), row.begin(), row.end()); }
+    return f;
 }
 // rows [row0, row0 + rows) of a matrix as a matrix of its own
 DMat rows_of(const Engine *e, const DMat &m, int row0, int rows) {
@@ -79,64 +82,83 @@ int seq_rows(const PlanLayer &l, int max_seq) {
     return l.p.window > 0 ? (int)std::min<long long>(all, ((long long)l.p.window + PLAN_BLOCK + 64 + 127) / 128 * 128) : all;
 }
 
+// What a mixer holds besides its projections: filters [channels][taps] (of q, k, v, or of x | B | C), and the vectors of its kind.
+struct SeqWeights { std::vector<float> conv[3], conv_b, dt_bias, a_log, d, norm, lam[4]; };
+
+// false, after a message: sizes beyond what the kernels hold
+bool seq_layer_weights(const Engine *e, int i, PlanLayer &l, const SeqWeights &w) {
+    const struct lg_plan_layer &p = l.p;
+    const int H = p.heads, G = p.kv_heads, M = p.maps;
+    std::vector<float> cw((size_t)p.taps * l.nch, 0.0f);
+    bool ok = true;
+    if (p.mixer == LG_MIX_GROUPED) {
+        put_taps(cw, l.nch, 0, w.conv[0], 0, H * M, p.dim, l.dimp, p.taps);
+        put_taps(cw, l.nch, l.q_cols, w.conv[1], 0, G * M, p.dim, l.dimp, p.taps);
+        put_taps(cw, l.nch, l.q_cols + l.k_cols, w.conv[2], 0, G, p.vdim, l.vdp, p.taps);
+        l.out_mult = 1.0f;
+        if (M == 2) {                        // weight of the second map
+            double s[2] = {0.0, 0.0};
+            for (int j = 0; j < 2; j++) for (int d = 0; d < p.dim; d++) s[j] += (double)w.lam[2 * j][d] * w.lam[2 * j + 1][d];
+            l.lambda = (float)(exp(s[0]) - exp(s[1]) + (double)p.diff);
+            l.out_mult = 1.0f - p.diff;
+        }
+        if (l.vdp > (M == 1 ? 256 : 128) || lg_win_pf_smem(M, l.dimp, l.vdp) > PLAN_SMEM_SMALL) l.chunked = 0;
+        l.rt = !e->f32 && l.vdp <= 256 && lg_win_dec_smem(M, l.dimp, l.vdp) <= PLAN_SMEM_MAX;
+        ok = (size_t)(M * (l.dimp + l.vdp) + M * 128) * 4 <= PLAN_SMEM_SMALL;
+    } else {
+        const int inner = H * p.vdim, gn = p.groups * p.state, part_n = inner / p.norm_groups;
+        const int part[3][5] = {{0, 0, H, p.vdim, l.vdp}, {H * l.vdp, inner, p.groups, p.state, l.np}, {H * l.vdp + p.groups * l.np, inner + gn, p.groups, p.state, l.np}};
+        std::vector<float> cb(l.nch, 0.0f), gn_w((size_t)H * l.vdp, 0.0f);
+        for (auto &q : part) {                                             // x, B, C
+            put_taps(cw, l.nch, q[0], w.conv[0], q[1], q[2], q[3], q[4], p.taps);
+            put_sections(cb, q[0], w.conv_b, q[1], q[2], q[3], q[4]);
+        }
+        put_sections(gn_w, 0, w.norm, 0, H, p.vdim, l.vdp);
+        l.conv_b = upload_f32(cb.data(), cb.size());
+        l.dt_bias = upload_f32(w.dt_bias.data(), H); l.a_log = upload_f32(w.a_log.data(), H); l.d = upload_f32(w.d.data(), H);
+        l.gnorm = upload_f32(gn_w.data(), gn_w.size());
+        ok = l.npl && part_n <= (p.vdim % 4 || part_n % 4 ? 16 : 32) * 1024;
+        l.vs = std::min(l.vdp, 128);
+        if (lg_ssd_out_smem(l.np, l.vs) > PLAN_SMEM_SMALL) l.vs = std::min(l.vdp, 64);
+        if (l.np > 256 || lg_ssd_out_smem(l.np, l.vs) > PLAN_SMEM_MAX - 2048 || lg_ssd_state_smem(l.np, l.vs) > PLAN_SMEM_MAX - 2048) l.chunked = 0;
+    }
+    l.conv_w = upload_f32(cw.data(), cw.size());
+    if (!ok) fprintf(stderr, "lg_b200: layer %d: sizes beyond what the kernels hold\n", i);
+    return ok;
+}
+
 void seq_layer_load(Engine *e, int i, PlanLayer &l) {
     PlanModel *pm = e->plan;
     const struct lg_plan *P = pm->plan;
     const struct lg_plan_layer &p = l.p;
-    const int W = P->width, H = p.heads, G = p.kv_heads;
-    std::vector<float> cw((size_t)p.taps * l.nch, 0.0f);
+    const int W = P->width, H = p.heads, G = p.kv_heads, M = p.maps;
+    SeqWeights w;
     MatBuild b(e, l.in_rows + (p.ff ? up(l.ffp, 32) : 0), W);
     if (p.mixer == LG_MIX_GROUPED) {
-        const int M = p.maps;
         put_groups(b, 0, need(e, i, "attn_q", H * M * p.dim, W), H * M, p.dim, l.dimp);
         put_groups(b, l.q_cols, need(e, i, "attn_k", G * M * p.dim, W), G * M, p.dim, l.dimp);
         put_groups(b, l.q_cols + l.k_cols, need(e, i, "attn_v", G * p.vdim, W), G, p.vdim, l.vdp);
-        put_taps(cw, l.nch, 0, need(e, i, "attn_q_conv", H * M * p.dim, p.taps), 0, H * M, p.dim, l.dimp, p.taps);
-        put_taps(cw, l.nch, l.q_cols, need(e, i, "attn_k_conv", G * M * p.dim, p.taps), 0, G * M, p.dim, l.dimp, p.taps);
-        put_taps(cw, l.nch, l.q_cols + l.k_cols, need(e, i, "attn_v_conv", G * p.vdim, p.taps), 0, G, p.vdim, l.vdp, p.taps);
-        l.out_mult = 1.0f;
-        if (M == 2) {                        // weight of the second map
-            double s[2] = {0.0, 0.0};
-            const char *const names[4] = {"attn_lambda_q1", "attn_lambda_k1", "attn_lambda_q2", "attn_lambda_k2"};
-            for (int j = 0; j < 2; j++) {
-                const std::vector<float> q = row_f32(need(e, i, names[2 * j], p.dim, 0), 0), k = row_f32(need(e, i, names[2 * j + 1], p.dim, 0), 0);
-                for (int d = 0; d < p.dim; d++) s[j] += (double)q[d] * k[d];
-            }
-            l.lambda = (float)(exp(s[0]) - exp(s[1]) + (double)p.diff);
-            l.out_mult = 1.0f - p.diff;
-        }
-        const bool vd_ok = p.maps == 1 ? l.vdp <= 256 : l.vdp <= 128;
-        if (!vd_ok || lg_win_pf_smem(p.maps, l.dimp, l.vdp) > PLAN_SMEM_SMALL) l.chunked = 0;
-        l.rt = !e->f32 && l.vdp <= 256 && lg_win_dec_smem(p.maps, l.dimp, l.vdp) <= PLAN_SMEM_MAX;
-        if ((size_t)(p.maps * (l.dimp + l.vdp) + p.maps * 128) * 4 > PLAN_SMEM_SMALL) { fprintf(stderr, "lg_b200: layer %d: head sizes beyond what the kernels hold\n", i); exit(1); }
+        w.conv[0] = mat_f32(need(e, i, "attn_q_conv", H * M * p.dim, p.taps));
+        w.conv[1] = mat_f32(need(e, i, "attn_k_conv", G * M * p.dim, p.taps));
+        w.conv[2] = mat_f32(need(e, i, "attn_v_conv", G * p.vdim, p.taps));
+        static const char *const names[4] = {"attn_lambda_q1", "attn_lambda_k1", "attn_lambda_q2", "attn_lambda_k2"};
+        if (M == 2) for (int j = 0; j < 4; j++) w.lam[j] = row_f32(need(e, i, names[j], p.dim, 0), 0);
     } else {
-        const int inner = H * p.vdim, gn = p.groups * p.state, x_at = l.ch0;
-        const struct gguf_tensor *t = need(e, i, "ssm_in", 2 * inner + 2 * gn + H, W), *c = need(e, i, "ssm_conv1d", inner + 2 * gn, p.taps);
-        const std::vector<float> bias = row_f32(need(e, i, "ssm_conv1d_bias", inner + 2 * gn, 0), 0);
+        const int inner = H * p.vdim, gn = p.groups * p.state;
+        const struct gguf_tensor *t = need(e, i, "ssm_in", 2 * inner + 2 * gn + H, W);
         auto sections = [&](int dst, int src, int n, int per, int to) {
             for (int s = 0; s < n; s++) for (int r = 0; r < per; r++) b.row(dst + s * to + r, t, src + s * per + r);
         };
-        std::vector<float> cb(l.nch, 0.0f);
-        const int part[3][5] = {{0, 0, H, p.vdim, l.vdp}, {H * l.vdp, inner, p.groups, p.state, l.np}, {H * l.vdp + p.groups * l.np, inner + gn, p.groups, p.state, l.np}};
-        sections(0, 0, H, p.vdim, l.vdp);                                  // z
-        for (auto &q : part) {                                             // x, B, C
-            sections(x_at + q[0], inner + q[1], q[2], q[3], q[4]);
-            put_taps(cw, l.nch, q[0], c, q[1], q[2], q[3], q[4], p.taps);
-            put_sections(cb, q[0], bias, q[1], q[2], q[3], q[4]);
-        }
+        sections(0, 0, H, p.vdim, l.vdp);                                  // z, x, B, C, step sizes
+        sections(l.ch0, inner, H, p.vdim, l.vdp);
+        sections(l.ch0 + H * l.vdp, 2 * inner, 2 * p.groups, p.state, l.np);
         sections(l.dt_off, 2 * inner + 2 * gn, 1, H, H);
-        l.conv_b = upload_f32(cb.data(), cb.size());
-        l.dt_bias = vec(e, i, "ssm_dt_bias", H); l.a_log = vec(e, i, "ssm_a_log", H); l.d = vec(e, i, "ssm_d", H);
-        std::vector<float> gn_w((size_t)H * l.vdp, 0.0f);
-        put_sections(gn_w, 0, row_f32(need(e, i, "ssm_norm", inner, 0), 0), 0, H, p.vdim, l.vdp);
-        l.gnorm = upload_f32(gn_w.data(), gn_w.size());
-        const int part_n = inner / p.norm_groups;
-        if (!l.npl || part_n > (p.vdim % 4 || part_n % 4 ? 16 : 32) * 1024) { fprintf(stderr, "lg_b200: layer %d: state-space sizes beyond what the kernels hold\n", i); exit(1); }
-        l.vs = std::min(l.vdp, 128);
-        if (lg_ssd_out_smem(l.np, l.vs) > PLAN_SMEM_SMALL) l.vs = std::min(l.vdp, 64);
-        if (lg_ssd_out_smem(l.np, l.vs) > PLAN_SMEM_MAX - 2048 || lg_ssd_state_smem(l.np, l.vs) > PLAN_SMEM_MAX - 2048) l.chunked = 0;
+        w.conv[0] = mat_f32(need(e, i, "ssm_conv1d", inner + 2 * gn, p.taps));
+        w.conv_b = row_f32(need(e, i, "ssm_conv1d_bias", inner + 2 * gn, 0), 0);
+        w.dt_bias = row_f32(need(e, i, "ssm_dt_bias", H, 0), 0); w.a_log = row_f32(need(e, i, "ssm_a_log", H, 0), 0); w.d = row_f32(need(e, i, "ssm_d", H, 0), 0);
+        w.norm = row_f32(need(e, i, "ssm_norm", inner, 0), 0);
     }
-    l.conv_w = upload_f32(cw.data(), cw.size());
+    if (!seq_layer_weights(e, i, l, w)) exit(1);
     const struct gguf_tensor *o = need(e, i, "attn_output", W, H * p.vdim);
     l.act_off = up(l.at_cols, 64);
     MatBuild c(e, W, l.act_off + (p.ff ? up(l.ffp, 64) : 0));
@@ -368,7 +390,8 @@ void launch_win(Engine *e, const PlanLayer &l, int form, int n, int q_rows, LgWi
     else launch_k(e, lg_win_pf_attn_kernel<1>, grid, dim3(lg_win_pf_threads<1>()), lg_win_pf_smem(1, l.dimp, l.vdp), mq, mc, a);
 }
 
-// The mixer of layer l with the state of slot `slot`: projection rows b.pj -> the first columns of b.at.
+// The mixer of layer l with the state of slot `slot`: projection rows b.pj -> the first columns of b.at.  Kernel classes: C_ATTN the
+// attention / state-space kernels, C_PLE the convolution and the gated norm around them.
 void seq_mixer(Engine *e, const struct kvcache *kv, const PlanLayer &l, int slot, const Pass &p, int only) {
     PlanBuf &b = *p.b;
     const struct lg_plan_layer &q = l.p;
@@ -381,11 +404,11 @@ void seq_mixer(Engine *e, const struct kvcache *kv, const PlanLayer &l, int slot
     c.run = p.n <= LG_MAXM ? LG_MAXM : 16;
     if (c.run < q.taps - 1) c.run = q.taps - 1;
     if (q.mixer == LG_MIX_GROUPED) {
-        if (!(only & C_ATTN)) return;
         uint8_t *rows = (uint8_t *)kv->k[slot];
         c.o[0] = {l.q_cols, b.q, l.q_cols, 0};
         c.o[1] = {l.nch, rows, l.ldc, kv->seq[slot]};
-        launch_conv(e, c, f32_rows);
+        if (only & C_PLE) launch_conv(e, c, f32_rows);
+        if (!(only & C_ATTN)) return;
         LgWinArgs a{};
         a.q = b.q; a.cache = rows; a.seq = kv->seq[slot]; a.pos = p.pos; a.out = b.at; a.ldo = l.o.ldk;
         launch_win(e, l, e->f32 ? 1 : p.wide ? (l.chunked ? 2 : 1) : l.rt ? 0 : 1, p.n, b.cap, a);
@@ -400,27 +423,25 @@ void seq_mixer(Engine *e, const struct kvcache *kv, const PlanLayer &l, int slot
     LgGatedNormArgs g{};
     g.y = b.y; g.ldy = inner; g.z = b.pj; g.ldz = l.in.rows; g.w = l.gnorm; g.vd = q.vdim; g.vdp = l.vdp; g.n = q.heads * q.vdim / q.norm_groups; g.eps = l.eps;
     g.out = b.at; g.ldo = l.o.ldk;
-    if (only & C_ATTN) {
-        if (!p.wide) launch_ssm_step(e, l, s, false);
-        else {
-            if (p.first && p.pos0 > 0) {                         // up to the block's start: states of the narrow block before it
-                LgSsmStepArgs r = s;
-                r.M = 0;
-                launch_ssm_step(e, l, r, false);
-            }
-            c.o[0] = {l.nch, b.cv, l.nch, 0};
-            c.silu = 1;
-            launch_conv(e, c, f32_rows);
-            const float *dt = e->f32 ? b.pj + l.dt_off : b.dt;
-            const int ld_dt = e->f32 ? l.in.rows : l.in.rows - l.dt_off;
-            if (l.chunked && !e->f32) launch_ssd(e, l, p.n, b.cap, b.cv, dt, ld_dt, b, state, p.pos0 == 0, b.y, inner);
-            else {
-                s.src = b.cv; s.ld = l.nch; s.dt_src = dt; s.ld_dt = ld_dt; s.fresh = p.pos0 == 0;
-                launch_ssm_step(e, l, s, true);
-            }
+    if (p.wide) {
+        if (p.first && p.pos0 > 0 && (only & C_ATTN)) {          // up to the block's start: states of the narrow block before it
+            LgSsmStepArgs r = s;
+            r.M = 0;
+            launch_ssm_step(e, l, r, false);
         }
-        launch_gated_norm(e, p.n, q.norm_groups, g, f32_rows);
-    }
+        c.o[0] = {l.nch, b.cv, l.nch, 0};
+        c.silu = 1;
+        if (only & C_PLE) launch_conv(e, c, f32_rows);
+        const float *dt = e->f32 ? b.pj + l.dt_off : b.dt;
+        const int ld_dt = e->f32 ? l.in.rows : l.in.rows - l.dt_off;
+        if (!(only & C_ATTN)) { }
+        else if (l.chunked && !e->f32) launch_ssd(e, l, p.n, b.cap, b.cv, dt, ld_dt, b, state, p.pos0 == 0, b.y, inner);
+        else {
+            s.src = b.cv; s.ld = l.nch; s.dt_src = dt; s.ld_dt = ld_dt; s.fresh = p.pos0 == 0;
+            launch_ssm_step(e, l, s, true);
+        }
+    } else if (only & C_ATTN) launch_ssm_step(e, l, s, false);
+    if (only & C_PLE) launch_gated_norm(e, p.n, q.norm_groups, g, f32_rows);
 }
 
 // x in place -> every layer run -> (with final_norm) the normed rows in b->h and, narrow, in e->hidden

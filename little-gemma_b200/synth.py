@@ -531,6 +531,112 @@ class LatentShape:
         return t
 
 
+@dataclass
+class SsmLayer:
+    """One state-space layer of a Baporax model (ff = 0: no feed-forward)."""
+    heads: int = 4
+    vdim: int = 32
+    state: int = 32
+    groups: int = 2
+    norm_groups: int = 2
+    conv: int = 4
+    ff: int = 96
+
+    type = "mamba2"
+
+    def mixer(self) -> dict:
+        return {"heads": self.heads, "vdim": self.vdim, "state": self.state, "groups": self.groups, "norm_groups": self.norm_groups, "conv": self.conv}
+
+    def tensors(self, W: int) -> Dict[str, tuple]:
+        inner, gn = self.heads * self.vdim, self.groups * self.state
+        return {"in": (2 * inner + 2 * gn + self.heads, W), "conv": (inner + 2 * gn, self.conv), "conv.b": (inner + 2 * gn,), "dt_bias": (self.heads,),
+                "A_log": (self.heads,), "D": (self.heads,), "norm": (inner,), "o": (W, inner)}
+
+
+@dataclass
+class DiffLayer:
+    """One layer of windowed differential attention of a Baporax model."""
+    heads: int = 4
+    kv_heads: int = 2
+    dim: int = 32                     # per map
+    vdim: int = 64
+    window: int = 50
+    conv: int = 3
+    diff: float = 0.4
+    scale: Optional[float] = None     # None: dim ** -0.5
+    ff: int = 96
+
+    type = "attention"
+
+    def mixer(self) -> dict:
+        return {"heads": self.heads, "kv_heads": self.kv_heads, "dim": self.dim, "vdim": self.vdim, "conv": self.conv, "diff": self.diff,
+                "scale": self.scale if self.scale is not None else self.dim ** -0.5, "mask": {"size": self.window}}
+
+    def tensors(self, W: int) -> Dict[str, tuple]:
+        q, k, v = self.heads * 2 * self.dim, self.kv_heads * 2 * self.dim, self.kv_heads * self.vdim
+        t = {"q": (q, W), "k": (k, W), "v": (v, W), "q.conv": (q, self.conv), "k.conv": (k, self.conv), "v.conv": (v, self.conv)}
+        t.update({n: (self.dim,) for n in ("lq1", "lk1", "lq2", "lk2")})
+        t["o"] = (W, self.heads * self.vdim)
+        return t
+
+
+@dataclass
+class HybridShape:
+    """A Baporax model: loop = (start, stop, times) or None."""
+    width: int
+    vocab: int
+    layers: list
+    loop: Optional[tuple] = None
+    eps: float = 1e-5
+    logit_scale: float = 1.0
+
+    def config(self) -> dict:
+        out = {"architecture": "Baporax", "width": self.width, "vocab": self.vocab, "norm": {"eps": self.eps}, "logit_scale": self.logit_scale,
+               "layers": [{"type": l.type, "mixer": l.mixer(), "mlp": {"kind": "dense", "ff": l.ff} if l.ff else None} for l in self.layers]}
+        if self.loop:
+            out["loop"] = dict(zip(("start", "stop", "times"), self.loop))
+        return out
+
+    def runs(self) -> list:
+        """the layers in the order of execution"""
+        if not self.loop:
+            return list(self.layers)
+        a, b, n = self.loop
+        return self.layers[:a] + self.layers[a:b] * n + self.layers[b:]
+
+    def tensors(self) -> Dict[str, tuple]:
+        W, t = self.width, {"embed": (self.vocab, self.width)}
+        if self.loop:
+            t["loop.step"] = (self.loop[2], W)
+        for i, l in enumerate(self.layers):
+            t[f"l{i}.norm1"] = (W,)
+            t.update({f"l{i}.mix.{k}": v for k, v in l.tensors(W).items()})
+            if l.ff:
+                t[f"l{i}.norm2"] = (W,)
+                t[f"l{i}.mlp.up"] = (l.ff, W); t[f"l{i}.mlp.down"] = (W, l.ff)
+        t["final.norm"] = (W,)
+        return t
+
+    def special(self, name: str, shape: tuple, rng) -> Optional[np.ndarray]:
+        """Values of the tensors that are not plain projections: norm weights around 0 (they are distances from 1), decays that
+        forget within tens to thousands of tokens, step sizes around 0.02 .. 0.5."""
+        leaf = name.split(".mix.")[-1] if ".mix." in name else name.split(".")[-1]
+        n = rng.standard_normal(shape)
+        if leaf in ("norm1", "norm2") or name == "final.norm":
+            return 0.2 * n
+        if leaf == "A_log":
+            return np.log(rng.uniform(0.02, 2.0, shape))
+        if leaf == "dt_bias":
+            return np.log(np.expm1(np.exp(rng.uniform(np.log(0.02), np.log(0.5), shape))))
+        if leaf in ("conv.b", "lq1", "lk1", "lq2", "lk2"):
+            return 0.2 * n
+        if leaf.endswith("conv"):
+            return n * shape[1] ** -0.5 + np.eye(1, shape[1], shape[1] - 1)
+        if name == "loop.step":
+            return 0.5 * n
+        return None
+
+
 def to_bf16(x: np.ndarray) -> np.ndarray:
     """float32 -> bf16 bit patterns (uint16), round to nearest even"""
     u = np.ascontiguousarray(x, dtype=np.float32).view(np.uint32)
@@ -541,7 +647,7 @@ def from_bf16(b: np.ndarray) -> np.ndarray:
     return (b.astype(np.uint32) << 16).view(np.float32)
 
 
-def random_weights(s: LatentShape, seed: int = 0, fast: bool = False) -> Dict[str, np.ndarray]:
+def random_weights(s, seed: int = 0, fast: bool = False) -> Dict[str, np.ndarray]:
     """Seeded bf16 weights (bit patterns): matrices N(0, 1/k) so that projections keep their input's size, norm weights around 1,
     sinks around 1, embeddings N(0, 1).  fast: big matrices repeat one random block (benchmarks, where only the sizes matter)."""
     rng = np.random.default_rng(seed)
@@ -549,7 +655,10 @@ def random_weights(s: LatentShape, seed: int = 0, fast: bool = False) -> Dict[st
     w = {}
     for name, shape in s.tensors().items():
         n = int(np.prod(shape))
-        if name.endswith("sink"):
+        own = s.special(name, shape, rng) if hasattr(s, "special") else None
+        if own is not None:
+            v = to_bf16(own)
+        elif name.endswith("sink"):
             v = to_bf16(1.0 + 0.5 * rng.standard_normal(shape))
         elif len(shape) == 1:
             v = to_bf16(1.0 + 0.2 * rng.standard_normal(shape))
@@ -563,7 +672,7 @@ def random_weights(s: LatentShape, seed: int = 0, fast: bool = False) -> Dict[st
     return w
 
 
-def write_checkpoint(path: str, s: LatentShape, seed: int = 0, weights: Optional[Dict[str, np.ndarray]] = None, fast: bool = False) -> str:
+def write_checkpoint(path: str, s, seed: int = 0, weights: Optional[Dict[str, np.ndarray]] = None, fast: bool = False) -> str:
     """A checkpoint folder at `path`: config.json and model.safetensors (bf16)."""
     import json
     os.makedirs(path, exist_ok=True)

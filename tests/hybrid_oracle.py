@@ -83,8 +83,13 @@ def softmax(scores, seen):
 def attention_map(q, k, v, scale, first, size):
     """q [n, H, d], k [keys, G, d], v [keys, G, vd] -> [n, H, vd]; head h reads group h // (H / G)"""
     of = np.arange(q.shape[1]) // (q.shape[1] // k.shape[1])
-    s = np.einsum("nhd,khd->hnk", q, k[:, of]) * scale
-    return np.einsum("hnk,khv->nhv", softmax(s, window_mask(len(q), len(k), first, size)), v[:, of])
+    out = []
+    for i in range(0, len(q), 256):                  # (keys that no query of the stretch sees are left out)
+        some = q[i:i + 256]
+        lo, hi = max(0, first + i - size + 1) if size else 0, min(len(k), first + i + len(some))
+        s = np.einsum("nhd,khd->hnk", some, k[lo:hi, of], optimize=True) * scale
+        out.append(np.einsum("hnk,khv->nhv", softmax(s, window_mask(len(some), hi - lo, first + i - lo, size)), v[lo:hi, of], optimize=True))
+    return np.concatenate(out)
 
 
 def differential(a1, a2, lam, diff, eps):

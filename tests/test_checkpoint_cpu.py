@@ -8,18 +8,14 @@ import numpy as np
 import pytest
 
 from tests import latent_oracle as o
-from tests.conftest import synth_module
+from tests.conftest import lg_module, synth_module
 from tests.latent_models import model, shapes
-
-
-class PlanLayer(C.Structure):
-    _fields_ = [(n, C.c_int) for n in ("mixer", "heads", "dim", "rot_dim", "vdim", "q_rank", "kv_rank", "kv_src", "rot_dims")] + \
-               [("scale", C.c_float), ("rot_base", C.c_float), ("ff", C.c_int)]
 
 
 class Plan(C.Structure):
     _fields_ = [(n, C.c_int) for n in ("n_layer", "width", "vocab", "norm_kind", "act")] + \
-               [("norm_eps", C.c_float), ("residual_mult", C.c_float), ("layer", C.POINTER(PlanLayer))]
+               [("norm_eps", C.c_float), ("residual_mult", C.c_float), ("layer", C.POINTER(lg_module().PlanLayer)), ("form", C.c_int),
+                ("norm_offset", C.c_float), ("logit_scale", C.c_float)] + [(n, C.c_int) for n in ("loop_start", "loop_stop", "loop_times")]
 
 
 class Tensor(C.Structure):
