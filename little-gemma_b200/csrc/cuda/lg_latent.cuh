@@ -408,15 +408,15 @@ lg_latent_pf_attn_kernel(const __grid_constant__ CUtensorMap tmq, const __grid_c
     const int kb = lg_latent_blocks(a.dimp), nb = kb + lg_latent_blocks(a.rotp), dq = a.dimp + a.rotp;
     unsigned char *sQ = (unsigned char *)(((uintptr_t)lat_smem + 1023) & ~(uintptr_t)1023), *sK = sQ + nb * Q_BYTES, *sV = sK + nb * K_BYTES;
     uint64_t *qfull = (uint64_t *)(sV + (size_t)a.vdp * 128), *kfull = qfull + 1, *kempty = qfull + 2, *vfull = qfull + 3, *vempty = qfull + 4,
-             *sfull = qfull + 5 /* two */, *pready = qfull + 7, *odone = qfull + 8;
-    uint32_t *tmem_slot = (uint32_t *)(qfull + 9);
+             *sfull = qfull + 5 /* two */, *pready = qfull + 7 /* two */, *odone = qfull + 9;
+    uint32_t *tmem_slot = (uint32_t *)(qfull + 10);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int h = blockIdx.y, qb = (gridDim.x - 1 - blockIdx.x) * LG_LP_Q;       // longest rows first
     const uint32_t tcols = a.vdp <= 128 ? 256 : 512;                             // S / P twice 64 columns, O vdp columns
 
     if (threadIdx.x == 0) {
         mbar_init(qfull, 1); mbar_init(kfull, 1); mbar_init(kempty, 1); mbar_init(vfull, 1); mbar_init(vempty, 1);
-        mbar_init(sfull, 1); mbar_init(sfull + 1, 1); mbar_init(pready, 128); mbar_init(odone, 1);
+        mbar_init(sfull, 1); mbar_init(sfull + 1, 1); mbar_init(pready, 128); mbar_init(pready + 1, 128); mbar_init(odone, 1);
     }
     if (warp == 5) {
         asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" :: "r"(smem_u32(tmem_slot)), "r"(tcols) : "memory");
@@ -479,7 +479,7 @@ lg_latent_pf_attn_kernel(const __grid_constant__ CUtensorMap tmq, const __grid_c
             ok = ok && scores(0);
             for (int i = 0; i < n_tiles && ok; i++) {
                 if (i + 1 < n_tiles) ok = scores(i + 1);
-                ok = ok && mbar_wait(pready, i & 1) && mbar_wait(vfull, i & 1);
+                ok = ok && mbar_wait(pready + (i & 1), (i >> 1) & 1) && mbar_wait(vfull, i & 1);
                 if (!ok) break;
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
                 const uint32_t tP = tmem + (i & 1) * LG_LP_S;
@@ -555,7 +555,7 @@ lg_latent_pf_attn_kernel(const __grid_constant__ CUtensorMap tmq, const __grid_c
             }
             tmem_wait_st();
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
-            mbar_arrive(pready);
+            mbar_arrive(pready + (i & 1));       // (a barrier per buffer: both tiles' weights may be ready before the products ask for the first)
         }
         ok = __all_sync(0xffffffffu, ok && mbar_wait(odone, (n_tiles - 1) & 1));
         if (!ok) atomicOr(a.err, LG_ERR_MBAR_TIMEOUT | 32);

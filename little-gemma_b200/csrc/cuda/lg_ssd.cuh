@@ -121,7 +121,7 @@ __global__ void __launch_bounds__(LG_SSD_THREADS) lg_ssd_state_kernel(const __gr
     }
     if (ok) ok = mbar_wait(done, 0);
     ok = __syncthreads_and(ok);
-    if (!ok && tid == 0) atomicOr(a.err, LG_ERR_MBAR_TIMEOUT | 16);
+    if (!ok && tid == 0) atomicOr(a.err, LG_ERR_MBAR_TIMEOUT | 512);
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
     if (ok)
         for (int m = 0; m < bm; m++) {
@@ -306,7 +306,7 @@ __global__ void __launch_bounds__(LG_SSD_THREADS) lg_ssd_out_kernel(const __grid
     }
     if (ok) ok = mbar_wait(ydone, 0);
     ok = __syncthreads_and(ok);
-    if (!ok && tid == 0) atomicOr(a.err, LG_ERR_MBAR_TIMEOUT | 32);
+    if (!ok && tid == 0) atomicOr(a.err, LG_ERR_MBAR_TIMEOUT | 1024);
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
     if (ok) {
         const float er = ex2(run);

@@ -317,7 +317,8 @@ __global__ void __launch_bounds__(LG_WM_THREADS) lg_win_merge_kernel(LgWinArgs a
 //   0 .. 4 MAPS - 1   map w / 4, one query row per thread: online softmax in f32, the weights back over the scores in tensor memory as bf16
 //                     high + low parts; the output is rescaled only when a row's maximum has grown by more than 2^LG_LP_SLACK;
 //   then one thread each:  Q and key tiles;  products;  value tiles (keys and values in two stages).
-// Per map tensor memory holds two score buffers of 64 columns and the output; values are an MN-major operand, as they lie in the cache.
+// Scores of two tiles may be finished before the first one's weights are used, so every buffer has barriers of its own: one barrier for both
+// would go through two phases behind a waiter's back.  Per map tensor memory holds two score buffers of 64 columns and the output; values are an MN-major operand, as they lie in the cache.
 // At the end both maps' rows sit in the same lanes: warps w and w + 4 share a row's columns, combine and norm them.
 #define LG_WP_Q 128
 #define LG_WP_S 64
@@ -335,7 +336,7 @@ lg_win_pf_attn_kernel(const __grid_constant__ CUtensorMap tmq, const __grid_cons
     const int kb = lg_ssd_blocks(a.dimp), vb = lg_ssd_blocks(a.vdp), nb = MAPS * kb, vo = (a.vdp + 31) & ~31;
     unsigned char *sQ = (unsigned char *)(((uintptr_t)win_smem + 1023) & ~(uintptr_t)1023), *sK = sQ + nb * Q_BYTES, *sV = sK + ST * nb * T_BYTES;
     uint64_t *qfull = (uint64_t *)(sV + ST * vb * T_BYTES), *kfull = qfull + 1, *kempty = kfull + ST, *vfull = kempty + ST, *vempty = vfull + ST,
-             *sfull = vempty + ST /* [map][2] */, *pready = sfull + 2 * MAPS, *odone = pready + MAPS;
+             *sfull = vempty + ST /* [map][2] */, *pready = sfull + 2 * MAPS /* [map][2] */, *odone = pready + 2 * MAPS;
     uint32_t *tmem_slot = (uint32_t *)(odone + MAPS);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int h = blockIdx.y, g = h / (a.H / a.G), qb = (gridDim.x - 1 - blockIdx.x) * LG_WP_Q;       // longest rows first
@@ -343,7 +344,7 @@ lg_win_pf_attn_kernel(const __grid_constant__ CUtensorMap tmq, const __grid_cons
     if (threadIdx.x == 0) {
         mbar_init(qfull, 1);
         for (int i = 0; i < ST; i++) { mbar_init(kfull + i, 1); mbar_init(kempty + i, 1); mbar_init(vfull + i, 1); mbar_init(vempty + i, 1); }
-        for (int i = 0; i < MAPS; i++) { mbar_init(sfull + 2 * i, 1); mbar_init(sfull + 2 * i + 1, 1); mbar_init(pready + i, 128); mbar_init(odone + i, 1); }
+        for (int i = 0; i < MAPS; i++) { mbar_init(sfull + 2 * i, 1); mbar_init(sfull + 2 * i + 1, 1); mbar_init(pready + 2 * i, 128); mbar_init(pready + 2 * i + 1, 128); mbar_init(odone + i, 1); }
     }
     if (warp == ROWW + 1) {
         asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" :: "r"(smem_u32(tmem_slot)), "r"(tcols) : "memory");
@@ -367,7 +368,7 @@ lg_win_pf_attn_kernel(const __grid_constant__ CUtensorMap tmq, const __grid_cons
             int i = 0;
             for (; i < n_tiles; i++) {
                 const int s = i % ST;
-                if (i >= ST && !mbar_wait(kempty + s, (i / ST - 1) & 1)) { atomicOr(a.err, LG_ERR_MBAR_TIMEOUT | 4); break; }
+                if (i >= ST && !mbar_wait(kempty + s, (i / ST - 1) & 1)) { atomicOr(a.err, LG_ERR_MBAR_TIMEOUT | 2048); break; }
                 mbar_expect_tx(kfull + s, nb * T_BYTES);
                 for (int m = 0; m < MAPS; m++)
                     for (int c = 0; c < kb; c++) tma_load_2d(sK + (s * nb + m * kb + c) * T_BYTES, &tmc, (g * MAPS + m) * a.dimp + c * 64, cache_row(i), kfull + s);
@@ -382,7 +383,7 @@ lg_win_pf_attn_kernel(const __grid_constant__ CUtensorMap tmq, const __grid_cons
             int i = 0;
             for (; i < n_tiles; i++) {
                 const int s = i % ST;
-                if (i >= ST && !mbar_wait(vempty + s, (i / ST - 1) & 1)) { atomicOr(a.err, LG_ERR_MBAR_TIMEOUT | 16); break; }
+                if (i >= ST && !mbar_wait(vempty + s, (i / ST - 1) & 1)) { atomicOr(a.err, LG_ERR_MBAR_TIMEOUT | 4096); break; }
                 mbar_expect_tx(vfull + s, vb * T_BYTES);
                 for (int c = 0; c < vb; c++) tma_load_2d(sV + (s * vb + c) * T_BYTES, &tmc, a.v_off + g * a.vdp + c * 64, cache_row(i), vfull + s);
             }
@@ -416,7 +417,7 @@ lg_win_pf_attn_kernel(const __grid_constant__ CUtensorMap tmq, const __grid_cons
                 ok = ok && mbar_wait(vfull + s, (i / ST) & 1);
                 #pragma unroll
                 for (int m = 0; m < MAPS; m++) {
-                    ok = ok && mbar_wait(pready + m, i & 1);
+                    ok = ok && mbar_wait(pready + 2 * m + (i & 1), (i >> 1) & 1);
                     if (!ok) break;
                     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
                     const uint64_t vd = umma_desc_mn128(smem_u32(sV + s * vb * T_BYTES), T_BYTES);
@@ -429,7 +430,7 @@ lg_win_pf_attn_kernel(const __grid_constant__ CUtensorMap tmq, const __grid_cons
                 }
                 umma_commit(vempty + s);
             }
-            if (!ok) atomicOr(a.err, LG_ERR_MBAR_TIMEOUT | 8);
+            if (!ok) atomicOr(a.err, LG_ERR_MBAR_TIMEOUT | 8192);
         }
     } else {
         const int map = warp >> 2, row = threadIdx.x & 127, tok = qb + row, q_pos = pos + tok, q_lo = lg_win_first(q_pos, a.window);
@@ -497,10 +498,10 @@ lg_win_pf_attn_kernel(const __grid_constant__ CUtensorMap tmq, const __grid_cons
             }
             tmem_wait_st();
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
-            mbar_arrive(pready + map);
+            mbar_arrive(pready + 2 * map + (i & 1));
         }
         ok = __all_sync(0xffffffffu, ok && mbar_wait(odone + map, (n_tiles - 1) & 1));
-        if (!ok) atomicOr(a.err, LG_ERR_MBAR_TIMEOUT | 32);
+        if (!ok) atomicOr(a.err, LG_ERR_MBAR_TIMEOUT | 16384);
         asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
         s_l[map][row] = l;
         asm volatile("bar.sync 1, %0;" :: "n"(MAPS * 128) : "memory");        // both maps' products have finished
