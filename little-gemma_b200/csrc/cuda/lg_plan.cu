@@ -51,7 +51,7 @@ struct PlanBuf {
     float *x = nullptr, *pj = nullptr, *o = nullptr, *gu = nullptr;
     void *h = nullptr, *cq = nullptr, *q = nullptr, *qa = nullptr, *ol = nullptr, *at = nullptr, *act = nullptr;
     void *h2 = nullptr, *cv = nullptr, *y = nullptr;          // second norm; convolved rows; state-space outputs
-    float *dt = nullptr, *ds = nullptr, *decay = nullptr; bf16 *s_hi = nullptr, *s_lo = nullptr;    // raw step sizes; chunk sums, decays and states
+    float *dt = nullptr; bf16 *s_hi = nullptr, *s_lo = nullptr;    // raw step sizes; states before every chunk
     std::vector<float2 *> tab;
     int *toks = nullptr, *pos = nullptr;                      // of the block (narrow: the engine's round state)
 };
@@ -197,7 +197,7 @@ void buf_alloc(Engine *e, PlanBuf &b, int cap, bool narrow) {
 void buf_free(PlanBuf &b, bool narrow) {
     if (!narrow) cudaFree(b.x);
     cudaFree(b.pj); cudaFree(b.o); cudaFree(b.gu); cudaFree(b.h); cudaFree(b.cq); cudaFree(b.q); cudaFree(b.qa); cudaFree(b.ol); cudaFree(b.at); cudaFree(b.act);
-    cudaFree(b.h2); cudaFree(b.cv); cudaFree(b.y); cudaFree(b.dt); cudaFree(b.ds); cudaFree(b.decay); cudaFree(b.s_hi); cudaFree(b.s_lo);
+    cudaFree(b.h2); cudaFree(b.cv); cudaFree(b.y); cudaFree(b.dt); cudaFree(b.s_hi); cudaFree(b.s_lo);
     for (auto t : b.tab) cudaFree(t);
     cudaFree(b.toks); cudaFree(b.pos);
     b = PlanBuf();

@@ -118,9 +118,8 @@ bool seq_layer_weights(const Engine *e, int i, PlanLayer &l, const SeqWeights &w
         l.dt_bias = upload_f32(w.dt_bias.data(), H); l.a_log = upload_f32(w.a_log.data(), H); l.d = upload_f32(w.d.data(), H);
         l.gnorm = upload_f32(gn_w.data(), gn_w.size());
         ok = l.npl && part_n <= (p.vdim % 4 || part_n % 4 ? 16 : 32) * 1024;
-        l.vs = std::min(l.vdp, 128);
-        if (lg_ssd_out_smem(l.np, l.vs) > PLAN_SMEM_SMALL) l.vs = std::min(l.vdp, 64);
-        if (l.np > 256 || lg_ssd_out_smem(l.np, l.vs) > PLAN_SMEM_MAX - 2048 || lg_ssd_state_smem(l.np, l.vs) > PLAN_SMEM_MAX - 2048) l.chunked = 0;
+        l.vs = std::min(l.vdp, 64);
+        if (l.np > 256) l.chunked = 0;
     }
     l.conv_w = upload_f32(cw.data(), cw.size());
     if (!ok) fprintf(stderr, "lg_b200: layer %d: sizes beyond what the kernels hold\n", i);
@@ -178,8 +177,36 @@ void seq_layer_load(Engine *e, int i, PlanLayer &l) {
 void seq_layer_free(PlanLayer &l) {
     for (float *v : {l.conv_w, l.conv_b, l.dt_bias, l.a_log, l.d, l.gnorm}) cudaFree(v);
 }
+// The kernels of a decode step ask for one division of an SM's memory between cache and shared memory (percent of the latter): where it
+// changes from one kernel to the next, the SM has to run empty first, and nothing overlaps.  64 KB hold the mixers' CTAs and leave the
+// weight stream of the matmuls the cache lines its loads in flight need.
+constexpr int STEP_CARVEOUT = 28;
+template <typename K> void same_carveout(K kernel) { LG_CHECK(cudaFuncSetAttribute(kernel, cudaFuncAttributePreferredSharedMemoryCarveout, STEP_CARVEOUT)); }
+template <int EPI> void gemv_carveout() {
+    same_carveout(lg_dn_gemv_kernel<EPI, 1, false>); same_carveout(lg_dn_gemv_kernel<EPI, 2, false>);
+    same_carveout(lg_dn_gemv_kernel<EPI, 4, false>); same_carveout(lg_dn_gemv_kernel<EPI, 8, false>);
+}
+template <typename T> void step_carveout() {
+    same_carveout(lg_ssm_step_kernel<T, 1, false>); same_carveout(lg_ssm_step_kernel<T, 2, false>);
+    same_carveout(lg_ssm_step_kernel<T, 4, false>); same_carveout(lg_ssm_step_kernel<T, 8, false>);
+}
+constexpr size_t SSM_SMEM = lg_ssm_step_smem(LG_CONV_MAX_TAPS, 256);
 void seq_attributes() {
     smem_attr(lg_dn_gemm_kernel<128, DN_G_RELU2>, dn_gemm_smem<128>()); smem_attr(lg_dn_gemm_kernel<256, DN_G_RELU2>, dn_gemm_smem<256>());
+    smem_attr(lg_ssm_step_kernel<float, 1, false>, SSM_SMEM); smem_attr(lg_ssm_step_kernel<float, 2, false>, SSM_SMEM);
+    smem_attr(lg_ssm_step_kernel<float, 4, false>, SSM_SMEM); smem_attr(lg_ssm_step_kernel<float, 8, false>, SSM_SMEM);
+    smem_attr(lg_ssm_step_kernel<bf16, 1, false>, SSM_SMEM); smem_attr(lg_ssm_step_kernel<bf16, 2, false>, SSM_SMEM);
+    smem_attr(lg_ssm_step_kernel<bf16, 4, false>, SSM_SMEM); smem_attr(lg_ssm_step_kernel<bf16, 8, false>, SSM_SMEM);
+    gemv_carveout<DN_STORE>(); gemv_carveout<DN_PAIR>(); gemv_carveout<DN_HEAD>();
+    step_carveout<bf16>();
+    same_carveout(lg_row_norm_kernel<bf16, 2, 4, true>); same_carveout(lg_row_norm_kernel<bf16, 4, 4, true>); same_carveout(lg_row_norm_kernel<bf16, 16, 1, true>);
+    same_carveout(lg_conv_kernel<float, bf16, 2>); same_carveout(lg_conv_kernel<float, bf16, 3>); same_carveout(lg_conv_kernel<float, bf16, 4>);
+    same_carveout(lg_conv_any_kernel<float, bf16>);
+    same_carveout(lg_gated_norm_kernel<float, bf16, 4, 2>); same_carveout(lg_gated_norm_kernel<float, bf16, 4, 8>);
+    same_carveout(lg_gated_norm_kernel<float, bf16, 1, 4>); same_carveout(lg_gated_norm_kernel<float, bf16, 1, 16>);
+    same_carveout(lg_win_dec_attn_kernel<1, 4>); same_carveout(lg_win_dec_attn_kernel<2, 4>); same_carveout(lg_win_dec_attn_kernel<2, 8>);
+    same_carveout(lg_win_merge_kernel<1>); same_carveout(lg_win_merge_kernel<2>);
+    same_carveout(lg_dn_embed_rows<bf16>); same_carveout(lg_seq_begin_kernel);
     smem_attr(lg_ssd_state_kernel, PLAN_SMEM_MAX - 2048); smem_attr(lg_ssd_out_kernel, PLAN_SMEM_MAX - 2048);
     smem_attr(lg_win_dec_attn_kernel<1, 4>); smem_attr(lg_win_dec_attn_kernel<2, 4>); smem_attr(lg_win_dec_attn_kernel<2, 8>);
     smem_attr(lg_win_pf_attn_kernel<1>, PLAN_SMEM_SMALL); smem_attr(lg_win_pf_attn_kernel<2>, PLAN_SMEM_SMALL);
@@ -215,7 +242,6 @@ void seq_buf_alloc(Engine *e, PlanBuf &b, int cap, bool narrow) {
         b.pos = dalloc<int>(1);
         if (!e->f32) {
             b.dt = dalloc<float>((size_t)cap * up((int)heads, 32) + 16);
-            b.ds = dalloc<float>(chunks * ds + 16); b.decay = dalloc<float>(chunks * heads + 16);
             b.s_hi = dalloc<bf16>(chunks * ds + 16); b.s_lo = dalloc<bf16>(chunks * ds + 16);
         }
     }
@@ -296,13 +322,14 @@ void seq_bind(Engine *e, const struct kvcache *kv) {
 // ------------------------------------------------------------------------------------------
 // mixers
 // ------------------------------------------------------------------------------------------
-template <typename TI, typename T> void conv_go(Engine *e, const LgConvArgs &a) {
+template <typename TI, typename T> void conv_go(Engine *e, LgConvArgs a) {
+    a.run = a.taps >= 2 && a.taps <= 4 ? LG_CONV_RUN : std::max(16, a.taps - 1);          // the first run alone reads the ring
     const dim3 grid((a.nch / LG_CONV_V + LG_CONV_THREADS - 1) / LG_CONV_THREADS, (a.M + a.run - 1) / a.run), block(LG_CONV_THREADS);
     switch (a.taps) {
     case 2: launch_k(e, lg_conv_kernel<TI, T, 2>, grid, block, 0, a); break;
     case 3: launch_k(e, lg_conv_kernel<TI, T, 3>, grid, block, 0, a); break;
     case 4: launch_k(e, lg_conv_kernel<TI, T, 4>, grid, block, 0, a); break;
-    default: launch_k(e, lg_conv_kernel<TI, T, 0>, grid, block, 0, a); break;
+    default: launch_k(e, lg_conv_any_kernel<TI, T>, grid, block, 0, a); break;
     }
 }
 void launch_conv(Engine *e, const LgConvArgs &a, bool f32_src) {
@@ -312,11 +339,12 @@ void launch_conv(Engine *e, const LgConvArgs &a, bool f32_src) {
 }
 template <typename T, bool WIDE> void step_go(Engine *e, const PlanLayer &l, const LgSsmStepArgs &a) {
     const dim3 grid(l.p.heads, l.vdp / LG_SSM_ROWS), block(LG_SSM_THREADS);
+    const size_t sm = WIDE ? 0 : lg_ssm_step_smem(a.taps, a.np);
     switch (l.npl) {
-    case 1: launch_k(e, lg_ssm_step_kernel<T, 1, WIDE>, grid, block, 0, a); break;
-    case 2: launch_k(e, lg_ssm_step_kernel<T, 2, WIDE>, grid, block, 0, a); break;
-    case 4: launch_k(e, lg_ssm_step_kernel<T, 4, WIDE>, grid, block, 0, a); break;
-    default: launch_k(e, lg_ssm_step_kernel<T, 8, WIDE>, grid, block, 0, a); break;
+    case 1: launch_k(e, lg_ssm_step_kernel<T, 1, WIDE>, grid, block, sm, a); break;
+    case 2: launch_k(e, lg_ssm_step_kernel<T, 2, WIDE>, grid, block, sm, a); break;
+    case 4: launch_k(e, lg_ssm_step_kernel<T, 4, WIDE>, grid, block, sm, a); break;
+    default: launch_k(e, lg_ssm_step_kernel<T, 8, WIDE>, grid, block, sm, a); break;
     }
 }
 void launch_ssm_step(Engine *e, const PlanLayer &l, const LgSsmStepArgs &a, bool wide) {
@@ -331,19 +359,33 @@ void launch_ssd(Engine *e, const PlanLayer &l, int n, int cap, const void *u, co
     LgSsdArgs a{};
     a.dt = dt; a.ld_dt = ld_dt; a.dt_bias = l.dt_bias; a.a_log = l.a_log; a.d = l.d;
     a.heads = H; a.groups = l.p.groups; a.np = l.np; a.vdp = l.vdp; a.vs = l.vs; a.n = n;
-    a.ds = b.ds; a.decay = b.decay; a.y = (bf16 *)y; a.ldy = ldy; a.err = e->err;
-    const dim3 grid(chunks, H, (l.vdp + l.vs - 1) / l.vs);
+    a.nst = l.nst; a.chunks = chunks; a.fresh = fresh; a.state = state; a.hi = b.s_hi; a.lo = b.s_lo; a.y = (bf16 *)y; a.ldy = ldy; a.err = e->err;
     const CUtensorMap &mu = buf_map(pm, u, l.nch, l.nch, cap, LG_SSD_Q);
-    launch_k(e, lg_ssd_state_kernel, grid, dim3(LG_SSD_THREADS), lg_ssd_state_smem(l.np, l.vs), mu, a);
-    LgSsdScanArgs s{};
-    s.ds = b.ds; s.decay = b.decay; s.heads = H; s.np = l.np; s.vdp = l.vdp; s.nst = l.nst; s.chunks = chunks; s.fresh = fresh;
-    s.state = state; s.hi = b.s_hi; s.lo = b.s_lo;
-    launch_k(e, lg_ssd_scan_kernel, dim3(H, l.nst / 32, (l.vdp + 31) / 32), dim3(LG_SSD_SCAN_THREADS), 0, s);
-    launch_k(e, lg_ssd_out_kernel, grid, dim3(LG_SSD_THREADS), lg_ssd_out_smem(l.np, l.vs), mu,
+    LgSsdArgs c = a;
+    const int tiles = H * ((l.np + 127) / 128);
+    c.vs = std::min(l.vdp, 64);                                  // fewer value columns per CTA while there are SMs without one
+    while (c.vs > 16 && tiles * ((l.vdp + c.vs - 1) / c.vs) * 2 <= e->sm_count + e->sm_count / 8) c.vs = up(c.vs / 2, 16);
+    launch_k(e, lg_ssd_state_kernel, dim3(H, (l.vdp + c.vs - 1) / c.vs, (l.np + 127) / 128), dim3(LG_SSD_STATE_THREADS), lg_ssd_state_smem(c.vs), mu, c);
+    // heads of a group that one CTA takes in turn (they share C B^T): the fewest rounds of CTAs, at about three heads' time to start one
+    const int per = H / l.p.groups, slices = (l.vdp + l.vs - 1) / l.vs;
+    long long best = 0;
+    for (int sp = 1; sp <= per; sp++) {
+        const long long rounds = ((long long)chunks * l.p.groups * slices * sp + e->sm_count - 1) / e->sm_count, cost = rounds * ((per + sp - 1) / sp + 3);
+        if (!best || cost < best) { best = cost; a.splits = sp; }
+    }
+    a.stages = lg_ssd_out_smem(l.np, 2) <= PLAN_SMEM_MAX - 2048 ? 2 : 1;
+    const dim3 grid(chunks, l.p.groups * a.splits, slices);
+    launch_k(e, lg_ssd_out_kernel, grid, dim3(LG_SSD_OUT_THREADS), lg_ssd_out_smem(l.np, a.stages), mu,
              buf_map(pm, b.s_hi, l.vdp, l.vdp, all, l.np), buf_map(pm, b.s_lo, l.vdp, l.vdp, all, l.np), a);
 }
 template <typename TI, typename TO> void gated_norm_go(Engine *e, int n, int parts, const LgGatedNormArgs &a) {
     const bool v4 = a.n % 4 == 0 && a.vd % 4 == 0;
+    if (v4 && a.n <= 1024 && n > LG_MAXM) {           // (few rows: more threads per part)
+        const dim3 grid((n * parts + LG_GN_WARPS - 1) / LG_GN_WARPS), block(LG_GN_WARPS * 32);
+        if (a.n <= 512) launch_k(e, lg_gated_norm_warp_kernel<TI, TO, 4>, grid, block, 0, a, parts, n);
+        else launch_k(e, lg_gated_norm_warp_kernel<TI, TO, 8>, grid, block, 0, a, parts, n);
+        return;
+    }
     const int items = v4 ? a.n / 4 : a.n, ipt_few = v4 ? 2 : 4;
     const int threads = std::min(1024, std::max(32, up((items + ipt_few - 1) / ipt_few, 32)));
     const bool few = (items + threads - 1) / threads <= ipt_few;
@@ -401,8 +443,6 @@ void seq_mixer(Engine *e, const struct kvcache *kv, const PlanLayer &l, int slot
     LgConvArgs c{};
     c.src = b.pj; c.ld = l.in.rows; c.ch0 = l.ch0; c.nch = l.nch; c.w = l.conv_w; c.bias = l.conv_b; c.taps = q.taps;
     c.ring = blk + sb.ring; c.mask = l.mask; c.pos = p.pos; c.M = p.n;
-    c.run = p.n <= LG_MAXM ? LG_MAXM : 16;
-    if (c.run < q.taps - 1) c.run = q.taps - 1;
     if (q.mixer == LG_MIX_GROUPED) {
         uint8_t *rows = (uint8_t *)kv->k[slot];
         c.o[0] = {l.q_cols, b.q, l.q_cols, 0};
