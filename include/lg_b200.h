@@ -9,6 +9,7 @@
 #define LG_B200_H
 
 #include "lg_abi.h"
+#include "lg_plan.h"
 
 #ifdef __cplusplus
 extern "C" {
@@ -184,7 +185,6 @@ int  lg_latent_prompt_attn_host(const float *q, const float *k, const float *k_r
 /* Layers whose mixer and feed-forward run side by side.  The stacked input projections: out = w x [n][m], act = relu(w_up x_up)^2
  * [n][m_up]; x += add + bias (either may be NULL) and the RMS norms of x with two weights; a mixer between its projections, run
  * block by block on projected rows (see lg_plan.cu; -2: sizes the kernels do not hold). */
-struct lg_plan_layer;
 int  lg_dense_pair_host(const float *w, int m, const float *w_up, int m_up, int k, const float *x, const float *x_up, int n, int f32,
                         float *out, float *act);
 int  lg_row_norm_pair_host(float *x, int rows, int n, const float *add, const float *bias, const float *norm_w, const float *norm_w2, float eps,
