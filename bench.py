@@ -30,7 +30,8 @@ one model (KV depth x verify width x acceptance) and writes them as markdown.
 
 --design mubopel times prefill and decode of the latent-attention design at sizes of real models' layers (random weights)
 beside the block-quantised family at equal width, heads, feed-forward, depth and vocabulary, kernel class by kernel class
-against its roofline; it replaces the benchmark line.
+against its roofline; it replaces the benchmark line.  --design baporax does the same for the state-space / windowed-attention
+design, beside the latent-attention one.
 
 N > 1 (torchrun): one independent replica per GPU, own prompt seed, no collective on the data
 path; a gloo barrier brackets the timed region and the max time over ranks is used.

@@ -359,6 +359,8 @@ __global__ void __launch_bounds__(LG_LM_THREADS) lg_latent_merge_kernel(LgLatent
 //                        high + low parts.  O is rescaled only when a row's maximum has grown by more than 2^LG_LP_SLACK since
 //                        the maximum in use -- until then the weights are merely larger than 1 -- which needs the previous
 //                        product to have finished.
+//   The rows can be two tiles ahead of the products, so the weights' and the products' barriers exist once per buffer: of one barrier for both,
+//   a parity could stand for the phase before or after the one that is waited for.
 // The softmax starts from the sink: maximum = sink, sum = 1.  The output gate is applied to the finished rows.
 #define LG_LP_Q 128
 #define LG_LP_S 64
@@ -408,15 +410,15 @@ lg_latent_pf_attn_kernel(const __grid_constant__ CUtensorMap tmq, const __grid_c
     const int kb = lg_latent_blocks(a.dimp), nb = kb + lg_latent_blocks(a.rotp), dq = a.dimp + a.rotp;
     unsigned char *sQ = (unsigned char *)(((uintptr_t)lat_smem + 1023) & ~(uintptr_t)1023), *sK = sQ + nb * Q_BYTES, *sV = sK + nb * K_BYTES;
     uint64_t *qfull = (uint64_t *)(sV + (size_t)a.vdp * 128), *kfull = qfull + 1, *kempty = qfull + 2, *vfull = qfull + 3, *vempty = qfull + 4,
-             *sfull = qfull + 5 /* two */, *pready = qfull + 7 /* two */, *odone = qfull + 9;
-    uint32_t *tmem_slot = (uint32_t *)(qfull + 10);
+             *sfull = qfull + 5 /* two */, *pready = qfull + 7 /* two */, *odone = qfull + 9 /* two */;
+    uint32_t *tmem_slot = (uint32_t *)(qfull + 11);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int h = blockIdx.y, qb = (gridDim.x - 1 - blockIdx.x) * LG_LP_Q;       // longest rows first
     const uint32_t tcols = a.vdp <= 128 ? 256 : 512;                             // S / P twice 64 columns, O vdp columns
 
     if (threadIdx.x == 0) {
         mbar_init(qfull, 1); mbar_init(kfull, 1); mbar_init(kempty, 1); mbar_init(vfull, 1); mbar_init(vempty, 1);
-        mbar_init(sfull, 1); mbar_init(sfull + 1, 1); mbar_init(pready, 128); mbar_init(pready + 1, 128); mbar_init(odone, 1);
+        mbar_init(sfull, 1); mbar_init(sfull + 1, 1); mbar_init(pready, 128); mbar_init(pready + 1, 128); mbar_init(odone, 1); mbar_init(odone + 1, 1);
     }
     if (warp == 5) {
         asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" :: "r"(smem_u32(tmem_slot)), "r"(tcols) : "memory");
@@ -488,7 +490,7 @@ lg_latent_pf_attn_kernel(const __grid_constant__ CUtensorMap tmq, const __grid_c
                 #pragma unroll
                 for (int j = 0; j < 4; j++) umma_f16_ta(tO, tP + 32 + 8 * j, vd + 2 * j, idO, 1u);
                 umma_commit(vempty);
-                umma_commit(odone);
+                umma_commit(odone + (i & 1));
             }
             if (!ok) atomicOr(a.err, LG_ERR_MBAR_TIMEOUT | 8);
         }
@@ -524,7 +526,7 @@ lg_latent_pf_attn_kernel(const __grid_constant__ CUtensorMap tmq, const __grid_c
             if (__any_sync(0xffffffffu, grow)) {
                 const float m_new = fmaxf(m, mt), alpha = exp2f(m - m_new);
                 if (i) {
-                    ok = __all_sync(0xffffffffu, mbar_wait(odone, (i - 1) & 1));
+                    ok = __all_sync(0xffffffffu, mbar_wait(odone + ((i - 1) & 1), ((i - 1) >> 1) & 1));
                     if (!ok) break;
                     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
                     for (int c = 0; c < a.vdp; c += 32) {
@@ -557,7 +559,7 @@ lg_latent_pf_attn_kernel(const __grid_constant__ CUtensorMap tmq, const __grid_c
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
             mbar_arrive(pready + (i & 1));       // (a barrier per buffer: both tiles' weights may be ready before the products ask for the first)
         }
-        ok = __all_sync(0xffffffffu, ok && mbar_wait(odone, (n_tiles - 1) & 1));
+        ok = __all_sync(0xffffffffu, ok && mbar_wait(odone + ((n_tiles - 1) & 1), ((n_tiles - 1) >> 1) & 1));
         if (!ok) atomicOr(a.err, LG_ERR_MBAR_TIMEOUT | 32);
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
         const float inv = 1.0f / l;

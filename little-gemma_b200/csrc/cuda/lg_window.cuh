@@ -317,8 +317,8 @@ __global__ void __launch_bounds__(LG_WM_THREADS) lg_win_merge_kernel(LgWinArgs a
 //   0 .. 4 MAPS - 1   map w / 4, one query row per thread: online softmax in f32, the weights back over the scores in tensor memory as bf16
 //                     high + low parts; the output is rescaled only when a row's maximum has grown by more than 2^LG_LP_SLACK;
 //   then one thread each:  Q and key tiles;  products;  value tiles (keys and values in two stages).
-// Scores of two tiles may be finished before the first one's weights are used, so every buffer has barriers of its own: one barrier for both
-// would go through two phases behind a waiter's back.  Per map tensor memory holds two score buffers of 64 columns and the output; values are an MN-major operand, as they lie in the cache.
+// Scores of two tiles may be finished before the first one's weights are used, so every buffer has barriers of its own, for its weights and
+// for the product with them: of one barrier for both, a parity could stand for the phase before or after the one that is waited for.  Per map tensor memory holds two score buffers of 64 columns and the output; values are an MN-major operand, as they lie in the cache.
 // At the end both maps' rows sit in the same lanes: warps w and w + 4 share a row's columns, combine and norm them.
 #define LG_WP_Q 128
 #define LG_WP_S 64
@@ -336,15 +336,15 @@ lg_win_pf_attn_kernel(const __grid_constant__ CUtensorMap tmq, const __grid_cons
     const int kb = lg_ssd_blocks(a.dimp), vb = lg_ssd_blocks(a.vdp), nb = MAPS * kb, vo = (a.vdp + 31) & ~31;
     unsigned char *sQ = (unsigned char *)(((uintptr_t)win_smem + 1023) & ~(uintptr_t)1023), *sK = sQ + nb * Q_BYTES, *sV = sK + ST * nb * T_BYTES;
     uint64_t *qfull = (uint64_t *)(sV + ST * vb * T_BYTES), *kfull = qfull + 1, *kempty = kfull + ST, *vfull = kempty + ST, *vempty = vfull + ST,
-             *sfull = vempty + ST /* [map][2] */, *pready = sfull + 2 * MAPS /* [map][2] */, *odone = pready + 2 * MAPS;
-    uint32_t *tmem_slot = (uint32_t *)(odone + MAPS);
+             *sfull = vempty + ST /* [map][2] */, *pready = sfull + 2 * MAPS /* [map][2] */, *odone = pready + 2 * MAPS /* [map][2] */;
+    uint32_t *tmem_slot = (uint32_t *)(odone + 2 * MAPS);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int h = blockIdx.y, g = h / (a.H / a.G), qb = (gridDim.x - 1 - blockIdx.x) * LG_WP_Q;       // longest rows first
     const uint32_t tcols = lg_tmem_cols(MAPS * (2 * LG_WP_S + vo));
     if (threadIdx.x == 0) {
         mbar_init(qfull, 1);
         for (int i = 0; i < ST; i++) { mbar_init(kfull + i, 1); mbar_init(kempty + i, 1); mbar_init(vfull + i, 1); mbar_init(vempty + i, 1); }
-        for (int i = 0; i < MAPS; i++) { mbar_init(sfull + 2 * i, 1); mbar_init(sfull + 2 * i + 1, 1); mbar_init(pready + 2 * i, 128); mbar_init(pready + 2 * i + 1, 128); mbar_init(odone + i, 1); }
+        for (int i = 0; i < MAPS; i++) { mbar_init(sfull + 2 * i, 1); mbar_init(sfull + 2 * i + 1, 1); mbar_init(pready + 2 * i, 128); mbar_init(pready + 2 * i + 1, 128); mbar_init(odone + 2 * i, 1); mbar_init(odone + 2 * i + 1, 1); }
     }
     if (warp == ROWW + 1) {
         asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" :: "r"(smem_u32(tmem_slot)), "r"(tcols) : "memory");
@@ -426,7 +426,7 @@ lg_win_pf_attn_kernel(const __grid_constant__ CUtensorMap tmq, const __grid_cons
                     for (int j = 0; j < 4; j++) umma_f16_ta(tO + m * vo, tP + 8 * j, vd + 128 * j, idO, (i | j) ? 1u : 0u);
                     #pragma unroll
                     for (int j = 0; j < 4; j++) umma_f16_ta(tO + m * vo, tP + 32 + 8 * j, vd + 128 * j, idO, 1u);
-                    umma_commit(odone + m);
+                    umma_commit(odone + 2 * m + (i & 1));
                 }
                 umma_commit(vempty + s);
             }
@@ -467,7 +467,7 @@ lg_win_pf_attn_kernel(const __grid_constant__ CUtensorMap tmq, const __grid_cons
             if (__any_sync(0xffffffffu, grow)) {
                 const float m_new = fmaxf(m, mt), alpha = exp2f(m - m_new);
                 if (i) {
-                    ok = __all_sync(0xffffffffu, mbar_wait(odone + map, (i - 1) & 1));
+                    ok = __all_sync(0xffffffffu, mbar_wait(odone + 2 * map + ((i - 1) & 1), ((i - 1) >> 1) & 1));
                     if (!ok) break;
                     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
                     for (int c = 0; c < a.vdp; c += 32) {
@@ -500,7 +500,7 @@ lg_win_pf_attn_kernel(const __grid_constant__ CUtensorMap tmq, const __grid_cons
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
             mbar_arrive(pready + 2 * map + (i & 1));
         }
-        ok = __all_sync(0xffffffffu, ok && mbar_wait(odone + map, (n_tiles - 1) & 1));
+        ok = __all_sync(0xffffffffu, ok && mbar_wait(odone + 2 * map + ((n_tiles - 1) & 1), ((n_tiles - 1) >> 1) & 1));
         if (!ok) atomicOr(a.err, LG_ERR_MBAR_TIMEOUT | 16384);
         asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
         s_l[map][row] = l;

@@ -19,6 +19,8 @@ def shapes():
         "big": H(256, 520, [S(heads=10, vdim=64, state=128, groups=2, norm_groups=2, ff=512), A(heads=8, kv_heads=2, dim=64, vdim=128, window=200, ff=384)], loop=(0, 2, 2), logit_scale=4.0),
         # beyond what the prompt kernels hold: wide values, states of 200 columns with wide heads
         "huge": H(64, 96, [A(heads=2, kv_heads=1, dim=144, vdim=272, window=40, ff=64), S(heads=2, vdim=144, state=250, groups=1, norm_groups=2, ff=64)], loop=(1, 2, 1)),
+        # many layers of few, large CTAs: kernels of several layers are resident at once, and finished scores wait for slow products
+        "deep": H(128, 120, [A(heads=16, kv_heads=4, dim=64, vdim=128, window=150, ff=512) for _ in range(8)] + [S(heads=24, vdim=64, state=128, groups=4, norm_groups=4, ff=512)]),
         # one kind of layer each, no feed-forward anywhere; a vocabulary beyond one pass of the head's CTAs
         "states": H(64, 9000, [S(heads=8, vdim=16, state=16, groups=8, norm_groups=8, ff=0) for _ in range(2)], loop=(0, 1, 4), logit_scale=1.7),
         "windows": H(72, 150, [A(heads=6, kv_heads=2, dim=24, vdim=24, window=64 + i, ff=0) for i in range(3)], loop=(2, 3, 2)),

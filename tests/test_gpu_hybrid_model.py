@@ -117,6 +117,16 @@ def test_verify_rows_equal_plain_steps(lg, case):
                 s.prefill(toks[:base])
 
 
+def test_prompts_through_many_resident_kernels(lg):
+    c = Case("deep", 400, seed=3)
+    with lg.Session(c.path, None, 420) as s:
+        first = run(s, c.toks, [400])
+        c.check(first, "bfloat16")
+        for _ in range(20):
+            s.prefill(c.toks[:100])
+            assert np.array_equal(run(s, c.toks, [400]), first)
+
+
 def test_positions_without_state_are_refused(lg):
     c = Case("looped", 80)
     with lg.Session(c.path, None, 200) as s:
@@ -230,3 +240,25 @@ def test_trace_replay(lg, tmp_path, dtype):
         if i in expect:
             got = np.fromfile(f, "<f4").reshape(expect[i].shape)
             assert np.sqrt(np.square(got - expect[i]).mean(axis=1)).max() / ca.scale < ca.tol[dtype]
+
+
+@pytest.mark.parametrize("family,name", [("hybrid", "big"), ("hybrid", "looped"), ("hybrid", "deep"), ("latent", "mixed"), ("latent", "big")])
+def test_bits_do_not_depend_on_what_the_caches_hold(lg, family, name):
+    """Prompts and steps behind an overwritten L2: copies and code arrive late and in another order, the bits stay."""
+    import torch
+    from tests import latent_models
+    shape, _, path = model(name) if family == "hybrid" else latent_models.model(name)
+    toks = synth_module().prompt_ids(330, shape.vocab, seed=31)
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")
+    with lg.Session(path, None, 340) as s:
+        want = run(s, toks, [320, 1])
+        for k in range(60):
+            flush.zero_()
+            torch.cuda.synchronize()
+            got = s.prefill_logits(toks[:320], 0, range(320))
+            assert np.array_equal(got, want[:320]), int(np.flatnonzero((got != want[:320]).any(axis=1))[0])
+            if k % 10 == 0:
+                for i in range(320, 330):
+                    flush.zero_()
+                    torch.cuda.synchronize()
+                    assert np.array_equal(s.prefill_logits(toks[i:i + 1], i, [0]), want[i:i + 1])
